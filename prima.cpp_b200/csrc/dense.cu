@@ -19,7 +19,7 @@ extern std::atomic<uint64_t> g_launches;
 namespace pb {
 
 int launch_dense_tc(const __nv_bfloat16 * A, int64_t lda, const __nv_bfloat16 * W, int64_t ldw, float * C, int64_t ldc, int T, int N, int K,
-                    const float * bias, const float * resid, int64_t ldr, float alpha, cudaStream_t stream);   // dense_tc.cu
+                    const float * bias, const float * resid, int64_t ldr, float alpha, cudaStream_t stream, int plane_rows = 0, int64_t a_plane = 0);   // dense_tc.cu
 bool dense_tc_ok(int T, int N, int K, int64_t lda, int64_t ldw, const void * A, const void * W);
 int launch_dense_tc_grouped(const __nv_bfloat16 * A, int64_t lda, const __nv_bfloat16 * W, int64_t ldw, int64_t w_stride, float * C, int64_t ldc,
                             const int32_t * start, const int32_t * count, int groups, int max_rows, int N, int K, cudaStream_t st);
@@ -109,12 +109,13 @@ template <int N> __device__ __forceinline__ void unpack(const uint4 & raw, float
 template <typename WT, int TB, bool VEC>
 __global__ void __launch_bounds__(256) k_dense_rows(const WT * __restrict__ A, int64_t lda, const WT * __restrict__ W, int64_t ldw, float * C, int64_t ldc,
                                                     int T, int N, int K, const float * __restrict__ bias, const float * resid, int64_t ldr, float alpha,
-                                                    int KS) {
+                                                    int KS, int plane_rows, int64_t a_plane) {
     __shared__ float parts[8][TB];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int rows_per_cta = (blockDim.x >> 5) / KS;
     const int n = blockIdx.x * rows_per_cta + warp / KS, part = warp % KS;
     const bool live = n < N;
+    if (plane_rows > 0) A += (int64_t) (n / plane_rows) * a_plane;   // several products over operands of their own (n < N: a valid plane)
     constexpr int V = Vec16<WT>::n;
     const int Kc = KS == 1 ? K : ((K + KS - 1) / KS + 32 * V - 1) / (32 * V) * (32 * V);
     const int k_begin = part * Kc, k_end = min(K, k_begin + Kc);
@@ -195,24 +196,24 @@ int rows_max_t() {
 
 template <typename WT>
 int dense_typed(const WT * A, int64_t lda, const WT * W, int64_t ldw, float * C, int64_t ldc, int T, int N, int K, const float * bias,
-                const float * resid, int64_t ldr, float alpha, cudaStream_t st) {
+                const float * resid, int64_t ldr, float alpha, cudaStream_t st, int plane_rows = 0, int64_t a_plane = 0) {
     if (T <= ROWS_MAX_T) {
         constexpr int V = Vec16<WT>::n;
-        const bool vec = K % V == 0 && lda % V == 0 && ldw % V == 0 && ((uintptr_t) A & 15) == 0 && ((uintptr_t) W & 15) == 0;
+        const bool vec = K % V == 0 && lda % V == 0 && ldw % V == 0 && a_plane % V == 0 && ((uintptr_t) A & 15) == 0 && ((uintptr_t) W & 15) == 0;
         // warps per row: few rows leave most of the machine's load slots empty, so 2, 4 or 8 warps split a long row
         int KS = 1;
         while (KS < 8 && (int64_t) N * KS < 6144 && K / (2 * KS) >= 1024) KS *= 2;
         const dim3 grid((unsigned) ((N + 8 / KS - 1) / (8 / KS))), block(256);
         g_launches++;
         if (T <= 1) {
-            if (vec) k_dense_rows<WT, 1, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS);
-            else k_dense_rows<WT, 1, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS);
+            if (vec) k_dense_rows<WT, 1, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
+            else k_dense_rows<WT, 1, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
         } else if (T <= 4) {
-            if (vec) k_dense_rows<WT, 4, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS);
-            else k_dense_rows<WT, 4, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS);
+            if (vec) k_dense_rows<WT, 4, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
+            else k_dense_rows<WT, 4, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
         } else {
-            if (vec) k_dense_rows<WT, ROWS_MAX_T, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS);
-            else k_dense_rows<WT, ROWS_MAX_T, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS);
+            if (vec) k_dense_rows<WT, ROWS_MAX_T, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
+            else k_dense_rows<WT, ROWS_MAX_T, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
         }
         return (int) cudaGetLastError();
     }
@@ -235,6 +236,28 @@ int launch_dense_grouped(int type, const void * A, int64_t lda, const void * W, 
                          const int32_t * count, int groups, int max_rows, int N, int K, cudaStream_t st) {
     if (!dense_grouped_ok(type, N, K, lda, ldw, w_stride, A, W)) return (int) cudaErrorInvalidValue;
     return launch_dense_tc_grouped((const __nv_bfloat16 *) A, lda, (const __nv_bfloat16 *) W, ldw, w_stride, C, ldc, start, count, groups, max_rows, N, K, st);
+}
+
+int launch_dense_planes(int type, const void * A, int64_t a_plane, int64_t lda, const void * W, int64_t ldw, float * C, int64_t ldc, int planes, int T, int N,
+                        int K, cudaStream_t st) {
+    if (T <= 0 || N <= 0 || planes <= 0) return 0;
+    if (K <= 0 || !A || !W || !C || (type != 0 && type != T_BF16)) return (int) cudaErrorInvalidValue;
+    const bool tc = type == T_BF16 && T > rows_max_t() && a_plane % 8 == 0 && dense_tc_ok(T, N, K, lda, ldw, A, W);
+    if (tc && N % 128 == 0)   // a weight tile lies inside one plane: one launch
+        return launch_dense_tc((const __nv_bfloat16 *) A, lda, (const __nv_bfloat16 *) W, ldw, C, ldc, T, planes * N, K, nullptr, nullptr, 0, 1.f, st, N, a_plane);
+    if (!tc && T <= ROWS_MAX_T) {
+        if (type == 0)
+            return dense_typed<float>((const float *) A, lda, (const float *) W, ldw, C, ldc, T, planes * N, K, nullptr, nullptr, 0, 1.f, st, N, a_plane);
+        return dense_typed<__nv_bfloat16>((const __nv_bfloat16 *) A, lda, (const __nv_bfloat16 *) W, ldw, C, ldc, T, planes * N, K, nullptr, nullptr, 0, 1.f, st, N,
+                                          a_plane);
+    }
+    const size_t es = type == T_BF16 ? 2 : 4;
+    for (int p = 0; p < planes; p++) {
+        const int rc = launch_dense(type, (const uint8_t *) A + (size_t) p * a_plane * es, lda, (const uint8_t *) W + (size_t) p * N * ldw * es, ldw, C + (int64_t) p * N,
+                                    ldc, T, N, K, nullptr, nullptr, 0, 1.f, st);
+        if (rc) return rc;
+    }
+    return 0;
 }
 
 int launch_dense(int type, const void * A, int64_t lda, const void * W, int64_t ldw, float * C, int64_t ldc, int T, int N, int K, const float * bias,

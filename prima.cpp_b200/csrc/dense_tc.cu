@@ -38,6 +38,8 @@ struct TcParams {
     // The counts live on the device: blockIdx.y numbers the token tiles of all groups in a row (group 0's tiles, then group 1's, ...), the
     // grid has room for the most tiles there can be (rows / BN + groups) and a CTA past the last tile leaves at once.
     const int32_t * grp_start; const int32_t * grp_count; int64_t grp_w_stride; int groups;
+    // planes: weight rows [p * plane_rows, + plane_rows) meet the operand a_plane * p elements further on (plane_rows a multiple of the row tile)
+    int plane_rows; int64_t a_plane;
 };
 
 __device__ __forceinline__ uint64_t desc_sw128(uint32_t saddr) {   // K-major, SWIZZLE_128B: rows of 128 B, 8-row groups 1024 B apart
@@ -86,6 +88,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constan
     const __nv_bfloat16 * Am = P.A, * Wm = P.W;
     float * Cm = P.C;
     int Tn = P.T, tile_y = blockIdx.y;
+    if (P.plane_rows > 0) Am += (int64_t) ((blockIdx.x * TC_BM) / P.plane_rows) * P.a_plane;
     if (P.grp_count) {
         int g = 0;
         for (; g < P.groups; g++) {
@@ -224,8 +227,8 @@ bool dense_tc_ok(int T, int N, int K, int64_t lda, int64_t ldw, const void * A, 
 }
 
 int launch_dense_tc(const __nv_bfloat16 * A, int64_t lda, const __nv_bfloat16 * W, int64_t ldw, float * C, int64_t ldc, int T, int N, int K, const float * bias,
-                    const float * resid, int64_t ldr, float alpha, cudaStream_t st) {
-    TcParams P{A, lda, W, ldw, C, ldc, bias, resid, ldr, alpha, T, N, K, abort_flag(), nullptr, nullptr, 0, 0};
+                    const float * resid, int64_t ldr, float alpha, cudaStream_t st, int plane_rows, int64_t a_plane) {
+    TcParams P{A, lda, W, ldw, C, ldc, bias, resid, ldr, alpha, T, N, K, abort_flag(), nullptr, nullptr, 0, 0, plane_rows, a_plane};
     return T <= 64 ? launch_tc<64>(P, st) : T <= 128 ? launch_tc<128>(P, st) : launch_tc<256>(P, st);
 }
 
@@ -233,7 +236,7 @@ int launch_dense_tc_grouped(const __nv_bfloat16 * A, int64_t lda, const __nv_bfl
                             const int32_t * start, const int32_t * count, int groups, int max_rows, int N, int K, cudaStream_t st) {
     if (groups <= 0 || max_rows <= 0) return 0;
     // T bounds the grid only (all groups together hold max_rows rows); the kernel reads each group's own count
-    TcParams P{A, lda, W, ldw, C, ldc, nullptr, nullptr, 0, 1.f, max_rows, N, K, abort_flag(), start, count, w_stride, groups};
+    TcParams P{A, lda, W, ldw, C, ldc, nullptr, nullptr, 0, 1.f, max_rows, N, K, abort_flag(), start, count, w_stride, groups, 0, 0};
     const int avg = (max_rows + groups - 1) / groups;   // the token tile follows the expected rows of a group
     return avg <= 64 ? launch_tc<64>(P, st) : avg <= 128 ? launch_tc<128>(P, st) : launch_tc<256>(P, st);
 }

@@ -2,7 +2,7 @@
 // stream around it (declarations and semantics: layers.h): hashed bigram embedding; a short causal convolution over a range of projection
 // channels with the slot's last inputs as history; the preparation of attention inputs (RMS norm over a whole projection or per head,
 // partial rotation by position in either pair layout, values turned by their position) with the cache store; turning an attention
-// result back + gate; gated linear recurrences whose decay comes with every token (gated delta rule, HGRN2) with the state in registers;
+// result back + gate; gated linear recurrences whose decay comes with every token (gated delta rule, HGRN2, WKV) with the state in registers;
 // two normed branch results joined onto the stream with the next norm in the same pass.  Everything here is fp32: positions, angles,
 // norms, decays, the recurrent state and what enters it; only a value written for a dense product takes its operand type.
 #include <cuda_bf16.h>
@@ -90,7 +90,8 @@ __device__ __forceinline__ void pair_of(int i, int dims, int layout, int & ia, i
 
 // One CTA per token.  (1) RMS norm over the whole query projection and over the whole key projection with weights; (2) rotation of the
 // leading entries of every query and key head; (3) every head divided by its own root mean square; (4) rotation of the value heads;
-// (5) the K / V rows later tokens can still see go to the cache.  Steps that the design does not have are skipped.
+// (3b) every query head times its own factor; (5) the K / V rows later tokens can still see go to the cache.  Steps that the design does not
+// have are skipped.
 // cs: scratch of rot_dims + vdim floats in shared memory: the token's cosines and sines, computed once for all heads
 __device__ __forceinline__ void attn_prep_rows(float * qr, float * kr, float * vr, float fp, const AttnParams & a, const AttnPrep & pr, float * red, float * cs) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -133,6 +134,10 @@ __device__ __forceinline__ void attn_prep_rows(float * qr, float * kr, float * v
             const float inv = 1.f / sqrtf(wsum(ss) / (float) a.dim + pr.eps);
             for (int i = lane; i < a.dim; i += 32) hv[i] *= inv;
         }
+    }
+    if (pr.q_scale) {
+        if (pr.norm == QKN_HEAD_UNIT) __syncthreads();
+        for (int i = threadIdx.x; i < QD; i += blockDim.x) qr[i] *= pr.q_scale[i / a.dim];
     }
     if (pr.v_rot && a.vdim > 1) {
         const int hp = a.vdim / 2, total = a.kv_heads * hp;
@@ -332,12 +337,16 @@ __global__ void __launch_bounds__(128) k_dual_post(const float * __restrict__ o,
 // n = NREG ng .. NREG ng + NREG - 1 (consecutive, so that a token's k and q entries come out of shared memory as 16-byte loads).  Tokens are walked in chunks of 16 whose q, k (or per-channel decay) rows, v columns and per-head
 // numbers go through registers into shared memory; the loads of the next chunk are in flight while the current one runs.  A token costs a
 // thread NREG fused steps and the column ONE shuffle reduction: for the delta rule the products of the OLD state with k and with q are
-// reduced together (with k . q), and  u = beta (v - g S_old^T k),  y = g S_old^T q + u (k . q)  follow without a second pass.
+// reduced together (with k . q), and  u = beta (v - g S_old^T k),  y = g S_old^T q + u (k . q)  follow without a second pass.  The bonus form
+// stages the decay rows as well and, once per chunk, one warp per token sums q . (u k), so that a token costs  y = S^T q + (q . u k) v  and
+// S <- diag(w) S + k v^T.
 constexpr int GCHUNK = 16, GCOLS = 16;
-template <int NREG, int LN, bool DELTA, bool CHAN>
+enum : int { GL_DELTA = 0, GL_TIED = 1, GL_BONUS = 2 };
+template <int NREG, int LN, int MODE>
 __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
                                                                   GatedLinParams p, float * __restrict__ state, int64_t slot_stride, float * __restrict__ y) {
     extern __shared__ float sm[];
+    constexpr bool DELTA = MODE == GL_DELTA, TIED = MODE == GL_TIED, BONUS = MODE == GL_BONUS;
     constexpr int NT = GCOLS * LN;
     constexpr int NV = (GCHUNK * GCOLS + NT - 1) / NT;
     const int N = p.dim, P = p.vdim, inner = p.heads * p.vdim;
@@ -350,7 +359,8 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
     float * Ks = sm;                        // [GCHUNK][N]  key, or the per-channel decay when the key is tied to it
     float * Qs = Ks + GCHUNK * N;           // [GCHUNK][N]
     float * Vs = Qs + GCHUNK * N;           // [GCHUNK][GCOLS]
-    float * Gs = Vs + GCHUNK * GCOLS;       // [GCHUNK] decay per token (one per head), [GCHUNK] beta
+    float * Gs = Vs + GCHUNK * GCOLS;       // [GCHUNK] decay per token (one per head) or the bonus product q . (u k), [GCHUNK] beta
+    float * Ws = Gs + 2 * GCHUNK;           // [GCHUNK][N]  BONUS: the decay per channel
     float * gst = state + (int64_t) slot[e] * slot_stride + (int64_t) h * N * P;
     float S[NREG];
 #pragma unroll
@@ -377,7 +387,7 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
             }
         }
     };
-    float rk[NREG], rq[NREG], rv[NV], rg = 0.f;
+    float rk[NREG], rq[NREG], rw[BONUS ? NREG : 1], rv[NV], rg = 0.f;
     auto fetch = [&](int c0) {
         const int nc = min(GCHUNK, n - c0);
 #pragma unroll
@@ -386,7 +396,8 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
             if (i < nc * N) {
                 const int tt = i / N, nn = i - tt * N;
                 const int64_t tok = t0 + c0 + tt;
-                rk[k] = CHAN ? io.decay[tok * io.ldd + hk * N + nn] : io.k[tok * io.ldk + hk * N + nn];
+                rk[k] = TIED ? io.decay[tok * io.ldd + hk * N + nn] : io.k[tok * io.ldk + hk * N + nn];
+                if constexpr (BONUS) rw[k] = io.decay[tok * io.ldd + hk * N + nn];
                 rq[k] = io.q[tok * io.ldq + hk * N + nn];
             }
         }
@@ -395,11 +406,11 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
             const int i = tid + NT * k, tt = i / GCOLS, pp = i - tt * GCOLS;
             rv[k] = (tt < nc && pt * GCOLS + pp < P) ? io.v[(int64_t) (t0 + c0 + tt) * io.ldv + h * P + pt * GCOLS + pp] : 0.f;
         }
-        if (tid < 2 * GCHUNK) {
+        if (!BONUS && tid < 2 * GCHUNK) {
             const int tt = tid & (GCHUNK - 1);
             rg = 0.f;
             if (tt < nc) {
-                if (tid < GCHUNK) { if (!CHAN) rg = io.decay[(int64_t) (t0 + c0 + tt) * io.ldd + h]; }
+                if (tid < GCHUNK) { if (DELTA) rg = io.decay[(int64_t) (t0 + c0 + tt) * io.ldd + h]; }
                 else if (DELTA) rg = io.beta[(int64_t) (t0 + c0 + tt) * io.ldb + h];
             }
         }
@@ -411,14 +422,27 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
 #pragma unroll
         for (int k = 0; k < NREG; k++) {
             const int i = tid + NT * k;
-            if (i < nc * N) { Ks[i] = rk[k]; Qs[i] = rq[k]; }
+            if (i < nc * N) {
+                Ks[i] = rk[k]; Qs[i] = rq[k];
+                if constexpr (BONUS) Ws[i] = rw[k];
+            }
         }
 #pragma unroll
         for (int k = 0; k < NV; k++)
             if (tid + NT * k < GCHUNK * GCOLS) Vs[tid + NT * k] = rv[k];
-        if (tid < 2 * GCHUNK) Gs[tid] = rg;
+        if (!BONUS && tid < 2 * GCHUNK) Gs[tid] = rg;
         __syncthreads();
         if (c0 + GCHUNK < n) fetch(c0 + GCHUNK);
+        if constexpr (BONUS) {
+            const float * ub = io.bonus + (int64_t) hk * N;
+            for (int tt = tid >> 5; tt < nc; tt += NT / 32) {
+                float s = 0.f;
+                for (int nn = tid & 31; nn < N; nn += 32) s = fmaf(Qs[tt * N + nn] * ub[nn], Ks[tt * N + nn], s);
+                s = wsum(s);
+                if ((tid & 31) == 0) Gs[tt] = s;
+            }
+            __syncthreads();
+        }
         for (int tt = 0; tt < nc; tt++) {
             const float xv = Vs[tt * GCOLS + pl];
             float kk[NREG], qq[NREG];
@@ -444,12 +468,23 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
 #pragma unroll
                 for (int j = 0; j < NREG; j++) S[j] = fmaf(kk[j], u, g * S[j]);
                 out = fmaf(u, kq, g * sq);
+            } else if constexpr (BONUS) {
+                float ww[NREG];
+                row_regs(Ws + tt * N, ww);
+                float acc = 0.f;
+#pragma unroll
+                for (int j = 0; j < NREG; j++) {
+                    acc = fmaf(S[j], qq[j], acc);                                      // the state before this token; q is zero beyond the key size
+                    S[j] = fmaf(ww[j], S[j], kk[j] * xv);
+                }
+#pragma unroll
+                for (int o = 1; o < LN; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+                out = fmaf(Gs[tt], xv, acc);
             } else {
                 float acc = 0.f;
 #pragma unroll
                 for (int j = 0; j < NREG; j++) {
-                    if constexpr (CHAN) S[j] = fmaf(kk[j], S[j], (1.f - kk[j]) * xv);   // key tied to the decay
-                    else S[j] = fmaf(Gs[tt], S[j], kk[j] * xv);
+                    S[j] = fmaf(kk[j], S[j], (1.f - kk[j]) * xv);                      // key tied to the decay
                     acc = fmaf(S[j], qq[j], acc);                                      // q is zero beyond the key size
                 }
 #pragma unroll
@@ -516,7 +551,14 @@ __global__ void __launch_bounds__(256) k_gated_linattn_smem(GatedLinIO io, const
             __syncthreads();
         }
         float acc = 0.f;
-        for (int nn = q4; nn < N; nn += 4) {
+        if (p.bonus) {
+            const float * ub = io.bonus + (int64_t) hk * N;
+            for (int nn = q4; nn < N; nn += 4) {
+                const float s = S[nn * GSCOLS + cc], kv = ks[nn] * u;
+                acc = fmaf(fmaf(ub[nn], kv, s), qs[nn], acc);
+                S[nn * GSCOLS + cc] = fmaf(fs[nn], s, kv);
+            }
+        } else for (int nn = q4; nn < N; nn += 4) {
             const float s = p.delta ? fmaf(ks[nn], u, S[nn * GSCOLS + cc]) : fmaf(fs[nn], S[nn * GSCOLS + cc], ks[nn] * u);
             S[nn * GSCOLS + cc] = s;
             acc = fmaf(s, qs[nn], acc);
@@ -668,18 +710,24 @@ int launch_hgrn2_prep(float * q, int64_t ldq, float * f, int64_t ldf, const floa
 int launch_gated_linattn(const GatedLinIO & io, const BatchView & b, const GatedLinParams & p, float * state, int64_t slot_stride, float * y, cudaStream_t st) {
     if (b.n_tokens <= 0) return 0;
     if (p.heads <= 0 || p.qk_heads <= 0 || p.heads % p.qk_heads || p.dim <= 0 || p.vdim <= 0 || !state || !io.q || !io.v || !io.decay || (p.delta && !io.beta) ||
-        (p.tied_key && (!p.decay_per_channel || p.delta)) || (!p.tied_key && !io.k) || (p.decay_per_channel && !p.tied_key))
+        (p.tied_key && (!p.decay_per_channel || p.delta)) || (!p.tied_key && !io.k) || (p.decay_per_channel && !p.tied_key && !p.bonus) ||
+        (p.bonus && (!p.decay_per_channel || p.delta || p.tied_key || !io.bonus)))
         return (int) cudaErrorInvalidValue;
-    // the two register kernels: delta rule with one decay per head, tied key with a decay per channel
-    if (p.dim <= 256 && ((p.delta && !p.decay_per_channel) || (p.tied_key && !p.delta))) {
+    // the register kernels: delta rule with one decay per head, tied key with a decay per channel, bonus form with a decay per channel
+    if (p.dim <= 256 && ((p.delta && !p.decay_per_channel) || (p.tied_key && !p.delta) || p.bonus)) {
         const int ln = p.dim <= 32 ? 8 : p.dim <= 64 ? 16 : 32;
         const int nreg = (p.dim + ln - 1) / ln;
-        const size_t smem = ((size_t) 2 * GCHUNK * p.dim + GCHUNK * GCOLS + 2 * GCHUNK) * sizeof(float);
+        const size_t smem = ((size_t) (p.bonus ? 3 : 2) * GCHUNK * p.dim + GCHUNK * GCOLS + 2 * GCHUNK) * sizeof(float);
         const dim3 grid((unsigned) (p.heads * ((p.vdim + GCOLS - 1) / GCOLS)), (unsigned) b.n_entries);
 #define PB_GL(NR, LNV)                                                                                                                               \
     do {                                                                                                                                             \
-        if (p.delta) return ck_launch([&] { k_gated_linattn_reg<NR, LNV, true, false><<<grid, GCOLS * LNV, smem, st>>>(io, b.slot, b.off, p, state, slot_stride, y); }); \
-        return ck_launch([&] { k_gated_linattn_reg<NR, LNV, false, true><<<grid, GCOLS * LNV, smem, st>>>(io, b.slot, b.off, p, state, slot_stride, y); });            \
+        if (p.bonus) {                                                                                                                               \
+            const int rc = raise_smem(k_gated_linattn_reg<NR, LNV, GL_BONUS>, smem);                                                                 \
+            if (rc) return rc;                                                                                                                       \
+            return ck_launch([&] { k_gated_linattn_reg<NR, LNV, GL_BONUS><<<grid, GCOLS * LNV, smem, st>>>(io, b.slot, b.off, p, state, slot_stride, y); });            \
+        }                                                                                                                                            \
+        if (p.delta) return ck_launch([&] { k_gated_linattn_reg<NR, LNV, GL_DELTA><<<grid, GCOLS * LNV, smem, st>>>(io, b.slot, b.off, p, state, slot_stride, y); }); \
+        return ck_launch([&] { k_gated_linattn_reg<NR, LNV, GL_TIED><<<grid, GCOLS * LNV, smem, st>>>(io, b.slot, b.off, p, state, slot_stride, y); });            \
     } while (0)
 #define PB_GL_LN(LNV)                 \
     do {                              \

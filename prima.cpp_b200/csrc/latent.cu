@@ -14,7 +14,12 @@
 namespace pb {
 namespace {
 
-// rotates the pair (u, v) = (x[i], x[i + half]) by the angle pos * freq[i]; cos and sin carry the factor mag
+// entries of pair i
+__device__ __forceinline__ void pair_at(const LatentParams & p, int i, int & ia, int & ib) {
+    if (p.rot_layout == ROT_INTERLEAVED) { ia = 2 * i; ib = 2 * i + 1; }
+    else { ia = i; ib = i + p.rot_dims / 2; }
+}
+// rotates the pair (u, v) by the angle pos * freq; cos and sin carry the factor mag
 __device__ __forceinline__ void turn(float u, float v, int pos, float f, float mag, float & ou, float & ov) {
     const float ang = (float) pos * f;
     const float c = cosf(ang) * mag, s = sinf(ang) * mag;
@@ -22,56 +27,74 @@ __device__ __forceinline__ void turn(float u, float v, int pos, float f, float m
     ov = v * c + u * s;
 }
 
+// turns the rotated part of every query head of one token
+__device__ __forceinline__ void rope_q_row(float * __restrict__ row, int pos, const LatentParams & p, const float * __restrict__ freq) {
+    const int half = p.rot_dims / 2, DQ = p.dim + p.rot_dim;
+    for (int i = threadIdx.x; i < p.heads * half; i += blockDim.x) {
+        const int h = i / half, j = i - h * half;
+        float * r = row + h * DQ + p.dim;
+        int ia, ib;
+        pair_at(p, j, ia, ib);
+        float a, b;
+        turn(r[ia], r[ib], pos, freq[j], p.rot_mag, a, b);
+        r[ia] = a;
+        r[ib] = b;
+    }
+}
+
 template <typename OT>
-__global__ void __launch_bounds__(256) k_latent_prep(const float * __restrict__ proj, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
+__global__ void __launch_bounds__(256) k_latent_prep(float * __restrict__ proj, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
                                                      const int32_t * __restrict__ pos0, const int32_t * __restrict__ entry_of, LatentParams p,
                                                      const float * __restrict__ wq, const float * __restrict__ wkv, const float * __restrict__ freq, float eps,
-                                                     OT * __restrict__ cq, float * __restrict__ cache, int64_t slot_stride) {
+                                                     OT * __restrict__ cq, float * __restrict__ cache, int64_t slot_stride, OT * __restrict__ lat,
+                                                     float * __restrict__ kr, int turn_q) {
     __shared__ float red[33];
     const int t = blockIdx.x;
     const int e = entry_of[t];
     const int pos = pos0[e] + (t - off[e]);
     const int C = latent_proj_cols(p), Rq = p.q_rank, R = p.kv_rank, Dr = p.rot_dim;
-    const float * row = proj + (int64_t) t * C;
-    float s = 0.f;
-    for (int i = threadIdx.x; i < Rq; i += blockDim.x) s = fmaf(row[i], row[i], s);
-    const float invq = 1.f / sqrtf(block_sum(s, red) / (float) Rq + eps);
-    for (int i = threadIdx.x; i < Rq; i += blockDim.x) put(cq, (int64_t) t * Rq + i, row[i] * invq * wq[i]);
+    float * row = proj + (int64_t) t * C;
+    if (Rq > 0) {
+        float s = 0.f;
+        for (int i = threadIdx.x; i < Rq; i += blockDim.x) s = fmaf(row[i], row[i], s);
+        const float invq = 1.f / sqrtf(block_sum(s, red) / (float) Rq + eps);
+        for (int i = threadIdx.x; i < Rq; i += blockDim.x) put(cq, (int64_t) t * Rq + i, row[i] * invq * wq[i]);
+    } else if (turn_q) {
+        rope_q_row(row, pos, p, freq);
+    }
     if (!p.own_kv) return;
-    const float * kv = row + Rq + p.heads * p.vdim;
-    s = 0.f;
+    const float * kv = row + latent_kv_col(p);
+    float s = 0.f;
     for (int i = threadIdx.x; i < R; i += blockDim.x) s = fmaf(kv[i], kv[i], s);
     const float invk = 1.f / sqrtf(block_sum(s, red) / (float) R + eps);
     float * crow = cache + (int64_t) slot[e] * slot_stride + (int64_t) pos * (R + Dr);
-    for (int i = threadIdx.x; i < R; i += blockDim.x) crow[i] = kv[i] * invk * wkv[i];
+    for (int i = threadIdx.x; i < R; i += blockDim.x) {
+        const float v = kv[i] * invk * wkv[i];
+        crow[i] = v;
+        if (lat) put(lat, (int64_t) t * R + i, v);
+    }
     const int half = p.rot_dims / 2;
     for (int i = threadIdx.x; i < Dr; i += blockDim.x) {
         if (i < half) {
+            int ia, ib;
+            pair_at(p, i, ia, ib);
             float a, b;
-            turn(kv[R + i], kv[R + i + half], pos, freq[i], p.rot_mag, a, b);
-            crow[R + i] = a;
-            crow[R + i + half] = b;
+            turn(kv[R + ia], kv[R + ib], pos, freq[i], p.rot_mag, a, b);
+            crow[R + ia] = a;
+            crow[R + ib] = b;
+            if (kr) { kr[(int64_t) t * Dr + ia] = a; kr[(int64_t) t * Dr + ib] = b; }
         } else if (i >= 2 * half) {
             crow[R + i] = kv[R + i];
+            if (kr) kr[(int64_t) t * Dr + i] = kv[R + i];
         }
     }
 }
 
-__global__ void k_latent_rope_q(float * __restrict__ q, const int32_t * __restrict__ off, const int32_t * __restrict__ pos0,
+__global__ void k_latent_rope_q(float * __restrict__ q, int64_t ldq, const int32_t * __restrict__ off, const int32_t * __restrict__ pos0,
                                 const int32_t * __restrict__ entry_of, LatentParams p, const float * __restrict__ freq) {
     const int t = blockIdx.x;
     const int e = entry_of[t];
-    const int pos = pos0[e] + (t - off[e]);
-    const int half = p.rot_dims / 2, DQ = p.dim + p.rot_dim;
-    float * row = q + (int64_t) t * p.heads * DQ;
-    for (int i = threadIdx.x; i < p.heads * half; i += blockDim.x) {
-        const int h = i / half, j = i - h * half;
-        float * r = row + h * DQ + p.dim;
-        float a, b;
-        turn(r[j], r[j + half], pos, freq[j], p.rot_mag, a, b);
-        r[j] = a;
-        r[j + half] = b;
-    }
+    rope_q_row(q + (int64_t) t * ldq, pos0[e] + (t - off[e]), p, freq);
 }
 
 template <typename OT>
@@ -90,13 +113,13 @@ __global__ void k_latent_gather(const float * __restrict__ cache, int64_t slot_s
 // CTA (head, token, 128 latent entries): qa[r] = sum_d W_uk[h * dim + d][r] q[d]; thread r walks a column of the head's block (coalesced
 // over r, eight loads in flight)
 template <typename WT>
-__global__ void __launch_bounds__(128) k_latent_absorb_q(const float * __restrict__ q, const int32_t * __restrict__ off, const int32_t * __restrict__ pos0,
+__global__ void __launch_bounds__(128) k_latent_absorb_q(const float * __restrict__ q, int64_t ldq, const int32_t * __restrict__ off, const int32_t * __restrict__ pos0,
                                                          const int32_t * __restrict__ entry_of, const WT * __restrict__ wuk, LatentParams p,
                                                          const float * __restrict__ freq, float * __restrict__ qa) {
     extern __shared__ float qs[];   // [dim]
     const int h = blockIdx.x, t = blockIdx.y;
     const int D = p.dim, Dr = p.rot_dim, R = p.kv_rank;
-    const float * qr = q + ((int64_t) t * p.heads + h) * (D + Dr);
+    const float * qr = q + (int64_t) t * ldq + (int64_t) h * (D + Dr);
     for (int d = threadIdx.x; d < D; d += blockDim.x) qs[d] = qr[d];
     __syncthreads();
     float * out = qa + ((int64_t) t * p.heads + h) * (R + Dr);
@@ -119,10 +142,12 @@ __global__ void __launch_bounds__(128) k_latent_absorb_q(const float * __restric
         const int e = entry_of[t], pos = pos0[e] + (t - off[e]), half = p.rot_dims / 2;
         for (int i = threadIdx.x; i < Dr; i += blockDim.x) {
             if (i < half) {
+                int ia, ib;
+                pair_at(p, i, ia, ib);
                 float a, b;
-                turn(qr[D + i], qr[D + i + half], pos, freq[i], p.rot_mag, a, b);
-                out[R + i] = a;
-                out[R + i + half] = b;
+                turn(qr[D + ia], qr[D + ib], pos, freq[i], p.rot_mag, a, b);
+                out[R + ia] = a;
+                out[R + ib] = b;
             } else if (i >= 2 * half) {
                 out[R + i] = qr[D + i];
             }
@@ -143,7 +168,7 @@ __global__ void __launch_bounds__(256) k_latent_up_v(const float * __restrict__ 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int dv = warp; dv < DV; dv += (int) (blockDim.x >> 5)) {
         const float acc = wsum(dot_lane8(wuv + ((int64_t) h * DV + dv) * R, os, R, lane));
-        if (lane == 0) put(out, (int64_t) t * p.heads * DV + h * DV + dv, acc * sigmoid_f(gate[(int64_t) t * ldg + h * DV + dv]));
+        if (lane == 0) put(out, (int64_t) t * p.heads * DV + h * DV + dv, gate ? acc * sigmoid_f(gate[(int64_t) t * ldg + h * DV + dv]) : acc);
     }
 }
 
@@ -262,7 +287,8 @@ __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __res
 // weighs splits lane and lane + 32.
 template <typename WT, typename OT>
 __global__ void __launch_bounds__(256) k_latent_merge_up_v(const float * __restrict__ part, int splits, const int32_t * __restrict__ off, const WT * __restrict__ wuv,
-                                                           LatentParams p, const float * __restrict__ gate, int64_t ldg, OT * __restrict__ out) {
+                                                           LatentParams p, const float * __restrict__ sink, const float * __restrict__ gate, int64_t ldg,
+                                                           OT * __restrict__ out) {
     extern __shared__ float os[];   // [kv_rank], then [64] weights of the splits
     const int h = blockIdx.x, e = blockIdx.y, t = off[e];
     const int R = p.kv_rank, DV = p.vdim, H = p.heads;
@@ -276,7 +302,8 @@ __global__ void __launch_bounds__(256) k_latent_merge_up_v(const float * __restr
         const float l0 = ok0 ? pe[lane * stride + R + 1] : 0.f, l1 = ok1 ? pe[(lane + 32) * stride + R + 1] : 0.f;
         const float M = wmax(fmaxf(m0, m1));
         const float f0 = m0 == -INFINITY ? 0.f : expf(m0 - M), f1 = m1 == -INFINITY ? 0.f : expf(m1 - M);
-        const float L = wsum(l0 * f0 + l1 * f1);
+        float L = wsum(l0 * f0 + l1 * f1);
+        if (sink && M != -INFINITY) L += expf(sink[h] - M);   // one more key in the denominator that has no value
         w[lane] = L > 0.f ? f0 / L : 0.f;
         w[lane + 32] = L > 0.f ? f1 / L : 0.f;
     }
@@ -298,32 +325,34 @@ __global__ void __launch_bounds__(256) k_latent_merge_up_v(const float * __restr
     const int dv_lo = blockIdx.z * ((DV + 1) / 2), dv_hi = min(DV, dv_lo + (DV + 1) / 2);
     for (int dv = dv_lo + warp; dv < dv_hi; dv += (int) (blockDim.x >> 5)) {
         const float acc = wsum(dot_lane8(wuv + ((int64_t) h * DV + dv) * R, os, R, lane));
-        if (lane == 0) put(out, (int64_t) t * H * DV + h * DV + dv, acc * sigmoid_f(gate[(int64_t) t * ldg + h * DV + dv]));
+        if (lane == 0) put(out, (int64_t) t * H * DV + h * DV + dv, gate ? acc * sigmoid_f(gate[(int64_t) t * ldg + h * DV + dv]) : acc);
     }
 }
 
 }  // namespace
 
 static bool latent_ok(const LatentParams & p) {
-    return p.heads > 0 && p.dim > 0 && p.rot_dim >= 0 && p.vdim > 0 && p.kv_rank > 0 && p.q_rank > 0 && p.rot_dims >= 0 && p.rot_dims <= p.rot_dim &&
+    return p.heads > 0 && p.dim > 0 && p.rot_dim >= 0 && p.vdim > 0 && p.kv_rank > 0 && p.q_rank >= 0 && p.rot_dims >= 0 && p.rot_dims <= p.rot_dim &&
            p.rot_dims % 2 == 0;
 }
 
-int launch_latent_prep(const float * proj, const BatchView & b, const LatentParams & p, const float * wq, const float * wkv, const float * freq, float eps,
-                       void * cq, int otype, float * cache, int64_t slot_stride, cudaStream_t st) {
+int launch_latent_prep(float * proj, const BatchView & b, const LatentParams & p, const float * wq, const float * wkv, const float * freq, float eps,
+                       void * cq, int otype, float * cache, int64_t slot_stride, void * lat, float * kr, int turn_q, cudaStream_t st) {
     if (b.n_tokens <= 0) return 0;
-    if (!latent_ok(p) || (p.own_kv && (!cache || !wkv))) return (int) cudaErrorInvalidValue;
+    if (!latent_ok(p) || (p.own_kv && (!cache || !wkv)) || (p.q_rank > 0 && (!wq || !cq)) || (p.rot_dims > 0 && !freq)) return (int) cudaErrorInvalidValue;
     return ck_launch([&] {
         if (otype == T_BF16)
             k_latent_prep<__nv_bfloat16><<<b.n_tokens, 256, 0, st>>>(proj, b.slot, b.off, b.pos0, b.entry_of, p, wq, wkv, freq, eps, (__nv_bfloat16 *) cq, cache,
-                                                                     slot_stride);
-        else k_latent_prep<float><<<b.n_tokens, 256, 0, st>>>(proj, b.slot, b.off, b.pos0, b.entry_of, p, wq, wkv, freq, eps, (float *) cq, cache, slot_stride);
+                                                                     slot_stride, (__nv_bfloat16 *) lat, kr, turn_q);
+        else
+            k_latent_prep<float><<<b.n_tokens, 256, 0, st>>>(proj, b.slot, b.off, b.pos0, b.entry_of, p, wq, wkv, freq, eps, (float *) cq, cache, slot_stride,
+                                                             (float *) lat, kr, turn_q);
     });
 }
-int launch_latent_rope_q(float * q, const BatchView & b, const LatentParams & p, const float * freq, cudaStream_t st) {
+int launch_latent_rope_q(float * q, int64_t ldq, const BatchView & b, const LatentParams & p, const float * freq, cudaStream_t st) {
     if (b.n_tokens <= 0 || p.rot_dims < 2) return 0;
     if (!latent_ok(p)) return (int) cudaErrorInvalidValue;
-    return ck_launch([&] { k_latent_rope_q<<<b.n_tokens, 128, 0, st>>>(q, b.off, b.pos0, b.entry_of, p, freq); });
+    return ck_launch([&] { k_latent_rope_q<<<b.n_tokens, 128, 0, st>>>(q, ldq, b.off, b.pos0, b.entry_of, p, freq); });
 }
 int launch_latent_gather(const float * cache, int64_t slot_stride, const BatchView & b, const LatentParams & p, void * lat, int otype, float * kr,
                          cudaStream_t st) {
@@ -334,7 +363,7 @@ int launch_latent_gather(const float * cache, int64_t slot_stride, const BatchVi
         else k_latent_gather<float><<<b.n_tokens, 128, 0, st>>>(cache, slot_stride, b.slot, b.off, b.pos0, b.entry_of, p, (float *) lat, kr);
     });
 }
-int launch_latent_absorb_q(const float * q, const BatchView & b, const void * wuk, int wtype, const LatentParams & p, const float * freq, float * qa,
+int launch_latent_absorb_q(const float * q, int64_t ldq, const BatchView & b, const void * wuk, int wtype, const LatentParams & p, const float * freq, float * qa,
                            cudaStream_t st) {
     const int n_tokens = b.n_tokens;
     if (n_tokens <= 0) return 0;
@@ -342,8 +371,8 @@ int launch_latent_absorb_q(const float * q, const BatchView & b, const void * wu
     const dim3 grid((unsigned) p.heads, (unsigned) n_tokens, (unsigned) ((p.kv_rank + 127) / 128));
     const size_t smem = (size_t) p.dim * sizeof(float);
     return ck_launch([&] {
-        if (wtype == T_BF16) k_latent_absorb_q<__nv_bfloat16><<<grid, 128, smem, st>>>(q, b.off, b.pos0, b.entry_of, (const __nv_bfloat16 *) wuk, p, freq, qa);
-        else k_latent_absorb_q<float><<<grid, 128, smem, st>>>(q, b.off, b.pos0, b.entry_of, (const float *) wuk, p, freq, qa);
+        if (wtype == T_BF16) k_latent_absorb_q<__nv_bfloat16><<<grid, 128, smem, st>>>(q, ldq, b.off, b.pos0, b.entry_of, (const __nv_bfloat16 *) wuk, p, freq, qa);
+        else k_latent_absorb_q<float><<<grid, 128, smem, st>>>(q, ldq, b.off, b.pos0, b.entry_of, (const float *) wuk, p, freq, qa);
     });
 }
 int launch_latent_up_v(const float * olat, const void * wuv, int wtype, const LatentParams & p, const float * gate, int64_t ldg, void * out, int otype,
@@ -364,7 +393,7 @@ int launch_latent_up_v(const float * olat, const void * wuv, int wtype, const La
 }
 
 int launch_latent_decode(const float * qa, const BatchView & b, const LatentParams & p, const float * cache, int64_t slot_stride, int splits, float * part,
-                         const void * wuv, int wtype, const float * gate, int64_t ldg, void * out, int otype, cudaStream_t st) {
+                         const void * wuv, int wtype, const float * sink, const float * gate, int64_t ldg, void * out, int otype, cudaStream_t st) {
     if (b.n_entries <= 0) return 0;
     if (!latent_ok(p) || p.kv_rank > 512 || splits < 1 || splits > 64 || !part || b.n_tokens != b.n_entries) return (int) cudaErrorInvalidValue;
     const int RW = latent_row(p);
@@ -378,11 +407,11 @@ int launch_latent_decode(const float * qa, const BatchView & b, const LatentPara
     const size_t smem2 = ((size_t) p.kv_rank + 64) * sizeof(float);
     return ck_launch([&] {
         if (wtype == T_BF16) {
-            if (otype == T_BF16) k_latent_merge_up_v<__nv_bfloat16, __nv_bfloat16><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const __nv_bfloat16 *) wuv, p, gate, ldg, (__nv_bfloat16 *) out);
-            else k_latent_merge_up_v<__nv_bfloat16, float><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const __nv_bfloat16 *) wuv, p, gate, ldg, (float *) out);
+            if (otype == T_BF16) k_latent_merge_up_v<__nv_bfloat16, __nv_bfloat16><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const __nv_bfloat16 *) wuv, p, sink, gate, ldg, (__nv_bfloat16 *) out);
+            else k_latent_merge_up_v<__nv_bfloat16, float><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const __nv_bfloat16 *) wuv, p, sink, gate, ldg, (float *) out);
         } else {
-            if (otype == T_BF16) k_latent_merge_up_v<float, __nv_bfloat16><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const float *) wuv, p, gate, ldg, (__nv_bfloat16 *) out);
-            else k_latent_merge_up_v<float, float><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const float *) wuv, p, gate, ldg, (float *) out);
+            if (otype == T_BF16) k_latent_merge_up_v<float, __nv_bfloat16><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const float *) wuv, p, sink, gate, ldg, (__nv_bfloat16 *) out);
+            else k_latent_merge_up_v<float, float><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const float *) wuv, p, sink, gate, ldg, (float *) out);
         }
     });
 }

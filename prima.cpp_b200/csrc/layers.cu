@@ -1,11 +1,12 @@
 // prima.cpp_b200/csrc/layers.cu — the engine of the layer-list family (arch.h): a configuration file lists the layers, every layer has
 // a sequence mixer (windowed attention with kept first tokens, a Mamba-2 state-space mixer, linear attention with a fixed decay per
-// head, softmax attention over a low-rank latent, or a dual mixer: an attention branch beside a gated linear recurrence) and an optional
-// feed-forward (tanh-GELU gated; clamped gated, dense or a routed mixture of experts), inside one of these layer frames: norms before and after every sublayer (FRAME_SANDWICH), or a grouped RMS norm
+// head, softmax attention over a low-rank latent, a WKV mixer, or a dual mixer: an attention branch beside a gated linear recurrence) and an
+// optional feed-forward (tanh-GELU gated; squared ReLU; xIELU; clamped gated, dense or a routed mixture of experts), inside one of these layer frames: norms before and after every sublayer (FRAME_SANDWICH), or a grouped RMS norm
 // before it with token shift and a depth average of all layer results (FRAME_PRENORM), or a layer norm with weight and bias on the
 // sublayer's result only, scaled by one factor, with a learned position table on the embedding (FRAME_POSTNORM), or an RMS norm with one
 // learned number before every sublayer, sublayer results times one factor, and a repeated block whose passes add the embedding output and
-// a step vector (FRAME_PRERMS).  Weights are dense f32 / bf16 matrices.  It lives behind the same model object and C ABI as the k-quant transformer engine
+// a step vector (FRAME_PRERMS; a norm may also have a weight per entry, and
+// the embedding may be normed).  A layer may borrow another layer's weights; its cache and state stay its own.  Weights are dense f32 / bf16 matrices.  It lives behind the same model object and C ABI as the k-quant transformer engine
 // (engine.cu): pb200_model_set_tensor / _synth / _finalize / _free, sequence slots, device arg-max — and steps through the ragged
 // batch step (pb200_batch_step) that the scheduler drives; the single-sequence entry points of the k-quant family answer PB200_ENOTSUP.
 //
@@ -14,7 +15,8 @@
 // in a ring as long as the window), Mamba-2 -> the last taps-1 convolution inputs and the fp32 state [heads][state][vdim], decay
 // attention -> the fp32 state [heads][dim][vdim], latent attention -> one row [latent | rotated key part] per position (a layer that
 // reads another layer's latent has none of its own), token shift -> the normed input of the last token, dual mixer -> K and V rows, the
-// last taps-1 convolution inputs of both branches and the recurrence's fp32 state.  A slot's arena is zeroed when it is handed out, so a
+// last taps-1 convolution inputs of both branches and the recurrence's fp32 state, chunked attention -> K and V rows of one chunk, WKV -> the
+// fp32 state [heads][dim][dim] and the normed input of the last token.  A slot's arena is zeroed when it is handed out, so a
 // reused slot starts like a new one; the token before a sequence's next one (bigram embedding) is kept per slot on the host.
 //
 // Precision: the residual stream, norms, attention scores / weights, recurrent state and everything that feeds the recurrence are
@@ -50,8 +52,8 @@ extern std::atomic<uint64_t> g_launches;
 
 namespace pb {
 
-enum : int { MIX_ATTENTION = 0, MIX_MAMBA2 = 1, MIX_DECAY = 2, MIX_LATENT = 3, MIX_DUAL = 4 };
-enum : int { FF_GELU = 0, FF_CLAMPED = 1, FF_MOE = 2, FF_RELU2 = 3 };   // FF_MOE: the expert form is MoeParams::act
+enum : int { MIX_ATTENTION = 0, MIX_MAMBA2 = 1, MIX_DECAY = 2, MIX_LATENT = 3, MIX_DUAL = 4, MIX_WKV = 5 };
+enum : int { FF_GELU = 0, FF_CLAMPED = 1, FF_MOE = 2, FF_RELU2 = 3, FF_XIELU = 4 };   // FF_MOE: the expert form is MoeParams::act
 enum : int { FRAME_SANDWICH = 0, FRAME_PRENORM = 1, FRAME_POSTNORM = 2, FRAME_PRERMS = 3 };
 enum : int { ROUTE_SOFTMAX_TOP = 0, ROUTE_SIGMOID_GROUPS = 1, ROUTE_SIGMOID_PLAIN = 2 };
 enum : int { REC_DELTA = 0, REC_HGRN2 = 1 };                 // recurrent branch of a dual mixer
@@ -105,8 +107,9 @@ struct LLayer {
     // latent attention (lproj: fused dq | gate | dkv)
     LatentParams lat;
     int kv_from = -1;                  // >= 0: the layer whose latent cache this one reads
-    DenseW lproj, uq, uk, uv;
-    VecF dq_norm, dkv_norm, rot_freq;
+    DenseW lproj, uq, ukv;             // ukv: key up-projection [heads * dim], then value up-projection [heads * vdim] of the latent
+    VecF dq_norm, dkv_norm, rot_freq, sink;
+    bool has_sink = false;             // a learned score per head of one more key without a value
     // mixture of experts: e_gateup [experts][2 ff][width], e_down [experts][width][ff]; a shared expert beside them (shared_ff > 0)
     MoeParams moe;
     DenseW e_gateup, e_down, s_gateup, s_down;
@@ -120,12 +123,22 @@ struct LLayer {
     // attention: RMS norm of every query / key head with a weight [dim] all heads share
     bool qk_norm = false;
     VecF q_norm, k_norm;
+    // attention whose inputs are prepared by launch_attn_prep_store: norm over the whole q / k projection, rotation, a factor per query head
+    bool att_prep = false;
+    int att_qkn = QKN_NONE, att_rot_dims = 0, att_rot_layout = ROT_INTERLEAVED;
+    VecF temp;
     // mixture of experts: form of the router; the shared expert's per-token gate vector [width] (ROUTE_SIGMOID_GROUPS)
     int route = ROUTE_SOFTMAX_TOP;
     VecF shared_gate;
     // dual mixer (qkvg: the fused projection of both branches; out: the output product over [left | right], or the left one; out_r: the right one)
     DualMix dual;
     DenseW out_r;
+    // WKV mixer: token mix with five blends (r, k, v, g, w), qkvg = one matrix of the four projections, decay from a low-rank map (fp32)
+    GatedLinParams wkv;
+    int decay_rank = 0;                // inner size of the decay's map: the configuration's, or what the first of its tensors to arrive has
+    VecF mix_mu, w1, w2, w0, bonus;
+    VecF ff_act;                       // FF_XIELU: its two numbers
+    int weights_of = -1;               // >= 0: no tensors of its own, runs with that layer's
     VecF dconv_w, vrot_freq, f_bias, f_lower, join_wl, join_wr;   // rot_freq, q_norm, k_norm, A_log, dt_bias, onorm are shared with the other mixers
 };
 
@@ -146,6 +159,10 @@ struct TensorPlace {
     // ... or (vrows > 0) a tensor [vrows][vcols] (n = vrows * vcols) placed at element v0 + r * vld + c, `repeat` copies vrep elements apart:
     // a block of a vector several tensors fill, a short convolution right-aligned in longer taps, a weight all heads share, one number for all
     int64_t v0 = 0, vrows = 0, vcols = 0, vld = 0, repeat = 1, vrep = 0;
+    float add = 0.f;          // added to every element of a vector (weights stored around zero)
+    // a size that only the tensor's shape tells: while *size is 0, the tensor's element count divided by size_unit settles it
+    int * size = nullptr;
+    int64_t size_unit = 0;
 };
 
 struct LayerList {
@@ -170,6 +187,8 @@ struct LayerList {
     float resid_mult = 1.f;   // factor on every normed sublayer result (FRAME_PRERMS: on every sublayer result)
     // FRAME_PRERMS: embedding factor, hashed bigram table [buckets + 1][width] (buckets == 0: none), the token before each slot's next one
     float embed_scale = 1.f;
+    bool embed_normed = false;   // the stream starts as the normed embedding (embed_norm) instead
+    VecF embed_norm;
     BigramParams bigram;
     DenseW bigram_table;
     std::vector<int32_t> seq_prev;
@@ -537,8 +556,8 @@ static bool mumizen_resolve(LayerList & ll, const std::string & name, TensorPlac
         if (w == "mix.dq.norm") return vec(L.dq_norm, a.q_rank);
         if (w == "mix.dkv.norm") return a.own_kv && vec(L.dkv_norm, a.kv_rank);
         if (w == "mix.uq") return mat(L.uq, 0, (int64_t) a.heads * (a.dim + a.rot_dim), a.q_rank, 0);
-        if (w == "mix.uk") return mat(L.uk, 0, (int64_t) a.heads * a.dim, a.kv_rank, 0);
-        if (w == "mix.uv") return mat(L.uv, 0, VD, a.kv_rank, 0);
+        if (w == "mix.uk") return mat(L.ukv, 0, (int64_t) a.heads * a.dim, a.kv_rank, 0);
+        if (w == "mix.uv") return mat(L.ukv, (int64_t) a.heads * a.dim, VD, a.kv_rank, 1);
         if (w == "mix.o") return mat(L.out, 0, W, VD, 0);
     }
     return false;
@@ -950,6 +969,182 @@ static bool zevedra_resolve(LayerList & ll, const std::string & name, TensorPlac
     return false;
 }
 
+// ---------------------------------------------------------------------------------------------------------------
+// Ruvuvik: configuration keys and tensor names.  The stream starts as the normed embedding; every layer is x <- x + mixer(norm x),
+// x <- x + ff(norm x) with an RMS norm whose weight is stored around zero; a layer may borrow another layer's tensors ("weights_of").  Mixers:
+// "attention" inside chunks of positions (RMS norm over the whole q / k projection, interleaved partial rotation, a temperature per head,
+// soft-capped scores, a gate per head), "latent_attention" (queries straight from the input, interleaved rotation of the shared key part, a
+// learned sink per head, no gate) and "wkv" (token mix, decay per channel from a low-rank map, bonus for the current token).  Feed-forward: xIELU.
+static int ruvuvik_rotation(const Json & mx, int head_dims, int & dims, VecF & freq, std::string & err) {
+    double base = 10000.0;
+    dims = 0;
+    const Json * rot = mx.get("rot");
+    if (rot && rot->kind == Json::OBJ) {
+        base = rot->number("base", 10000.0);
+        dims = (int) rot->integer("dims", head_dims);
+        if (dims < 0 || dims > head_dims || dims % 2 || !(base > 0.0)) { err = "rotated dimensions"; return PB200_EINVAL; }
+    }
+    plain_rotary_table(base, dims, freq.preset);
+    return 0;
+}
+static int ruvuvik_configure(const Json & cfg, LayerList & ll, std::string & err) {
+    ll.frame = FRAME_PRERMS;
+    ll.embed_normed = true;
+    ll.width = (int) cfg.integer("width", 0);
+    ll.vocab = (int) cfg.integer("vocab", 0);
+    ll.logit_scale = 1.f;
+    ll.resid_mult = 1.f;
+    if (const Json * nrm = cfg.get("norm")) ll.eps = (float) nrm->number("eps", 1e-6);
+    const Json * layers = cfg.get("layers");
+    if (ll.width <= 0 || ll.vocab <= 0 || !layers || layers->kind != Json::ARR || layers->arr.empty()) { err = "width, vocab and layers are required"; return PB200_EINVAL; }
+    const int nl = (int) layers->arr.size();
+    for (const Json & jl : layers->arr) {
+        LLayer L;
+        const Json * from = jl.get("weights_of");
+        if (from && from->kind == Json::NUM) {
+            L.weights_of = (int) from->num;
+            if (L.weights_of < 0 || L.weights_of >= nl || L.weights_of == (int) ll.layers.size()) { err = "weights_of must name another layer"; return PB200_EINVAL; }
+            ll.layers.push_back(std::move(L));   // everything else is the named layer's
+            continue;
+        }
+        const std::string type = jl.string("type");
+        const Json * mx = jl.get("mixer");
+        if (!mx || mx->kind != Json::OBJ) { err = "layer without mixer"; return PB200_EINVAL; }
+        if (type == "attention") {
+            L.kind = MIX_ATTENTION;
+            AttnParams & a = L.att;
+            a.heads = (int) mx->integer("heads", 0);
+            a.kv_heads = (int) mx->integer("kv_heads", a.heads);
+            a.dim = (int) mx->integer("dim", 0);
+            a.vdim = (int) mx->integer("vdim", a.dim);
+            a.scale = (float) mx->number("scale", a.dim > 0 ? 1.0 / std::sqrt((double) a.dim) : 1.0);
+            a.softcap = (float) mx->number("softcap", 0.0);
+            a.gated = 1;
+            if (const Json * mk = mx->get("mask"))
+                if (mk->kind == Json::OBJ) a.chunk = (int) std::min<long long>(std::max<long long>(mk->integer("size", 0), 0), 1 << 30);
+            L.att_prep = true;
+            L.att_qkn = QKN_WHOLE_WEIGHT;
+            L.att_rot_layout = ROT_INTERLEAVED;
+            if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dim <= 0 || a.vdim <= 0 || a.vdim > 512) { err = "attention sizes"; return PB200_EINVAL; }
+            const int rc = ruvuvik_rotation(*mx, a.dim, L.att_rot_dims, L.rot_freq, err);
+            if (rc) return rc;
+        } else if (type == "latent_attention") {
+            L.kind = MIX_LATENT;
+            LatentParams & a = L.lat;
+            a.heads = (int) mx->integer("heads", 0);
+            a.dim = (int) mx->integer("dim", 0);
+            a.rot_dim = (int) mx->integer("rot_dim", 0);
+            a.vdim = (int) mx->integer("vdim", a.dim);
+            a.kv_rank = (int) mx->integer("kv_rank", 0);
+            a.q_rank = 0;
+            a.gated = 0;
+            a.own_kv = 1;
+            a.rot_layout = ROT_INTERLEAVED;
+            a.scale = (float) mx->number("scale", a.dim + a.rot_dim > 0 ? 1.0 / std::sqrt((double) (a.dim + a.rot_dim)) : 1.0);
+            L.has_sink = true;
+            if (a.heads <= 0 || a.dim <= 0 || a.rot_dim < 0 || a.vdim <= 0 || a.kv_rank <= 0 || a.kv_rank > 512 || a.vdim > 512) { err = "latent attention sizes"; return PB200_EINVAL; }
+            const int rc = ruvuvik_rotation(*mx, a.rot_dim, a.rot_dims, L.rot_freq, err);
+            if (rc) return rc;
+        } else if (type == "wkv") {
+            L.kind = MIX_WKV;
+            GatedLinParams & p = L.wkv;
+            p.heads = p.qk_heads = (int) mx->integer("heads", 0);
+            p.dim = p.vdim = (int) mx->integer("dim", 0);
+            p.decay_per_channel = 1;
+            p.bonus = 1;
+            L.decay_rank = (int) mx->integer("decay_rank", 0);   // 0: the tensors tell
+            L.mix_mu.n_parts = 5;
+            if (p.heads <= 0 || p.dim <= 0 || p.dim > 512 || L.decay_rank < 0) { err = "wkv sizes"; return PB200_EINVAL; }
+        } else {
+            err = "unknown layer type '" + type + "'";
+            return PB200_ENOTSUP;
+        }
+        const Json * mlp = jl.get("mlp");
+        if (mlp && mlp->kind == Json::OBJ) {
+            const std::string kind = mlp->string("kind", "dense");
+            if (kind != "dense") { err = "unknown feed-forward kind '" + kind + "'"; return PB200_ENOTSUP; }
+            L.ff_kind = FF_XIELU;
+            L.ff = (int) mlp->integer("ff", 0);
+            if (L.ff <= 0) { err = "feed-forward size"; return PB200_EINVAL; }
+        }
+        ll.layers.push_back(std::move(L));
+    }
+    // every layer is one run of the layer whose tensors it uses
+    for (int i = 0; i < nl; i++) {
+        int j = i, hops = 0;
+        while (ll.layers[(size_t) j].weights_of >= 0 && hops++ <= nl) j = ll.layers[(size_t) j].weights_of;
+        if (ll.layers[(size_t) j].weights_of >= 0) { err = "weights_of goes round in a circle"; return PB200_EINVAL; }
+        LRun r;
+        r.layer = j;
+        ll.runs.push_back(r);
+    }
+    return 0;
+}
+
+static bool ruvuvik_resolve(LayerList & ll, const std::string & name, TensorPlace & o) {
+    const int64_t W = ll.width;
+    auto mat = [&](DenseW & m, int64_t row0, int64_t rows, int64_t cols, int part) { o.mat = &m; o.row0 = row0; o.rows = rows; o.cols = cols; o.part = part; return true; };
+    auto vec = [&](VecF & v, int64_t n) { o.vec = &v; o.n = n; return true; };
+    auto norm = [&](VecF & v, int64_t n) { o.add = 1.f; return vec(v, n); };   // stored around zero: the factor is 1 + w
+    if (name == "embed") return mat(ll.embed, 0, ll.vocab, W, 0);
+    if (name == "embed.norm") return norm(ll.embed_norm, W);
+    if (name == "head") return mat(ll.head, 0, ll.vocab, W, 0);
+    if (name == "final.norm") return norm(ll.final_norm, W);
+    int il = -1, used = 0;
+    if (sscanf(name.c_str(), "l%d.%n", &il, &used) != 1 || used <= 0 || il < 0 || il >= (int) ll.layers.size()) return false;
+    LLayer & L = ll.layers[(size_t) il];
+    if (L.weights_of >= 0) return false;
+    const std::string w = name.substr((size_t) used);
+    if (w == "norm1") return norm(L.norm1, W);
+    if (L.ff > 0) {
+        if (w == "norm2") return norm(L.norm2, W);
+        if (w == "mlp.up") return mat(L.gateup, 0, L.ff, W, 0);
+        if (w == "mlp.down") return mat(L.down, 0, W, L.ff, 0);
+        if (w == "mlp.act") return vec(L.ff_act, 2);
+    }
+    if (L.kind == MIX_ATTENTION) {
+        const AttnParams & a = L.att;
+        const int64_t QD = (int64_t) a.heads * a.dim, KD = (int64_t) a.kv_heads * a.dim, VD = (int64_t) a.kv_heads * a.vdim;
+        if (w == "mix.q") return mat(L.qkvg, 0, QD, W, 0);
+        if (w == "mix.k") return mat(L.qkvg, QD, KD, W, 1);
+        if (w == "mix.v") return mat(L.qkvg, QD + KD, VD, W, 2);
+        if (w == "mix.g") return mat(L.qkvg, QD + KD + VD, a.heads, W, 3);
+        if (w == "mix.q.norm") return vec(L.q_norm, QD);
+        if (w == "mix.k.norm") return vec(L.k_norm, KD);
+        if (w == "mix.temp") return vec(L.temp, a.heads);
+        if (w == "mix.o") return mat(L.out, 0, W, (int64_t) a.heads * a.vdim, 0);
+    } else if (L.kind == MIX_LATENT) {
+        const LatentParams & a = L.lat;
+        const int64_t VD = (int64_t) a.heads * a.vdim;
+        if (w == "mix.q") return mat(L.lproj, 0, latent_q_cols(a), W, 0);
+        if (w == "mix.dkv") return mat(L.lproj, latent_kv_col(a), a.kv_rank + a.rot_dim, W, 1);
+        if (w == "mix.dkv.norm") return vec(L.dkv_norm, a.kv_rank);
+        if (w == "mix.uk") return mat(L.ukv, 0, (int64_t) a.heads * a.dim, a.kv_rank, 0);
+        if (w == "mix.uv") return mat(L.ukv, (int64_t) a.heads * a.dim, VD, a.kv_rank, 1);
+        if (w == "mix.sink") return vec(L.sink, a.heads);
+        if (w == "mix.o") return mat(L.out, 0, W, VD, 0);
+    } else if (L.kind == MIX_WKV) {
+        const int64_t HD = (int64_t) L.wkv.heads * L.wkv.dim;
+        static const char * const proj[4] = {"mix.r", "mix.k", "mix.v", "mix.g"};
+        static const char * const mu[5] = {"mix.mu.r", "mix.mu.k", "mix.mu.v", "mix.mu.g", "mix.mu.w"};
+        for (int i = 0; i < 4; i++)
+            if (w == proj[i]) return mat(L.qkvg, i * HD, HD, W, i);
+        for (int i = 0; i < 5; i++)
+            if (w == mu[i]) { o.part = i; o.v0 = i * W; o.vrows = 1; o.vcols = o.vld = W; return vec(L.mix_mu, W); }
+        if (w == "mix.w1" || w == "mix.w2") {
+            const bool down = w == "mix.w1";
+            o.size = &L.decay_rank;
+            o.size_unit = down ? W : HD;
+            return vec(down ? L.w1 : L.w2, o.size_unit * L.decay_rank);
+        }
+        if (w == "mix.w0") return vec(L.w0, HD);
+        if (w == "mix.u") return vec(L.bonus, HD);
+        if (w == "mix.norm") return vec(L.onorm, HD);
+        if (w == "mix.o") return mat(L.out, 0, W, HD, 0);
+    }
+    return false;
+}
+
 static const ArchEntry g_archs[] = {
     {"llama", ARCH_KQUANT, 0, nullptr, nullptr},
     {"qwen2", ARCH_KQUANT, 2, nullptr, nullptr},
@@ -957,6 +1152,7 @@ static const ArchEntry g_archs[] = {
     {"Mumizen", ARCH_LAYERS, 0, mumizen_configure, mumizen_resolve},
     {"Sapudra", ARCH_LAYERS, 0, sapudra_configure, sapudra_resolve},
     {"Zevedra", ARCH_LAYERS, 0, zevedra_configure, zevedra_resolve},
+    {"Ruvuvik", ARCH_LAYERS, 0, ruvuvik_configure, ruvuvik_resolve},
 };
 int arch_count() { return (int) (sizeof(g_archs) / sizeof(g_archs[0])); }
 const ArchEntry * arch_at(int i) { return (i >= 0 && i < arch_count()) ? &g_archs[i] : nullptr; }
@@ -978,6 +1174,7 @@ static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
     fm(ll.head, (int64_t) ll.vocab, W, 1);
     fv(ll.final_norm, W, 0);
     if (ll.frame == FRAME_POSTNORM) { fm(ll.pos_table, (int64_t) ll.max_pos, W, 1); fv(ll.final_norm_bias, W, 1); }
+    if (ll.embed_normed) fv(ll.embed_norm, W, 0);
     if (ll.frame == FRAME_PRERMS && ll.bigram.buckets > 0) fm(ll.bigram_table, ll.bigram.buckets + 1, W, 1);
     if (ll.loop_times > 0) {
         if (ll.frame != FRAME_PRERMS) fm(ll.loop_in, W, 2 * W, 1);
@@ -985,6 +1182,7 @@ static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
     }
     int il = 0;
     for (LLayer & L : ll.layers) {
+        if (L.weights_of >= 0) { il++; continue; }   // another layer's parameters
         fv(L.norm1, W, 0);
         if (ll.frame == FRAME_SANDWICH) fv(L.norm1b, W, 0);
         else if (ll.frame == FRAME_POSTNORM) fv(L.norm1_bias, W, 1);
@@ -993,7 +1191,19 @@ static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
         if (L.kind == MIX_ATTENTION) {
             fm(L.qkvg, attn_qkvg_cols(L.att), W, L.att.gated ? 4 : 3);
             if (L.qk_norm) { fv(L.q_norm, L.att.dim, 0); fv(L.k_norm, L.att.dim, 0); }
+            if (L.att_prep) {
+                if (L.att_qkn == QKN_WHOLE_WEIGHT) { fv(L.q_norm, (int64_t) L.att.heads * L.att.dim, 0); fv(L.k_norm, (int64_t) L.att.kv_heads * L.att.dim, 0); }
+                fv(L.rot_freq, (int64_t) L.rot_freq.preset.size(), 0);
+                fv(L.temp, L.att.heads, 0);
+            }
             fm(L.out, W, (int64_t) L.att.heads * L.att.vdim, 1);
+        } else if (L.kind == MIX_WKV) {
+            const int64_t HD = (int64_t) L.wkv.heads * L.wkv.dim;
+            fm(L.qkvg, 4 * HD, W, 4);
+            fv(L.mix_mu, 5 * W, 5);
+            fv(L.w1, (int64_t) L.decay_rank * W, 7); fv(L.w2, HD * L.decay_rank, 7); fv(L.w0, HD, 3);
+            fv(L.bonus, HD, 1); fv(L.onorm, HD, 0);
+            fm(L.out, W, HD, 1);
         } else if (L.kind == MIX_MAMBA2) {
             const Mamba2Params & p = L.ssm;
             fm(L.in, mamba2_in_cols(p), W, 1);
@@ -1026,13 +1236,13 @@ static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
             }
         } else {
             const LatentParams & a = L.lat;
-            fm(L.lproj, latent_proj_cols(a), W, a.own_kv ? 3 : 2);
-            fv(L.dq_norm, a.q_rank, 0);
+            fm(L.lproj, latent_proj_cols(a), W, 1 + (a.gated ? 1 : 0) + (a.own_kv ? 1 : 0));
+            if (a.q_rank > 0) fv(L.dq_norm, a.q_rank, 0);
             if (a.own_kv) fv(L.dkv_norm, a.kv_rank, 0);
             fv(L.rot_freq, (int64_t) L.rot_freq.preset.size(), 0);
-            fm(L.uq, (int64_t) a.heads * (a.dim + a.rot_dim), a.q_rank, 1);
-            fm(L.uk, (int64_t) a.heads * a.dim, a.kv_rank, 1);
-            fm(L.uv, (int64_t) a.heads * a.vdim, a.kv_rank, 1);
+            if (a.q_rank > 0) fm(L.uq, (int64_t) a.heads * (a.dim + a.rot_dim), a.q_rank, 1);
+            fm(L.ukv, (int64_t) a.heads * (a.dim + a.vdim), a.kv_rank, 2);
+            if (L.has_sink) fv(L.sink, a.heads, 1);
             fm(L.out, W, (int64_t) a.heads * a.vdim, 1);
         }
         if (L.ff > 0) {
@@ -1049,9 +1259,10 @@ static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
                     fm(L.s_gateup, gated * (int64_t) L.shared_ff, W, gated); fm(L.s_down, W, L.shared_ff, 1);
                     if (L.route == ROUTE_SIGMOID_GROUPS) fv(L.shared_gate, W, 7);
                 }
-            } else if (L.ff_kind == FF_RELU2) {
+            } else if (L.ff_kind == FF_RELU2 || L.ff_kind == FF_XIELU) {
                 fm(L.gateup, (int64_t) L.ff, W, 1);
                 fm(L.down, W, L.ff, 1);
+                if (L.ff_kind == FF_XIELU) fv(L.ff_act, 2, 1);
             } else {
                 fm(L.gateup, 2 * (int64_t) L.ff, W, 2);
                 fm(L.down, W, L.ff, 1);
@@ -1060,21 +1271,22 @@ static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
     }
 }
 
+// allocates every parameter that has a size and no memory yet (a size that only a tensor's shape tells is 0 until that tensor arrives)
 static int ll_alloc_params(pb200_model * m) {
     LayerList & ll = *m->ll;
     int rc = 0;
-    int64_t bytes = 0;
+    int64_t bytes = ll.weight_bytes;
     for_each_param(
         ll,
         [&](DenseW & d, int64_t N, int64_t K, int parts) {
-            if (rc) return;
+            if (rc || d.data) return;
             d.N = N; d.K = K; d.filled.assign((size_t) parts, 0);
             const size_t b = (size_t) N * K * esize(ll.ctype);
             rc = m->alloc(&d.data, b + 16);
             bytes += (int64_t) b;
         },
         [&](VecF & v, int64_t n, int) {
-            if (rc) return;
+            if (rc || v.data || n <= 0) return;
             v.n = n; v.filled = false;
             v.parts.assign((size_t) std::max(v.n_parts, 0), 0);
             rc = m->alloc((void **) &v.data, (size_t) n * 4);
@@ -1114,9 +1326,17 @@ int ll_set_tensor(pb200_model * m, const char * name, int type, const void * hos
     if (type != T_F32 && type != T_BF16) return PB200_ENOTSUP;
     TensorPlace pl;
     if (!ll.arch->resolve(ll, name, pl)) return PB200_EINVAL;
+    cudaSetDevice(m->device);
+    if (pl.size && *pl.size == 0) {   // this tensor settles a size: then there is memory to allocate, and a place of that size
+        const int64_t have = (int64_t) (nbytes / esize(type));
+        if (pl.size_unit <= 0 || have <= 0 || have % pl.size_unit || have / pl.size_unit > (1 << 20)) return PB200_EINVAL;
+        *pl.size = (int) (have / pl.size_unit);
+        CK(ll_alloc_params(m));
+        pl = TensorPlace();
+        if (!ll.arch->resolve(ll, name, pl)) return PB200_EINVAL;
+    }
     const int64_t count = pl.mat ? pl.rows * pl.cols : pl.n;
     if (nbytes != (size_t) count * esize(type)) return PB200_EINVAL;
-    cudaSetDevice(m->device);
     const int dtype = pl.mat ? ll.ctype : T_F32;
     std::vector<uint8_t> conv;
     const void * src = host;
@@ -1124,6 +1344,14 @@ int ll_set_tensor(pb200_model * m, const char * name, int type, const void * hos
         conv.resize((size_t) count * esize(dtype));
         if (dtype == T_F32) bf16_to_f32((const uint16_t *) host, (float *) conv.data(), (size_t) count);
         else f32_to_bf16((const float *) host, (uint16_t *) conv.data(), (size_t) count);
+        src = conv.data();
+    }
+    if (pl.vec && pl.add != 0.f) {
+        std::vector<float> sum((size_t) count);
+        memcpy(sum.data(), src, (size_t) count * 4);
+        for (float & v : sum) v += pl.add;
+        conv.resize((size_t) count * 4);
+        memcpy(conv.data(), sum.data(), (size_t) count * 4);
         src = conv.data();
     }
     if (pl.mat) {
@@ -1173,6 +1401,9 @@ int ll_synth(pb200_model * m, uint64_t seed) {
     cudaSetDevice(m->device);
     uint64_t sd = seed * 0x100000001B3ull + 17;
     int rc = 0;
+    for (LLayer & L : ll.layers)
+        if (L.kind == MIX_WKV && L.decay_rank == 0) L.decay_rank = std::max(8, ll.width / 64);   // no tensor will tell
+    CK(ll_alloc_params(m));
     for_each_param(
         ll,
         [&](DenseW & d, int64_t N, int64_t K, int) {
@@ -1206,7 +1437,8 @@ int ll_finalize(pb200_model * m) {
     for_each_param(
         ll, [&](DenseW & d, int64_t, int64_t, int) { for (uint8_t f : d.filled) complete = complete && f; },
         [&](VecF & v, int64_t, int) {
-            if (v.parts.empty()) complete = complete && v.filled;
+            if (!v.data) complete = false;   // a size that no tensor has settled
+            else if (v.parts.empty()) complete = complete && v.filled;
             else for (uint8_t f : v.parts) complete = complete && f;
         });
     if (!complete) return PB200_ESTATE;
@@ -1225,7 +1457,7 @@ int ll_finalize(pb200_model * m) {
             if (L.lat.own_kv) off += (int64_t) ll.n_ctx * latent_row(L.lat);
             else r.state_off = ll.runs[(size_t) L.kv_from].state_off;   // FRAME_PRENORM: run i is layer i
         } else if (L.kind == MIX_ATTENTION || L.kind == MIX_DUAL) {
-            L.att.cache_rows = attn_cache_rows(L.att.window, L.att.keep_first, ll.n_ctx);
+            L.att.cache_rows = L.att.chunk > 0 ? std::min(L.att.chunk, ll.n_ctx) : attn_cache_rows(L.att.window, L.att.keep_first, ll.n_ctx);
             if (L.att.cache_rows >= ll.n_ctx) ll.ctx_limited = true;
             off += (int64_t) L.att.cache_rows * L.att.kv_heads * (L.att.dim + L.att.vdim);
             if (L.kind == MIX_DUAL) {   // then the convolution's last inputs and the recurrence's state
@@ -1235,6 +1467,11 @@ int ll_finalize(pb200_model * m) {
                 off = (off + 3) / 4 * 4;
                 off += (int64_t) d.rp.heads * d.rp.dim * d.rp.vdim;
             }
+        } else if (L.kind == MIX_WKV) {
+            off += (int64_t) L.wkv.heads * L.wkv.dim * L.wkv.vdim;
+            off = (off + 3) / 4 * 4;
+            r.shift_off = off;
+            off += ll.width;
         } else {
             off += (int64_t) (L.ssm.conv - 1) * mamba2_conv_channels(L.ssm) + (int64_t) L.ssm.heads * L.ssm.state * L.ssm.vdim;
         }
@@ -1324,7 +1561,16 @@ static int ll_reserve(pb200_model * m, int T, int nW, int nE) {
         int64_t maxact = ll.width, maxact2 = ll.width, maxbig = ll.width, maxch = 1, maxinner = 1, maxb2 = 0, maxb3 = 0, maxb4 = 0, maxkr = 0;
         int64_t moe_top = 0, moe_topff = 0, moe_e = 0;
         for (const LLayer & L : ll.layers) {
-            if (L.kind == MIX_ATTENTION) {
+            if (L.weights_of >= 0) continue;
+            if (L.kind == MIX_WKV) {
+                const int64_t HD = (int64_t) L.wkv.heads * L.wkv.dim;
+                maxact = std::max(maxact, std::max<int64_t>(4 * (int64_t) ll.width, HD));   // four operand planes of the token mix
+                maxbig = std::max(maxbig, 4 * HD);
+                maxch = std::max<int64_t>(maxch, ll.width);                                // the fifth one, fp32
+                maxinner = std::max(maxinner, HD);
+                maxb2 = std::max<int64_t>(maxb2, L.decay_rank);
+                maxb3 = std::max(maxb3, HD);                                               // decays
+            } else if (L.kind == MIX_ATTENTION) {
                 maxact = std::max<int64_t>(maxact, (int64_t) L.att.heads * L.att.vdim);
                 maxbig = std::max<int64_t>(maxbig, attn_qkvg_cols(L.att));
             } else if (L.kind == MIX_MAMBA2) {
@@ -1354,8 +1600,8 @@ static int ll_reserve(pb200_model * m, int T, int nW, int nE) {
                 maxact2 = std::max<int64_t>(maxact2, std::max(a.q_rank, a.kv_rank));
                 maxbig = std::max<int64_t>(maxbig, latent_proj_cols(a));
                 maxb2 = std::max(maxb2, H * (a.dim + a.rot_dim));
-                maxb3 = std::max(maxb3, std::max(H * a.dim, H * latent_row(a)));
-                maxb4 = std::max(maxb4, std::max(H * a.vdim, H * a.kv_rank));
+                maxb3 = std::max(maxb3, std::max(H * (a.dim + a.vdim), H * latent_row(a)));
+                maxb4 = std::max(maxb4, H * a.kv_rank);
                 maxkr = std::max<int64_t>(maxkr, a.rot_dim);
             }
             if (L.ff_kind == FF_MOE && L.ff > 0) {
@@ -1408,7 +1654,8 @@ static int ll_reserve(pb200_model * m, int T, int nW, int nE) {
     }
     size_t need_part = 0;
     for (const LLayer & L : ll.layers)
-        if (L.kind == MIX_LATENT)
+        if (L.weights_of >= 0) continue;
+        else if (L.kind == MIX_LATENT)
             need_part = std::max(need_part, (size_t) nE * (size_t) latent_decode_splits(ll.n_ctx) * (size_t) L.lat.heads * (size_t) (L.lat.kv_rank + 2));
         else if (L.kind == MIX_ATTENTION || L.kind == MIX_DUAL)
             need_part = std::max(need_part, attn_decode_part_floats(L.att, nE));
@@ -1484,7 +1731,14 @@ static int mix_attention(pb200_model * m, const BatchView & b, bool prefill, con
     CK(launch_dense(ct, ll.act, W, L.qkvg.data, W, ll.big, C, T, C, W, nullptr, nullptr, 0, 1.f, st));
     float * kc = sbase, * vc = sbase + (int64_t) a.cache_rows * a.kv_heads * a.dim;
     CAT(CAT_ATTN);
-    if (L.qk_norm) CK(launch_attn_qknorm_kv_store(ll.big, b, a, L.q_norm.data, L.k_norm.data, ll.eps, kc, vc, ll.slot_floats, st));
+    if (L.att_prep) {   // norm over the whole projections, rotation, temperatures and the cache store in one launch
+        AttnPrep pr;
+        pr.norm = L.att_qkn; pr.wq = L.q_norm.data; pr.wk = L.k_norm.data; pr.eps = ll.eps;
+        pr.rot_dims = L.att_rot_dims; pr.rot_layout = L.att_rot_layout; pr.rot_freq = L.rot_freq.data;
+        pr.q_scale = L.temp.data;
+        float * k = ll.big + a.heads * a.dim, * v = k + a.kv_heads * a.dim;
+        CK(launch_attn_prep_store(ll.big, C, k, C, v, C, b, a, pr, kc, vc, ll.slot_floats, st));
+    } else if (L.qk_norm) CK(launch_attn_qknorm_kv_store(ll.big, b, a, L.q_norm.data, L.k_norm.data, ll.eps, kc, vc, ll.slot_floats, st));
     else CK(launch_attn_kv_store(ll.big, b, a, kc, vc, ll.slot_floats, st));
     if (prefill) CK(launch_attn_window_prefill(ll.big, b, a, ll.act, ct, st));
     else CK(launch_attn_window_decode(ll.big, b, a, kc, vc, ll.slot_floats, ll.act, ct, st, ll.lat_part));
@@ -1530,49 +1784,90 @@ static int mix_latent(pb200_model * m, const BatchView & b, bool prefill, const 
     cudaStream_t st = m->stream;
     const int T = b.n_tokens, W = ll.width, ct = ll.ctype;
     const LatentParams & a = L.lat;
-    const int H = a.heads, C = latent_proj_cols(a), DQ = a.dim + a.rot_dim, VD = H * a.vdim, R = a.kv_rank, RW = latent_row(a);
+    const int H = a.heads, C = latent_proj_cols(a), DQ = a.dim + a.rot_dim, VD = H * a.vdim, R = a.kv_rank, RW = latent_row(a), KV = H * a.dim + VD;
     float * cache = ll.state + r.state_off;       // this layer's rows, or those of the layer it reads
-    const float * gate = ll.big + a.q_rank;
+    const float * gate = a.gated ? ll.big + latent_q_cols(a) : nullptr;
+    const float * sink = L.has_sink ? L.sink.data : nullptr;
+    const void * wuk = L.ukv.data, * wuv = (const uint8_t *) L.ukv.data + (size_t) H * a.dim * R * esize(ct);
+    const bool direct_q = a.q_rank <= 0;          // the fused projection ends in the queries themselves
+    float * q = direct_q ? ll.big : ll.big2;      // [T][heads][dim + rot_dim], rows ldq floats apart
+    const int64_t ldq = direct_q ? C : (int64_t) H * DQ;
     CAT(CAT_DENSE);
     CK(launch_dense(ct, ll.act, W, L.lproj.data, W, ll.big, C, T, C, W, nullptr, nullptr, 0, 1.f, st));
     CAT(CAT_LATENT);
-    CK(launch_latent_prep(ll.big, b, a, L.dq_norm.data, L.dkv_norm.data, L.rot_freq.data, ll.eps, ll.act2, ct, cache, ll.slot_floats, st));
-    CAT(CAT_DENSE);
-    CK(launch_dense(ct, ll.act2, a.q_rank, L.uq.data, a.q_rank, ll.big2, (int64_t) H * DQ, T, H * DQ, a.q_rank, nullptr, nullptr, 0, 1.f, st));
+    // a layer with a cache of its own and queries of its own: the batch's latents and key parts leave in the same launch that stores them
+    const bool fused = prefill && a.own_kv && direct_q;
+    CK(launch_latent_prep(ll.big, b, a, L.dq_norm.data, L.dkv_norm.data, L.rot_freq.data, ll.eps, ll.act2, ct, cache, ll.slot_floats, fused ? ll.act2 : nullptr,
+                          fused ? ll.krb : nullptr, prefill, st));
+    if (!direct_q) {
+        CAT(CAT_DENSE);
+        CK(launch_dense(ct, ll.act2, a.q_rank, L.uq.data, a.q_rank, ll.big2, (int64_t) H * DQ, T, H * DQ, a.q_rank, nullptr, nullptr, 0, 1.f, st));
+    }
     AttnParams ap;
     ap.heads = H; ap.scale = a.scale;
     AttnIO io;
     CAT(CAT_LATENT);
-    if (prefill) {   // keys and values of the batch, expanded from the cached latents
-        CK(launch_latent_rope_q(ll.big2, b, a, L.rot_freq.data, st));
-        CK(launch_latent_gather(cache, ll.slot_floats, b, a, ll.act2, ct, ll.krb, st));
+    if (prefill) {   // keys and values of the batch, expanded from the cached latents by one product
+        if (!direct_q) CK(launch_latent_rope_q(q, ldq, b, a, L.rot_freq.data, st));
+        if (!fused) CK(launch_latent_gather(cache, ll.slot_floats, b, a, ll.act2, ct, ll.krb, st));
         CAT(CAT_DENSE);
-        if (a.dim > 0) CK(launch_dense(ct, ll.act2, R, L.uk.data, R, ll.big3, (int64_t) H * a.dim, T, H * a.dim, R, nullptr, nullptr, 0, 1.f, st));
-        CK(launch_dense(ct, ll.act2, R, L.uv.data, R, ll.big4, VD, T, VD, R, nullptr, nullptr, 0, 1.f, st));
+        CK(launch_dense(ct, ll.act2, R, L.ukv.data, R, ll.big3, KV, T, KV, R, nullptr, nullptr, 0, 1.f, st));
         CAT(CAT_ATTN);
         ap.kv_heads = H; ap.dim = DQ; ap.vdim = a.vdim; ap.shared_dim = a.rot_dim;
-        io.q = ll.big2; io.ldq = (int64_t) H * DQ;
-        io.k = ll.big3; io.ldk = (int64_t) H * a.dim;
+        ap.sink = sink ? 1 : 0;
+        io.sink = sink;
+        io.q = q; io.ldq = ldq;
+        io.k = ll.big3; io.ldk = KV;
         io.ks = ll.krb; io.ldks = a.rot_dim;
-        io.v = ll.big4; io.ldv = VD;
-        io.gate = gate; io.ldg = C; io.gate_mode = 2;
+        io.v = ll.big3 + (int64_t) H * a.dim; io.ldv = KV;
+        io.gate = gate; io.ldg = C; io.gate_mode = gate ? 2 : 0;
         CK(launch_attn_prefill_io(io, b, ap, ll.act, ct, st));
     } else if (T == b.n_entries && R <= 512) {   // one token per entry: the key up-projection folded into the query, rows split over CTAs
-        CK(launch_latent_absorb_q(ll.big2, b, L.uk.data, ct, a, L.rot_freq.data, ll.big3, st));
+        CK(launch_latent_absorb_q(q, ldq, b, wuk, ct, a, L.rot_freq.data, ll.big3, st));
         CAT(CAT_ATTN);
-        CK(launch_latent_decode(ll.big3, b, a, cache, ll.slot_floats, latent_decode_splits(a.cache_rows), ll.lat_part, L.uv.data, ct, gate, C, ll.act, ct, st));
+        CK(launch_latent_decode(ll.big3, b, a, cache, ll.slot_floats, latent_decode_splits(a.cache_rows), ll.lat_part, wuv, ct, sink, gate, C, ll.act, ct, st));
     } else {         // the same through the shared decode kernel: one key / value head, the key is the whole row, the value its latent part
-        CK(launch_latent_absorb_q(ll.big2, b, L.uk.data, ct, a, L.rot_freq.data, ll.big3, st));
+        CK(launch_latent_absorb_q(q, ldq, b, wuk, ct, a, L.rot_freq.data, ll.big3, st));
         CAT(CAT_ATTN);
         ap.kv_heads = 1; ap.dim = RW; ap.vdim = R; ap.cache_rows = a.cache_rows;
+        ap.sink = sink ? 1 : 0;
+        io.sink = sink;
         io.q = ll.big3; io.ldq = (int64_t) H * RW;
         io.k_row = io.v_row = RW;
         CK(launch_attn_decode_io(io, b, ap, cache, cache, ll.slot_floats, ll.big4, T_F32, st));
         CAT(CAT_LATENT);
-        CK(launch_latent_up_v(ll.big4, L.uv.data, ct, a, gate, C, ll.act, ct, T, st));
+        CK(launch_latent_up_v(ll.big4, wuv, ct, a, gate, C, ll.act, ct, T, st));
     }
     CAT(CAT_DENSE);
     return launch_dense(ct, ll.act, VD, L.out.data, VD, out, W, T, W, VD, nullptr, resid, W, 1.f, st);
+}
+
+// ---- WKV mixer over the stream x (its norm and token mix are one launch): x[t] += W_o (heads normed one by one * weight * silu(gate)) ----
+static int mix_wkv(pb200_model * m, const BatchView & b, const LRun & r, LLayer & L, float * x) {
+    LayerList & ll = *m->ll;
+    cudaStream_t st = m->stream;
+    const int T = b.n_tokens, W = ll.width, ct = ll.ctype;
+    const GatedLinParams & p = L.wkv;
+    const int HD = p.heads * p.dim;
+    const int64_t plane = (int64_t) T * W, C = 4 * (int64_t) HD;
+    CAT(CAT_NORM);
+    CK(launch_rmsnorm_token_mix(x, b, L.norm1.data, ll.eps, L.mix_mu.data, 4, ll.state + r.shift_off, ll.slot_floats, ll.act, plane, ct, ll.xbc, W, st));
+    CAT(CAT_DENSE);
+    CK(launch_dense_planes(ct, ll.act, plane, W, L.qkvg.data, W, ll.big, C, 4, T, HD, W, st));   // r | k | v | gate
+    CAT(CAT_CONV);
+    CK(launch_lowrank_decay(ll.xbc, L.w1.data, L.w2.data, L.w0.data, T, W, L.decay_rank, HD, ll.big2, ll.big3, st));
+    CAT(CAT_SCAN);
+    GatedLinIO gi;
+    gi.q = ll.big; gi.ldq = C;
+    gi.k = ll.big + HD; gi.ldk = C;
+    gi.v = ll.big + 2 * HD; gi.ldv = C;
+    gi.decay = ll.big3; gi.ldd = HD;
+    gi.bonus = L.bonus.data;
+    CK(launch_gated_linattn(gi, b, p, ll.state + r.state_off, ll.slot_floats, ll.yssm, st));
+    CAT(CAT_NORM);
+    CK(launch_norm_gate(ll.yssm, ll.big + 3 * HD, C, p.heads, L.onorm.data, 1, ll.eps, ll.act, ct, T, HD, st));
+    CAT(CAT_DENSE);
+    return launch_dense(ct, ll.act, HD, L.out.data, HD, x, W, T, W, HD, nullptr, x, W, 1.f, st);
 }
 
 // ---- dual mixer over ll.act: x[t] += mult * join(attention branch, recurrent branch).  JOIN_SCALED_SUM: both branch results, scaled, lie
@@ -1726,6 +2021,18 @@ static int ff_relu2(pb200_model * m, int T, const DenseW & up, const DenseW & do
     CAT(CAT_DENSE);
     return launch_dense(ct, ll.act2, ff, down.data, ff, out, W, T, W, ff, nullptr, nullptr, 0, 1.f, st);
 }
+// ---- xIELU feed-forward: x[t] += down(xielu(up(ll.act[t]))) ----
+static int ff_xielu(pb200_model * m, int T, LLayer & L, float * x) {
+    LayerList & ll = *m->ll;
+    cudaStream_t st = m->stream;
+    const int W = ll.width, ct = ll.ctype, ff = L.ff;
+    CAT(CAT_DENSE);
+    CK(launch_dense(ct, ll.act, W, L.gateup.data, W, ll.big, ff, T, ff, W, nullptr, nullptr, 0, 1.f, st));
+    CAT(CAT_ELEM);
+    CK(launch_xielu(ll.big, L.ff_act.data, ll.act2, ct, (int64_t) T * ff, st));
+    CAT(CAT_DENSE);
+    return launch_dense(ct, ll.act2, ff, L.down.data, ff, x, W, T, W, ff, nullptr, x, W, 1.f, st);
+}
 // ---- mixture of experts over ll.act.  accumulate: x[t] += shared(h) + sum_k w_k expert_k(h) (the stream itself); otherwise x receives the
 // sublayer's result alone.  The router form and the expert form come from the layer (LLayer::route, MoeParams::act). ----
 static int ff_moe(pb200_model * m, int T, bool prefill, LLayer & L, float * x, bool accumulate, float out_scale = 1.f) {
@@ -1835,23 +2142,27 @@ static int ll_forward_postnorm(pb200_model * m, const BatchView & b, bool prefil
 
 // FRAME_PRERMS: the stream starts as embed * scale + bigram row; x <- x + mult * mixer(norm1 x), x <- x + mult * ff(norm2 x) with RMS norms of
 // one learned number (kept as a constant vector); every pass of the repeated block first adds the embedding output (not the first pass) and
-// its step vector.  ll.act holds the next sublayer's normed input in the operand type.
+// its step vector.  With embed_normed the stream starts as the normed embedding instead; norms may have a weight per entry (kept as factors).
+// ll.act holds the next sublayer's normed input in the operand type.
 static int ll_forward_prerms(pb200_model * m, const BatchView & b, bool prefill, const int32_t * tokens_dev, const int32_t * want_dev, int nW, int lrow0) {
     LayerList & ll = *m->ll;
     cudaStream_t st = m->stream;
     const int T = b.n_tokens, W = ll.width, ct = ll.ctype;
     CAT(CAT_ELEM);
-    CK(launch_embed_bigram(ll.embed.data, ll.bigram.buckets > 0 ? ll.bigram_table.data : nullptr, ct, W, ll.embed_scale, ll.bigram, tokens_dev, b, ll.x,
-                           ll.loop_times > 1 ? ll.x0 : nullptr, st));
     bool act_ready = false;   // the kernel that closed the previous sublayer has left this one's normed input in ll.act
+    if (ll.embed_normed) {
+        const LLayer & L0 = ll.layers[(size_t) ll.runs[0].layer];
+        act_ready = L0.kind != MIX_WKV;
+        CK(launch_embed_rmsnorm(ll.embed.data, ct, W, tokens_dev, T, ll.embed_norm.data, ll.eps, ll.x, L0.norm1.data, act_ready ? ll.act : nullptr, ct, st));
+    } else CK(launch_embed_bigram(ll.embed.data, ll.bigram.buckets > 0 ? ll.bigram_table.data : nullptr, ct, W, ll.embed_scale, ll.bigram, tokens_dev, b, ll.x,
+                           ll.loop_times > 1 ? ll.x0 : nullptr, st));
     for (size_t ir = 0; ir < ll.runs.size(); ir++) {
         const LRun & r = ll.runs[ir];
         LLayer & L = ll.layers[(size_t) r.layer];
-        if (L.kind != MIX_DUAL) return PB200_ENOTSUP;
         if (r.pass >= 0) {
             CAT(CAT_NORM);
             CK(launch_stream_add_rmsnorm(ll.x, r.pass > 0 ? ll.x0 : nullptr, ll.loop_step.data + (int64_t) r.pass * W, L.norm1.data, ll.eps, ll.act, ct, T, W, st));
-        } else if (!act_ready) {
+        } else if (!act_ready && L.kind != MIX_WKV) {   // a WKV mixer norms the stream itself, with the token mix
             CAT(CAT_NORM);
             CK(launch_group_rmsnorm(ll.x, nullptr, L.norm1.data, 1, ll.eps, ll.act, ct, T, W, st));
         }
@@ -1860,15 +2171,21 @@ static int ll_forward_prerms(pb200_model * m, const BatchView & b, bool prefill,
         const float * next_norm = nullptr;
         if (L.ff > 0) next_norm = L.norm2.data;
         else if (ir + 1 < ll.runs.size() && ll.runs[ir + 1].pass < 0) next_norm = ll.layers[(size_t) ll.runs[ir + 1].layer].norm1.data;
-        CK(mix_dual(m, b, prefill, r, L, ll.x, ll.resid_mult, next_norm));
-        const bool fused = L.dual.join == JOIN_NORMED_MEAN && next_norm;
+        if (L.kind == MIX_DUAL) CK(mix_dual(m, b, prefill, r, L, ll.x, ll.resid_mult, next_norm));
+        else if (ll.resid_mult != 1.f || r.pass >= 0) return PB200_ENOTSUP;
+        else if (L.kind == MIX_ATTENTION) CK(mix_attention(m, b, prefill, r, L, ll.x, ll.x));
+        else if (L.kind == MIX_LATENT) CK(mix_latent(m, b, prefill, r, L, ll.x, ll.x));
+        else if (L.kind == MIX_WKV) CK(mix_wkv(m, b, r, L, ll.x));
+        else return PB200_ENOTSUP;
+        const bool fused = L.kind == MIX_DUAL && L.dual.join == JOIN_NORMED_MEAN && next_norm;
         if (L.ff > 0) {
             if (!fused) {
                 CAT(CAT_NORM);
                 CK(launch_group_rmsnorm(ll.x, nullptr, L.norm2.data, 1, ll.eps, ll.act, ct, T, W, st));
             }
-            if (L.ff_kind != FF_MOE) return PB200_ENOTSUP;
-            CK(ff_moe(m, T, prefill, L, ll.x, true, ll.resid_mult));
+            if (L.ff_kind == FF_MOE) CK(ff_moe(m, T, prefill, L, ll.x, true, ll.resid_mult));
+            else if (L.ff_kind == FF_XIELU && ll.resid_mult == 1.f) CK(ff_xielu(m, T, L, ll.x));
+            else return PB200_ENOTSUP;
         } else {
             act_ready = fused;
         }
@@ -2168,7 +2485,7 @@ int ll_debug_read(pb200_model * m, const char * name, float * host, int64_t n) {
     LayerList & ll = *m->ll;
     cudaSetDevice(m->device);
     CK(cudaStreamSynchronize(m->stream));
-    if (strcmp(name, "profile") == 0) {   // ms of the last batch: dense, attention, convolution, scan, norms, element-wise, head, [7] = total,
+    if (strcmp(name, "profile") == 0) {   // ms of the last batch: dense, attention, convolution (or the map of a WKV mixer's decay), scan, norms, element-wise, head, [7] = total,
         if (n > 10) return PB200_EINVAL;   // [8] = routed experts, [9] = the small steps around latent attention (norm + rotation, gather, folds)
         memcpy(host, ll.prof_ms, (size_t) n * 4);
         return 0;

@@ -7,8 +7,10 @@
 // an RMS norm per query / key head, the squared-ReLU feed-forward, the router with sigmoid scores, a choice correction and expert groups,
 // and the tanh soft-cap of the logits; a hashed bigram embedding, a short causal convolution over any range of projection channels, the
 // preparation of attention inputs (RMS norm over a whole projection or per head, partial rotation in either pair layout, values rotated by
-// their position), a sink in the softmax denominator, gated linear recurrences with a decay per token (gated delta rule, HGRN2), experts
-// whose routing weight multiplies their input.  Every constant of a mechanism is a parameter, nothing is tied to one model.
+// their position), a sink in the softmax denominator, gated linear recurrences with a decay per token (gated delta rule, HGRN2, and the WKV form
+// that reads the state before the token's write with a bonus for the token itself), experts whose routing weight multiplies their input; attention
+// inside fixed chunks of positions, learned sinks and temperatures per head, latent attention with a direct query projection, a token mix with a
+// blend per input, a decay from a low-rank map of the token, the xIELU feed-forward.  Every constant of a mechanism is a parameter, nothing is tied to one model.
 // All launchers enqueue on `stream` and return a cudaError_t as int (0 = success).
 #pragma once
 #include <cuda_bf16.h>
@@ -42,12 +44,19 @@ int launch_dense(int type, const void * A, int64_t lda, const void * W, int64_t 
 // each) into the same rows of C, g < groups; start / count are device arrays and no group has more than max_rows rows.  Tensor-core
 // kernel only (bf16, aligned shapes): dense_grouped_ok says whether it applies; otherwise the caller multiplies group by group.
 int dense_grouped_ok(int type, int N, int K, int64_t lda, int64_t ldw, int64_t w_stride, const void * A, const void * W);
+// Several products of one shape over operands of their own, side by side: C[t][p * N + n] = sum_k A[p * a_plane + t * lda + k] * W[p * N + n][k],
+// p < planes (W: one [planes * N][K] matrix).
+int launch_dense_planes(int type, const void * A, int64_t a_plane, int64_t lda, const void * W, int64_t ldw, float * C, int64_t ldc, int planes, int T, int N,
+                        int K, cudaStream_t stream);
 int launch_dense_grouped(int type, const void * A, int64_t lda, const void * W, int64_t ldw, int64_t w_stride, float * C, int64_t ldc, const int32_t * start,
                          const int32_t * count, int groups, int max_rows, int N, int K, cudaStream_t stream);
 // 1: the tensor-core kernel takes this shape (bf16, aligned K / strides); informational (bench, tests)
 int dense_uses_tensor_cores(int type, int T, int N, int K, int64_t lda, int64_t ldw);
 
 // ---- element-wise / norms; `otype` (T_F32 | T_BF16) is the type of an activation that feeds a dense product ----
+// x[t] = rmsnorm(table[tokens[t]]) * w, then (y given) y[t] = rmsnorm(x[t]) * wn in the operand type: a normed embedding and the first layer's norm
+int launch_embed_rmsnorm(const void * table, int type, int width, const int32_t * tokens, int n_tokens, const float * w, float eps, float * x, const float * wn,
+                         void * y, int otype, cudaStream_t stream);
 int launch_embed(const void * table, int type, int width, const int32_t * tokens, int n_tokens, float * x, float * x_copy, cudaStream_t stream);
 // x[t] = table[tokens[t]] + pos_table[position of t] (fp32 sum; both tables in `type`); xa (if given) receives x in the operand type
 int launch_embed_pos(const void * table, const void * pos_table, int type, int width, const int32_t * tokens, const BatchView & b, float * x, void * xa,
@@ -71,6 +80,9 @@ int launch_layernorm_affine_residual(const float * m, const float * w, const flo
 // y[i] = max(u[i], 0)^2 -> operand type
 int launch_relu2(const float * u, void * y, int otype, int64_t n, cudaStream_t stream);
 // x[i] <- cap * tanh(x[i] / cap), in place
+// y[i] = xielu(u[i]) -> operand type, with the two numbers pq[0], pq[1] (device):  z > 0: softplus(p) z^2 + z / 2,
+// z <= 0: (1/2 + softplus(q)) (e^z - 1 - z) + z / 2
+int launch_xielu(const float * u, const float * pq, void * y, int otype, int64_t n, cudaStream_t stream);
 int launch_softcap(float * x, int64_t n, float cap, cudaStream_t stream);
 // x[t] += layernorm(m[t]) * w      (the post-norm of a sublayer and the residual sum, fp32)
 int launch_layernorm_residual(const float * m, const float * w, float eps, float * x, int n_rows, int width, cudaStream_t stream);
@@ -92,8 +104,15 @@ struct AttnParams {
     int cache_rows = 0;       // rows per slot: positions < keep_first at their own row, later ones in a ring over the rest
     int shared_dim = 0;       // prompt kernels: the last shared_dim of a key's dim entries come from one array all heads share
     int gated = 1;            // the fused projection ends with one gate logit per head (0: q | k | v only, the output is not gated)
-    int sink = 0;             // 1: one is added to the softmax denominator (a key of score 0 that has no value)
+    int sink = 0;             // 1: the softmax denominator has one more term, a key without a value: of score 0, or AttnIO::sink[head]
+    int chunk = 0;            // > 0: position i sees j <= i only inside its own chunk of positions, floor(i / chunk) = floor(j / chunk); the cache
+                              // is a ring of `chunk` rows then (window must be 0)
 };
+// lowest position that position i sees (apart from kept first tokens)
+__host__ __device__ inline int attn_first_visible(const AttnParams & a, int i) {
+    if (a.chunk > 0) return i - i % a.chunk;
+    return a.window > 0 && i >= a.window ? i - a.window + 1 : 0;
+}
 // Where the attention kernels read their inputs (fp32 rows, strides in floats).  Prompt kernels read keys and values of the batch:
 // k rows hold [kv_heads][dim - shared_dim], ks rows [shared_dim]; v rows [kv_heads][vdim].  Decode kernels read q and gate here and
 // the keys / values from the cache, whose rows are k_row / v_row floats apart (kv head h at + h * dim / + h * vdim).
@@ -105,6 +124,7 @@ struct AttnIO {
     const float * gate = nullptr; int64_t ldg = 0;     // gate logits; the output is multiplied by their sigmoid
     int gate_mode = 0;                                  // 0: no gate, 1: one logit per head, 2: one per output element [heads][vdim]
     int64_t k_row = 0, v_row = 0;
+    const float * sink = nullptr;                       // AttnParams::sink: the extra key's score per head (nullptr: 0)
 };
 __host__ __device__ inline int attn_qkvg_cols(const AttnParams & a) { return a.heads * a.dim + a.kv_heads * a.dim + a.kv_heads * a.vdim + (a.gated ? a.heads : 0); }
 // rows of a slot's cache so that every position a later token may still see is present, capped at n_ctx
@@ -196,36 +216,44 @@ int launch_norm_gate(const float * y, const float * gate, int64_t ldg, int group
 // ---- attention over a latent ----
 struct LatentParams {
     int heads = 0, dim = 0, rot_dim = 0, vdim = 0, kv_rank = 0, q_rank = 0;
-    int rot_dims = 0;         // leading entries of the rotated part that turn, in pairs (i, i + rot_dims / 2)
+    int rot_dims = 0;         // leading entries of the rotated part that turn, in pairs of rot_layout
+    int rot_layout = 1;       // ROT_HALVES (i, i + rot_dims / 2) or ROT_INTERLEAVED (2i, 2i + 1)
     float rot_mag = 1.f;      // factor on cos and sin
     float scale = 1.f;
     int cache_rows = 0;       // rows of kv_rank + rot_dim floats per slot: [normed latent | rotated shared key part] of every position
     int own_kv = 1;           // 0: the layer reads another layer's cache and has no down-projection of its own
+    int gated = 1;            // a gate logit per output element
 };
-__host__ __device__ inline int latent_proj_cols(const LatentParams & p) { return p.q_rank + p.heads * p.vdim + (p.own_kv ? p.kv_rank + p.rot_dim : 0); }
+// columns of the fused projection: the query latent (q_rank 0: the queries themselves, heads * (dim + rot_dim)), then the gate, then dkv
+__host__ __device__ inline int latent_q_cols(const LatentParams & p) { return p.q_rank > 0 ? p.q_rank : p.heads * (p.dim + p.rot_dim); }
+__host__ __device__ inline int latent_kv_col(const LatentParams & p) { return latent_q_cols(p) + (p.gated ? p.heads * p.vdim : 0); }
+__host__ __device__ inline int latent_proj_cols(const LatentParams & p) { return latent_kv_col(p) + (p.own_kv ? p.kv_rank + p.rot_dim : 0); }
 __host__ __device__ inline int latent_row(const LatentParams & p) { return p.kv_rank + p.rot_dim; }
-// proj: [T][dq | gate | dkv] f32 (one fused projection; dkv only with own_kv).  cq[t] = rmsnorm(dq) * wq -> operand type;
-// with own_kv: cache row of the token's position <- [rmsnorm(dkv[:kv_rank]) * wkv | rotate(dkv[kv_rank:], position)]
-int launch_latent_prep(const float * proj, const BatchView & b, const LatentParams & p, const float * wq, const float * wkv, const float * freq, float eps,
-                       void * cq, int otype, float * cache, int64_t slot_stride, cudaStream_t stream);
-// rotates the last rot_dim entries of every head of q [T][heads][dim + rot_dim] in place by the token's position
-int launch_latent_rope_q(float * q, const BatchView & b, const LatentParams & p, const float * freq, cudaStream_t stream);
+// proj: [T][dq or q | gate | dkv] f32 (one fused projection; gate only if gated, dkv only with own_kv).  q_rank > 0: cq[t] = rmsnorm(dq) * wq ->
+// operand type.  With own_kv: cache row of the token's position <- [rmsnorm(dkv[:kv_rank]) * wkv | rotate(dkv[kv_rank:], position)], and where
+// lat / kr are given the same two parts also go there (lat [T][kv_rank] operand type, kr [T][rot_dim] f32).  turn_q (q_rank 0): the last rot_dim
+// entries of every query head are rotated in place in the same launch.
+int launch_latent_prep(float * proj, const BatchView & b, const LatentParams & p, const float * wq, const float * wkv, const float * freq, float eps,
+                       void * cq, int otype, float * cache, int64_t slot_stride, void * lat, float * kr, int turn_q, cudaStream_t stream);
+// rotates the last rot_dim entries of every head of q (rows of ldq floats: [heads][dim + rot_dim]) in place by the token's position
+int launch_latent_rope_q(float * q, int64_t ldq, const BatchView & b, const LatentParams & p, const float * freq, cudaStream_t stream);
 // the batch's own cache rows: latent -> lat [T][kv_rank] (operand type), rotated key part -> kr [T][rot_dim] f32
 int launch_latent_gather(const float * cache, int64_t slot_stride, const BatchView & b, const LatentParams & p, void * lat, int otype, float * kr,
                          cudaStream_t stream);
 // decode: qa[t][h] = [ W_uk[h]^T q_unrotated[t][h]  (kv_rank) | rotate(q[t][h][dim:], position) (rot_dim) ]: the score against a cache row is
 // one dot product.  q comes straight from the projection (not rotated yet).
-int launch_latent_absorb_q(const float * q, const BatchView & b, const void * wuk, int wtype, const LatentParams & p, const float * freq, float * qa,
+int launch_latent_absorb_q(const float * q, int64_t ldq, const BatchView & b, const void * wuk, int wtype, const LatentParams & p, const float * freq, float * qa,
                            cudaStream_t stream);
-// decode: out[t][h][:] = (W_uv[h] olat[t][h]) * sigmoid(gate[t][h][:])   olat: [T][heads][kv_rank] (the weighted sum of latents)
+// decode: out[t][h][:] = (W_uv[h] olat[t][h]) * sigmoid(gate[t][h][:])   (gate may be null)   olat: [T][heads][kv_rank] (the weighted sum of latents)
 int launch_latent_up_v(const float * olat, const void * wuv, int wtype, const LatentParams & p, const float * gate, int64_t ldg, void * out, int otype,
                        int n_tokens, cudaStream_t stream);
 
 // decode attention of one-token entries over the slot's rows, split over `splits` CTAs per (entry, 16 heads), then the merge, the
-// value up-projection and the gate in a second kernel.  part: scratch of n_entries * splits * heads * (kv_rank + 2) floats.
+// value up-projection and the gate (may be null) in a second kernel.  sink (may be null): score per head of one more key in the denominator
+// that has no value.  part: scratch of n_entries * splits * heads * (kv_rank + 2) floats.
 inline int latent_decode_splits(int cache_rows) { return cache_rows >= 2048 ? 64 : cache_rows >= 64 ? cache_rows / 32 : 1; }
 int launch_latent_decode(const float * qa, const BatchView & b, const LatentParams & p, const float * cache, int64_t slot_stride, int splits, float * part,
-                         const void * wuv, int wtype, const float * gate, int64_t ldg, void * out, int otype, cudaStream_t stream);
+                         const void * wuv, int wtype, const float * sink, const float * gate, int64_t ldg, void * out, int otype, cudaStream_t stream);
 
 // ---- clamped gated feed-forward, dense or a mixture of experts ----
 // y[t][j] = g s(1.702 g) (u + 1),  g = min(gu[t][j], limit),  u = clamp(gu[t][ff + j], -limit, limit),  s = sigmoid     gu: [T][2 ff] f32
@@ -294,6 +322,7 @@ struct AttnPrep {
     int v_rot = 0;                // 1: every value head turns by its position over all vdim entries (pairs in v_layout, v_freq [vdim / 2]);
     int v_layout = ROT_INTERLEAVED;     // the cache holds the turned values and launch_attn_unrotate_gate turns a head's result back
     const float * v_freq = nullptr;
+    const float * q_scale = nullptr;    // [heads]: factor on every prepared query head (a temperature on its scores)
 };
 // q [T][heads][dim], k [T][kv_heads][dim], v [T][kv_heads][vdim] (rows ldq / ldk / ldv floats apart) are prepared in place; then the K / V
 // rows that later tokens can still see go to the cache (layout as launch_attn_kv_store).
@@ -320,10 +349,11 @@ int launch_dual_post(const float * o, const BatchView & b, int heads, int vdim, 
 //   decay_per_channel 0: S <- g S (g [T][heads]);  1: S <- diag(f) S (f [T][qk_heads][dim])
 //   delta 0: S <- S + k v^T;   1 (delta rule): u = beta (v - S^T k), S <- S + k u^T (beta [T][heads]), after the decay
 //   tied_key 1: k = 1 - f (needs decay_per_channel; io.k unused)
-//   y = S^T q, after the token's write.        Head h reads q / k head h / (heads / qk_heads).
+//   y = S^T q, after the token's write; bonus 1 (needs decay_per_channel, no delta, no tied key): y = (S + diag(u) k v^T)^T q with the state
+//   BEFORE the token's decay and write, u = io.bonus.        Head h reads q / k head h / (heads / qk_heads).
 struct GatedLinParams {
     int heads = 0, qk_heads = 0, dim = 0, vdim = 0;
-    int decay_per_channel = 0, delta = 0, tied_key = 0;
+    int decay_per_channel = 0, delta = 0, tied_key = 0, bonus = 0;
 };
 struct GatedLinIO {
     const float * q = nullptr;      int64_t ldq = 0;    // [qk_heads][dim]
@@ -331,6 +361,7 @@ struct GatedLinIO {
     const float * v = nullptr;      int64_t ldv = 0;    // [heads][vdim]
     const float * decay = nullptr;  int64_t ldd = 0;
     const float * beta = nullptr;   int64_t ldb = 0;
+    const float * bonus = nullptr;                      // [qk_heads][dim], the same for every token
 };
 int launch_gated_linattn(const GatedLinIO & io, const BatchView & b, const GatedLinParams & p, float * state, int64_t slot_stride, float * y,
                          cudaStream_t stream);
@@ -340,6 +371,17 @@ int launch_delta_prep(float * q, int64_t ldq, float * k, int64_t ldk, float * be
                       const float * dt_bias, int qk_heads, int heads, int dim, int n_tokens, cudaStream_t stream);
 // inputs of HGRN2, in place: q <- silu(q);  f <- lower + (1 - lower) * sigmoid(f + f_bias)      (n = heads * dim entries per token)
 int launch_hgrn2_prep(float * q, int64_t ldq, float * f, int64_t ldf, const float * f_bias, const float * lower, int n, int n_tokens, cudaStream_t stream);
+
+// ---- WKV mixer: token mix and decay ----
+// h = rmsnorm(x) * w;  planes: y[p * plane + t * width ..] = h[t] + (h[t-1] - h[t]) * mu[p] for p < n_planes in the operand type, and (yf given) the
+// same with mu[n_planes] in fp32.  The token before an entry's first one is the slot's shift state [width] (zeros for a new sequence), which
+// then holds the h of the entry's last token.
+int launch_rmsnorm_token_mix(const float * x, const BatchView & b, const float * w, float eps, const float * mu, int n_planes, float * shift_state,
+                             int64_t slot_stride, void * y, int64_t plane, int otype, float * yf, int width, cudaStream_t stream);
+// decay[t][c] = exp(-exp(w0[c] + sum_j w2[c][j] tanh(sum_k m[t][k] w1[j][k]))), fp32 throughout; w1 [rank][width], w2 [channels][rank];
+// tmp: [T][rank] floats
+int launch_lowrank_decay(const float * m, const float * w1, const float * w2, const float * w0, int n_tokens, int width, int rank, int channels, float * tmp,
+                         float * decay, cudaStream_t stream);
 
 // x[t] += (x0 ? x0[t] : 0) + (vec ? vec : 0), then y[t] = rmsnorm(x[t]) * w in the operand type: what opens a pass of a repeated block whose
 // passes add the embedding output and a step vector, with the first layer's norm

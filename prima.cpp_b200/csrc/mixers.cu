@@ -28,6 +28,28 @@ __global__ void k_embed(const WT * __restrict__ table, int width, const int32_t 
     }
 }
 
+// one CTA per token: the table row normed, and (y given) normed again for the first layer; every thread re-reads only what it has written itself
+template <typename WT, typename OT>
+__global__ void __launch_bounds__(256) k_embed_rmsnorm(const WT * __restrict__ table, int width, const int32_t * __restrict__ tokens, const float * __restrict__ w,
+                                                       float eps, float * __restrict__ x, const float * __restrict__ wn, OT * __restrict__ y) {
+    __shared__ float red[33];
+    const int t = blockIdx.x;
+    const WT * row = table + (int64_t) tokens[t] * width;
+    float * xr = x + (int64_t) t * width;
+    float s = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) { const float v = ld_f(row, i); s = fmaf(v, v, s); }
+    const float inv = 1.f / sqrtf(block_sum(s, red) / (float) width + eps);
+    float s2 = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = ld_f(row, i) * inv * w[i];
+        xr[i] = v;
+        s2 = fmaf(v, v, s2);
+    }
+    if (!y) return;
+    const float inv2 = 1.f / sqrtf(block_sum(s2, red) / (float) width + eps);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) put(y, (int64_t) t * width + i, xr[i] * inv2 * wn[i]);
+}
+
 template <typename OT>
 __global__ void k_cast(const float * __restrict__ x, OT * __restrict__ y, int64_t n) {
     const int64_t i = (int64_t) blockIdx.x * blockDim.x + threadIdx.x;
@@ -112,6 +134,15 @@ __global__ void k_relu2(const float * __restrict__ u, OT * __restrict__ y, int64
     const float v = fmaxf(u[i], 0.f);
     put(y, i, v * v);
 }
+__device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log1pf(expf(v)); }
+template <typename OT>
+__global__ void k_xielu(const float * __restrict__ u, const float * __restrict__ pq, OT * __restrict__ y, int64_t n) {
+    const int64_t i = (int64_t) blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const float z = u[i];
+    const float v = z > 0.f ? softplus_f(pq[0]) * z * z : (0.5f + softplus_f(pq[1])) * (expm1f(z) - z);
+    put(y, i, v + 0.5f * z);
+}
 __global__ void k_softcap(float * __restrict__ x, int64_t n, float cap) {
     const int64_t i = (int64_t) blockIdx.x * blockDim.x + threadIdx.x;
     if (i < n) x[i] = cap * tanhf(x[i] / cap);
@@ -190,6 +221,8 @@ __device__ __forceinline__ int cache_row(int p, int keep_first, int ring) { retu
 __device__ __forceinline__ float attn_key(const AttnIO & io, int64_t row, int kvh, int d, int DN) {
     return d < DN ? io.k[row * io.ldk + (int64_t) kvh * DN + d] : io.ks[row * io.ldks + (d - DN)];
 }
+// score of the sink of head h
+__device__ __forceinline__ float attn_sink(const AttnIO & io, int h) { return io.sink ? io.sink[h] : 0.f; }
 // factor on output element d of head h: sigmoid of a gate logit per head, per element, or none
 __device__ __forceinline__ float attn_gate(const AttnIO & io, int64_t row, int h, int d, int DV) {
     if (io.gate_mode == 1) return sigmoid_f(io.gate[row * io.ldg + h]);
@@ -297,9 +330,9 @@ __global__ void __launch_bounds__(AQ * 32) k_attn_window_prefill(const AttnIO io
     const bool qok = qi < n;
     for (int d = lane; d < D; d += 32) qs[warp * D + d] = qok ? io.q[(int64_t) (t_begin + qi) * io.ldq + h * D + d] : 0.f;
     const int q_last = min(q0 + AQ, n) - 1;
-    const bool windowed = a.window > 0;
-    const int w_lo = windowed ? max(0, q0 - a.window + 1) : 0;          // first key any query of the CTA sees through its window
-    const int s_hi = windowed ? min(a.keep_first, w_lo) : 0;            // kept first tokens below the window: [0, s_hi)
+    const int w_lo = attn_first_visible(a, q0);                         // first key any query of the CTA sees through its window or chunk
+    const int s_hi = min(a.keep_first, w_lo);                           // kept first tokens below the window: [0, s_hi)
+    const int lo_q = attn_first_visible(a, qi);                         // first key this warp's query sees
     float m = -INFINITY, l = 0.f, acc[NV];
 #pragma unroll
     for (int c = 0; c < NV; c++) acc[c] = 0.f;
@@ -320,7 +353,7 @@ __global__ void __launch_bounds__(AQ * 32) k_attn_window_prefill(const AttnIO io
             __syncthreads();
             if (!qok) continue;
             const int kj = k0 + lane;
-            bool valid = lane < nk && kj <= qi && (!windowed || qi - kj < a.window || kj < a.keep_first);
+            bool valid = lane < nk && kj <= qi && (kj >= lo_q || kj < a.keep_first);
             float s = 0.f;
             const float * qr = qs + warp * D, * kr = kt + lane * (D + 1);
             for (int d = 0; d < D; d++) s = fmaf(qr[d], kr[d], s);
@@ -330,7 +363,7 @@ __global__ void __launch_bounds__(AQ * 32) k_attn_window_prefill(const AttnIO io
         }
     }
     if (!qok) return;
-    if (a.sink && m != -INFINITY) l += expf(-m);   // the sink: a key of score 0 in the denominator only
+    if (a.sink && m != -INFINITY) l += expf(attn_sink(io, h) - m);   // the sink: a key in the denominator only
     const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
     for (int c = 0; c < NV; c++) {
@@ -370,13 +403,14 @@ __global__ void __launch_bounds__(256) k_attn_window_prefill_tiled(const AttnIO 
         Qt[d * PQS + q] = q0 + q < n ? io.q[(int64_t) (t_begin + q0 + q) * io.ldq + h * D + d] * a.scale : 0.f;
     }
     const int q_last = min(q0 + PQ, n) - 1;
-    const bool windowed = a.window > 0;
-    const int w_lo = windowed ? max(0, q0 - a.window + 1) : 0;
-    const int s_hi = windowed ? min(a.keep_first, w_lo) : 0;
+    const int w_lo = attn_first_visible(a, q0);
+    const int s_hi = min(a.keep_first, w_lo);
     float m[4], l[4], acc[4][NVC];
+    int lo_q[4];                        // first key each of the thread's queries sees
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         m[i] = -INFINITY; l[i] = 0.f;
+        lo_q[i] = attn_first_visible(a, q0 + ty * 4 + i);
 #pragma unroll
         for (int c = 0; c < NVC; c++) acc[i][c] = 0.f;
     }
@@ -437,7 +471,7 @@ __global__ void __launch_bounds__(256) k_attn_window_prefill_tiled(const AttnIO 
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
                     const int kj = k0 + tx + 16 * j;
-                    const bool valid = tx + 16 * j < nk && kj <= qi && (!windowed || qi - kj < a.window || kj < a.keep_first);
+                    const bool valid = tx + 16 * j < nk && kj <= qi && (kj >= lo_q[i] || kj < a.keep_first);
                     float v = s[i][j];
                     if (a.softcap > 0.f) v = a.softcap * tanhf(v / a.softcap);
                     s[i][j] = valid ? v : -INFINITY;
@@ -480,7 +514,7 @@ __global__ void __launch_bounds__(256) k_attn_window_prefill_tiled(const AttnIO 
     for (int i = 0; i < 4; i++) {
         const int qi = q0 + ty * 4 + i;
         if (qi >= n) continue;
-        if (a.sink && m[i] != -INFINITY) l[i] += expf(-m[i]);
+        if (a.sink && m[i] != -INFINITY) l[i] += expf(attn_sink(io, h) - m[i]);
         const float inv = l[i] > 0.f ? 1.f / l[i] : 0.f;
 #pragma unroll
         for (int c = 0; c < NVC; c++) {
@@ -521,7 +555,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) k_attn_window_decode(const Att
     float m = -INFINITY, l = 0.f, acc[NV];
 #pragma unroll
     for (int c = 0; c < NV; c++) acc[c] = 0.f;
-    const int rows_used = min(a.cache_rows, pi + 1);
+    const int rows_used = min(a.cache_rows, (a.chunk > 0 ? pi % a.chunk : pi) + 1);   // a chunk's rows start at row 0 of the ring
     const int r_begin = gridDim.z > 1 ? blockIdx.z * chunk : 0, r_end = gridDim.z > 1 ? min(rows_used, r_begin + chunk) : rows_used;
     const bool vec4 = (D & 3) == 0 && (KD & 3) == 0;
     for (int r0 = r_begin + warp * DEC_ROWS; r0 < r_end; r0 += nw * DEC_ROWS) {
@@ -610,7 +644,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) k_attn_window_decode(const Att
             }
             return;
         }
-        if (a.sink && M != -INFINITY) L += expf(-M);
+        if (a.sink && M != -INFINITY) L += expf(attn_sink(io, h) - M);
         const float inv = L > 0.f ? 1.f / L : 0.f;
 #pragma unroll
         for (int c = 0; c < NV; c++) {
@@ -634,7 +668,7 @@ __global__ void __launch_bounds__(128) k_attn_decode_merge(const AttnIO io, cons
         const float ms = pp[(int64_t) s * (DV + 2)];
         if (ms != -INFINITY) L += pp[(int64_t) s * (DV + 2) + 1] * expf(ms - M);
     }
-    if (a.sink && M != -INFINITY) L += expf(-M);
+    if (a.sink && M != -INFINITY) L += expf(attn_sink(io, h) - M);
     const float inv = L > 0.f ? 1.f / L : 0.f;
     for (int d = threadIdx.x; d < DV; d += blockDim.x) {
         float o = 0.f;
@@ -834,6 +868,16 @@ int launch_embed(const void * table, int type, int width, const int32_t * tokens
         else k_embed<float><<<n_tokens, 128, 0, st>>>((const float *) table, width, tokens, x, x_copy);
     });
 }
+int launch_embed_rmsnorm(const void * table, int type, int width, const int32_t * tokens, int n_tokens, const float * w, float eps, float * x, const float * wn,
+                         void * y, int otype, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
+    if (!w || (y && (!wn || otype != type))) return (int) cudaErrorInvalidValue;
+    return ck_launch([&] {
+        if (type == T_BF16)
+            k_embed_rmsnorm<__nv_bfloat16, __nv_bfloat16><<<n_tokens, 256, 0, st>>>((const __nv_bfloat16 *) table, width, tokens, w, eps, x, wn, (__nv_bfloat16 *) y);
+        else k_embed_rmsnorm<float, float><<<n_tokens, 256, 0, st>>>((const float *) table, width, tokens, w, eps, x, wn, (float *) y);
+    });
+}
 int launch_cast(const float * x, void * y, int otype, int64_t n, cudaStream_t st) {
     if (n <= 0) return 0;
     const unsigned grid = (unsigned) ((n + 255) / 256);
@@ -871,6 +915,15 @@ int launch_relu2(const float * u, void * y, int otype, int64_t n, cudaStream_t s
     return ck_launch([&] {
         if (otype == T_BF16) k_relu2<__nv_bfloat16><<<grid, 256, 0, st>>>(u, (__nv_bfloat16 *) y, n);
         else k_relu2<float><<<grid, 256, 0, st>>>(u, (float *) y, n);
+    });
+}
+int launch_xielu(const float * u, const float * pq, void * y, int otype, int64_t n, cudaStream_t st) {
+    if (n <= 0) return 0;
+    if (!pq) return (int) cudaErrorInvalidValue;
+    const unsigned grid = (unsigned) ((n + 255) / 256);
+    return ck_launch([&] {
+        if (otype == T_BF16) k_xielu<__nv_bfloat16><<<grid, 256, 0, st>>>(u, pq, (__nv_bfloat16 *) y, n);
+        else k_xielu<float><<<grid, 256, 0, st>>>(u, pq, (float *) y, n);
     });
 }
 int launch_softcap(float * x, int64_t n, float cap, cudaStream_t st) {

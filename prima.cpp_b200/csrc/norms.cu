@@ -89,6 +89,31 @@ __global__ void __launch_bounds__(256) k_shift_state(const float * __restrict__ 
     for (int i = threadIdx.x; i < width; i += blockDim.x) st[i] = in[i] * inv[i / part] * w[i];
 }
 
+// one CTA per token: the norm of the token and of the one before it, then one blend per plane (operand type) and one more in fp32
+template <typename OT>
+__global__ void __launch_bounds__(1024) k_rmsnorm_token_mix(const float * __restrict__ x, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
+                                                            const int32_t * __restrict__ entry_of, const float * __restrict__ w, float eps,
+                                                            const float * __restrict__ mu, int n_planes, float * __restrict__ shift_state, int64_t slot_stride,
+                                                            OT * __restrict__ y, int64_t plane, float * __restrict__ yf, int width) {
+    __shared__ float red[33];
+    __shared__ float inv[1], invp[1];
+    const int t = blockIdx.x;
+    const int e = entry_of[t];
+    const bool first = t == off[e], only = first && off[e + 1] == t + 1;
+    const float * in = x + (int64_t) t * width;
+    group_inv_rms(in, width, 1, eps, inv, red);
+    if (!first) group_inv_rms(in - width, width, 1, eps, invp, red);
+    const float i0 = inv[0], ip = first ? 0.f : invp[0];
+    float * st = shift_state + (int64_t) slot[e] * slot_stride;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float wi = w[i], h = in[i] * i0 * wi;
+        const float d = (first ? st[i] : in[i - width] * ip * wi) - h;
+        for (int p = 0; p < n_planes; p++) put(y, p * plane + (int64_t) t * width + i, fmaf(d, mu[(int64_t) p * width + i], h));
+        if (yf) yf[(int64_t) t * width + i] = fmaf(d, mu[(int64_t) n_planes * width + i], h);
+        if (only) st[i] = h;   // an entry of one token: this CTA is the state's only reader and writer (k_shift_state serves longer entries)
+    }
+}
+
 // sum_j coef[j] * planes[j * plane_stride + i], eight planes' loads in flight
 __device__ __forceinline__ float depth_sum(const float * __restrict__ planes, int64_t plane_stride, const float * __restrict__ coef, int n, int64_t i) {
     float acc = 0.f;
@@ -220,6 +245,22 @@ int launch_group_rmsnorm_shift(const float * x, const BatchView & b, const float
     });
     if (rc || b.max_n <= 1) return rc;   // one-token entries have written their state themselves
     return ck_launch([&] { k_shift_state<<<b.n_entries, 256, 0, st>>>(x, b.slot, b.off, w, groups, eps, shift_state, slot_stride, width); });
+}
+int launch_rmsnorm_token_mix(const float * x, const BatchView & b, const float * w, float eps, const float * mu, int n_planes, float * shift_state,
+                             int64_t slot_stride, void * y, int64_t plane, int otype, float * yf, int width, cudaStream_t st) {
+    if (b.n_tokens <= 0) return 0;
+    if (!mu || !shift_state || n_planes < 0 || (n_planes > 0 && !y)) return (int) cudaErrorInvalidValue;
+    const int threads = b.n_tokens >= 256 || width <= 1024 ? 256 : 1024;   // few tokens: more of a row's loads in flight
+    int rc = ck_launch([&] {
+        if (otype == T_BF16)
+            k_rmsnorm_token_mix<__nv_bfloat16><<<b.n_tokens, threads, 0, st>>>(x, b.slot, b.off, b.entry_of, w, eps, mu, n_planes, shift_state, slot_stride,
+                                                                               (__nv_bfloat16 *) y, plane, yf, width);
+        else
+            k_rmsnorm_token_mix<float><<<b.n_tokens, threads, 0, st>>>(x, b.slot, b.off, b.entry_of, w, eps, mu, n_planes, shift_state, slot_stride, (float *) y,
+                                                                       plane, yf, width);
+    });
+    if (rc || b.max_n <= 1) return rc;   // one-token entries have written their state themselves
+    return ck_launch([&] { k_shift_state<<<b.n_entries, 256, 0, st>>>(x, b.slot, b.off, w, 1, eps, shift_state, slot_stride, width); });
 }
 int launch_depth_average(const float * planes, int64_t plane_stride, const float * coef, int n, float * out, int64_t count, cudaStream_t st) {
     if (count <= 0 || n <= 0) return 0;

@@ -2,7 +2,8 @@
 equal width / feed-forward / head sizes / number of layer runs: Vamidra beside the Llama graph over Q4_K weights (``bench.py --arch
 vamidra``), Mumizen beside Vamidra (``bench.py --arch mumizen``, :func:`run_mumizen`), Sapudra beside Vamidra and, for its experts, Mumizen
 (``bench.py --arch sapudra``, :func:`run_sapudra`), Zevedra beside Vamidra (attention, convolution, plain products) and Mumizen (recurrence,
-experts) (``bench.py --arch zevedra``, :func:`run_zevedra`).  Prints one JSON line.
+experts) (``bench.py --arch zevedra``, :func:`run_zevedra`), Ruvuvik beside Mumizen (latent attention, linear attention) and Vamidra
+(windowed attention) (``bench.py --arch ruvuvik``, :func:`run_ruvuvik`).  Prints one JSON line.
 
 Per size: prompt tokens/s (one sequence of 512 and 2048 tokens) and decode tokens/s (batch 1 and 8 at a 1024-token context) of both
 models through their public entry points (host token ids in, host logits / greedy tokens out), the device time of a prompt and of a
@@ -69,6 +70,8 @@ def run(args, pkg, lib):
         return run_sapudra(args, pkg, lib)
     if args.arch == "zevedra":
         return run_zevedra(args, pkg, lib)
+    if args.arch == "ruvuvik":
+        return run_ruvuvik(args, pkg, lib)
     import numpy as np
     import torch
     hbm, tflops, src = peaks()
@@ -695,6 +698,142 @@ def run_zevedra(args, pkg, lib):
         out["mumizen_like_kernels"] = e
         res["sizes"][key] = out
         torch.cuda.empty_cache()
+    res["gpu_launches"] = int(lib.c.pb200_kernel_launches())
+    print(json.dumps(res))
+    return res
+
+
+# ---------------------------------------------------------------------------------------------------------------
+RUVUVIK_SIZES = {
+    "w2048": dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, wkv_heads=16, wkv_dim=128, decay_rank=64),
+    "w4096": dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, wkv_heads=32, wkv_dim=128, decay_rank=64),
+}
+
+
+def ruvuvik_layers(s, z):
+    """One layer of each mixer at the width / feed-forward / head sizes of SIZES."""
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot_dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"],
+                     "scale": (z["dim"] + z["rot_dim"]) ** -0.5, "rot": {"base": 500000.0, "dims": z["rot_dim"]}}}
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5, "softcap": 50.0,
+                     "mask": {"size": 2 * s["window"]}, "rot": {"base": 1000000.0, "dims": s["dim"]}}}
+    wkv = {"type": "wkv", "mlp": mlp, "mixer": {"heads": z["wkv_heads"], "dim": z["wkv_dim"], "decay_rank": z["decay_rank"]}}
+    return {"latent": lat, "attention": att, "wkv": wkv}
+
+
+def ruvuvik_config(s, layers):
+    return {"architecture": "Ruvuvik", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "layers": layers}
+
+
+def ruvuvik_products(s, cfg, prompt):
+    """(N, K) of the dense products of one token through all layer runs (head and the fp32 map of the decay not included)."""
+    W, out = s["width"], []
+    for l in cfg["layers"]:
+        m = l["mixer"]
+        if l["type"] == "latent_attention":
+            H = m["heads"]
+            out += [(H * (m["dim"] + m["rot_dim"]) + m["kv_rank"] + m["rot_dim"], W), (W, H * m["vdim"])]
+            if prompt:
+                out += [(H * (m["dim"] + m["vdim"]), m["kv_rank"])]
+        elif l["type"] == "attention":
+            out += [(m["heads"] * m["dim"] + m["kv_heads"] * (m["dim"] + m["vdim"]) + m["heads"], W), (W, m["heads"] * m["vdim"])]
+        else:
+            HD = m["heads"] * m["dim"]
+            out += [(4 * HD, W), (W, HD)]
+        out += [(l["mlp"]["ff"], W), (W, l["mlp"]["ff"])]
+    return out
+
+
+def run_ruvuvik(args, pkg, lib):
+    """Ruvuvik beside Mumizen (latent attention, linear attention with a matrix state, dense feed-forward: the closest existing model) and
+    Vamidra (windowed attention) at equal width / feed-forward / head sizes and six layer runs each: whole-model prompt and decode
+    throughput through the public entry points.  For the like kernels, models whose three layers all have ONE mixer: device time per kernel
+    category turned into a distance from the roofline."""
+    import numpy as np
+    import torch
+    hbm, tflops, src = peaks()
+    res = {"metric": "Ruvuvik prompt / decode throughput beside Mumizen and Vamidra at equal size", "impl": "b200", "arch": "Ruvuvik", "n_gpus": 1,
+           "dtype": "bf16", "data": "synthetic random weights", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": src}, "sizes": {}}
+    rng = np.random.default_rng(0)
+    CTX = 1024
+
+    def measured(cfg):
+        m = pkg.Model.from_config(cfg, dtype="bfloat16", n_ctx=4096, n_seq=16)
+        m.synth(0, 7)
+        m.finalize()
+        v = measure(m, cfg["vocab"], args, rng, CTX)
+        m.close()
+        torch.cuda.empty_cache()
+        return v
+
+    def dense_fracs(a, prompt_shapes, step_shapes, head):
+        for T in (512, 2048):
+            a[f"prompt{T}_dense_frac_of_tensor_peak"] = 2.0 * sum(n * k for n, k in prompt_shapes) * T / a[f"prompt{T}_device_ms"]["dense"] / 1e9 / tflops
+        wb = 2.0 * sum(n * k for n, k in step_shapes)
+        a["weight_bytes_per_token"] = wb + 2.0 * head
+        for B in (1, 8):
+            a[f"decode_b{B}_dense_frac_of_hbm_peak"] = wb / a[f"decode_b{B}_device_ms"]["dense"] / 1e6 / hbm
+            a[f"decode_b{B}_whole_step_frac_of_hbm_peak"] = a["weight_bytes_per_token"] / a[f"decode_b{B}_ms_per_step"] / 1e6 / hbm
+
+    for key in ([args.arch_size] if args.arch_size != "all" else list(SIZES)):
+        s, z, mz = SIZES[key], RUVUVIK_SIZES[key], MUMIZEN_SIZES[key]
+        W, V, D = s["width"], s["vocab"], s["dim"]
+        L = ruvuvik_layers(s, z)
+        out = {"config": dict(z, width=W, ff=s["ff"], kv_heads=s["kv_heads"], chunk=2 * s["window"], vocab=V), "layers": 6}
+        # ---------------- whole models, six layer runs each ----------------
+        cfg = ruvuvik_config(s, [L["latent"], L["attention"], L["latent"], L["wkv"], L["attention"], L["wkv"]])
+        a = measured(cfg)
+        dense_fracs(a, ruvuvik_products(s, cfg, True), ruvuvik_products(s, cfg, False), V * W)
+        out["ruvuvik"] = a
+        vcfg = vamidra_config(s)
+        b = measured(vcfg)
+        dense_fracs(b, dense_shapes(s, vcfg), dense_shapes(s, vcfg), V * W)
+        out["vamidra"] = b
+        mcfg = mumizen_config(s, mz)
+        ml = {l["type"]: dict(l, mlp=mcfg["layers"][0]["mlp"]) for l in mcfg["layers"][:3]}
+        lin, mlat = ml["retention"], ml["latent_attention"]
+        mcfg = dict(mcfg, layers=[mlat, lin, mlat, lin, lin, lin])       # dense feed-forward in every layer
+        c = measured(mcfg)
+        dense_fracs(c, mumizen_products(mcfg, True)[0], mumizen_products(mcfg, False)[0], V * W)
+        out["mumizen"] = c
+        # ---------------- one mixer at a time, three layers ----------------
+        like = {}
+        probes = {"ruvuvik_latent": ruvuvik_config(s, [L["latent"]] * 3), "mumizen_latent": dict(mcfg, layers=[mlat] * 3),
+                  "ruvuvik_attention": ruvuvik_config(s, [L["attention"]] * 3), "vamidra_attention": dict(vcfg, layers=[vcfg["layers"][0]] * 3, loop=None),
+                  "ruvuvik_wkv": ruvuvik_config(s, [L["wkv"]] * 3), "mumizen_retention": dict(mcfg, layers=[lin] * 3)}
+        for name, pc in probes.items():
+            v = measured(pc)
+            r = {}
+            for T in (512, 2048):
+                pm = v[f"prompt{T}_device_ms"]
+                r[f"prompt{T}_device_ms"] = pm
+                if name.endswith("_latent"):
+                    r[f"prompt{T}_attention_tflops"] = 3 * 2.0 * z["heads"] * (z["dim"] + z["rot_dim"] + z["vdim"]) * (T * (T + 1) // 2) / pm["attention"] / 1e9
+                elif name == "ruvuvik_attention":
+                    r[f"prompt{T}_attention_tflops"] = 3 * 4.0 * D * s["heads"] * sum(i % (2 * s["window"]) + 1 for i in range(T)) / pm["attention"] / 1e9
+                elif name == "vamidra_attention":
+                    vis = sum(min(i + 1, s["window"]) + max(0, min(s["keep_first"], i + 1 - s["window"])) for i in range(T))
+                    r[f"prompt{T}_attention_tflops"] = 3 * 4.0 * D * s["heads"] * vis / pm["attention"] / 1e9
+                else:
+                    r[f"prompt{T}_scan_state_updates_per_ns"] = 3.0 * z["wkv_heads"] * z["wkv_dim"] ** 2 * T / pm["scan"] / 1e6
+                    r[f"prompt{T}_norm_gbs"] = (3 * T * (4.0 * W + 12.0 * W + 6.0 * W + 10.0 * z["wkv_heads"] * z["wkv_dim"]) if name == "ruvuvik_wkv" else
+                                                3 * T * (6.0 * W + 6.0 * W + 10.0 * z["wkv_heads"] * z["wkv_dim"])) / pm["norm"] / 1e6
+            for B in (1, 8):
+                pm = v[f"decode_b{B}_device_ms"]
+                r[f"decode_b{B}_device_ms"] = pm
+                if name.endswith("_latent"):
+                    r[f"decode_b{B}_attention_gbs"] = 3.0 * B * CTX * (z["kv_rank"] + z["rot_dim"]) * 4.0 / pm["attention"] / 1e6
+                elif name.endswith("_attention"):
+                    rows = min(CTX, s["window"] + s["keep_first"]) if name.startswith("vamidra") else CTX
+                    r[f"decode_b{B}_attention_gbs"] = 3.0 * B * rows * s["kv_heads"] * 2 * D * 4.0 / pm["attention"] / 1e6
+                else:
+                    r[f"decode_b{B}_scan_gbs"] = 3.0 * B * z["wkv_heads"] * z["wkv_dim"] ** 2 * 8.0 / pm["scan"] / 1e6
+                r[f"decode_b{B}_ms_per_step"] = v[f"decode_b{B}_ms_per_step"]
+            like[name] = r
+        out["like_kernels"] = like
+        res["sizes"][key] = out
     res["gpu_launches"] = int(lib.c.pb200_kernel_launches())
     print(json.dumps(res))
     return res
