@@ -13,13 +13,13 @@
 #include <cstdlib>
 
 #include "layers.h"
-
-extern std::atomic<uint64_t> g_launches;
+#include "mixers.cuh"
 
 namespace pb {
 
 int launch_dense_tc(const __nv_bfloat16 * A, int64_t lda, const __nv_bfloat16 * W, int64_t ldw, float * C, int64_t ldc, int T, int N, int K,
-                    const float * bias, const float * resid, int64_t ldr, float alpha, cudaStream_t stream, int plane_rows = 0, int64_t a_plane = 0);   // dense_tc.cu
+                    const float * bias, const float * resid, int64_t ldr, float alpha, cudaStream_t stream, int plane_rows = 0, int64_t a_plane = 0,
+                    DenseAct act = DenseAct());   // dense_tc.cu
 bool dense_tc_ok(int T, int N, int K, int64_t lda, int64_t ldw, const void * A, const void * W);
 int launch_dense_tc_grouped(const __nv_bfloat16 * A, int64_t lda, const __nv_bfloat16 * W, int64_t ldw, int64_t w_stride, float * C, int64_t ldc,
                             const int32_t * start, const int32_t * count, int groups, int max_rows, int N, int K, cudaStream_t st);
@@ -35,7 +35,8 @@ constexpr int TM = 64, TN = 64, TK = 16;
 
 template <typename WT>
 __global__ void __launch_bounds__(256) k_dense_tile(const WT * __restrict__ A, int64_t lda, const WT * __restrict__ W, int64_t ldw, float * C, int64_t ldc,
-                                                    int T, int N, int K, const float * __restrict__ bias, const float * resid, int64_t ldr, float alpha) {
+                                                    int T, int N, int K, const float * __restrict__ bias, const float * resid, int64_t ldr, float alpha,
+                                                    DenseAct act) {
     __shared__ float As[TK][TM + 4];
     __shared__ float Ws[TK][TN + 4];
     const int t0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
@@ -70,6 +71,7 @@ __global__ void __launch_bounds__(256) k_dense_tile(const WT * __restrict__ A, i
         }
         __syncthreads();
     }
+    const float xp = act.xielu ? softplus_f(act.xielu[0]) : 0.f, xn = act.xielu ? 0.5f + softplus_f(act.xielu[1]) : 0.f;
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const int t = t0 + ty * 4 + i;
@@ -81,7 +83,8 @@ __global__ void __launch_bounds__(256) k_dense_tile(const WT * __restrict__ A, i
             float v = alpha * acc[i][j];
             if (bias) v += bias[n];
             if (resid) v += resid[(int64_t) t * ldr + n];
-            C[(int64_t) t * ldc + n] = v;
+            if (act.xielu) put((WT *) act.y, (int64_t) t * act.ldy + n, xielu_f(v, xp, xn));
+            else C[(int64_t) t * ldc + n] = v;
         }
     }
 }
@@ -109,7 +112,7 @@ template <int N> __device__ __forceinline__ void unpack(const uint4 & raw, float
 template <typename WT, int TB, bool VEC>
 __global__ void __launch_bounds__(256) k_dense_rows(const WT * __restrict__ A, int64_t lda, const WT * __restrict__ W, int64_t ldw, float * C, int64_t ldc,
                                                     int T, int N, int K, const float * __restrict__ bias, const float * resid, int64_t ldr, float alpha,
-                                                    int KS, int plane_rows, int64_t a_plane) {
+                                                    int KS, int plane_rows, int64_t a_plane, DenseAct act) {
     __shared__ float parts[8][TB];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int rows_per_cta = (blockDim.x >> 5) / KS;
@@ -169,13 +172,15 @@ __global__ void __launch_bounds__(256) k_dense_rows(const WT * __restrict__ A, i
         }
     }
     if (lane == 0 && live) {
+        const float xp = act.xielu ? softplus_f(act.xielu[0]) : 0.f, xn = act.xielu ? 0.5f + softplus_f(act.xielu[1]) : 0.f;
 #pragma unroll
         for (int t = 0; t < TB; t++) {
             if (t < T) {
                 float v = acc[t] * alpha;
                 if (bias) v += bias[n];
                 if (resid) v += resid[(int64_t) t * ldr + n];
-                C[(int64_t) t * ldc + n] = v;
+                if (act.xielu) put((WT *) act.y, (int64_t) t * act.ldy + n, xielu_f(v, xp, xn));
+                else C[(int64_t) t * ldc + n] = v;
             }
         }
     }
@@ -196,7 +201,8 @@ int rows_max_t() {
 
 template <typename WT>
 int dense_typed(const WT * A, int64_t lda, const WT * W, int64_t ldw, float * C, int64_t ldc, int T, int N, int K, const float * bias,
-                const float * resid, int64_t ldr, float alpha, cudaStream_t st, int plane_rows = 0, int64_t a_plane = 0) {
+                const float * resid, int64_t ldr, float alpha, cudaStream_t st, int plane_rows = 0, int64_t a_plane = 0,
+                const DenseAct & act = DenseAct()) {
     if (T <= ROWS_MAX_T) {
         constexpr int V = Vec16<WT>::n;
         const bool vec = K % V == 0 && lda % V == 0 && ldw % V == 0 && a_plane % V == 0 && ((uintptr_t) A & 15) == 0 && ((uintptr_t) W & 15) == 0;
@@ -206,20 +212,20 @@ int dense_typed(const WT * A, int64_t lda, const WT * W, int64_t ldw, float * C,
         const dim3 grid((unsigned) ((N + 8 / KS - 1) / (8 / KS))), block(256);
         g_launches++;
         if (T <= 1) {
-            if (vec) k_dense_rows<WT, 1, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
-            else k_dense_rows<WT, 1, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
+            if (vec) k_dense_rows<WT, 1, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
+            else k_dense_rows<WT, 1, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
         } else if (T <= 4) {
-            if (vec) k_dense_rows<WT, 4, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
-            else k_dense_rows<WT, 4, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
+            if (vec) k_dense_rows<WT, 4, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
+            else k_dense_rows<WT, 4, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
         } else {
-            if (vec) k_dense_rows<WT, ROWS_MAX_T, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
-            else k_dense_rows<WT, ROWS_MAX_T, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane);
+            if (vec) k_dense_rows<WT, ROWS_MAX_T, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
+            else k_dense_rows<WT, ROWS_MAX_T, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
         }
         return (int) cudaGetLastError();
     }
     const dim3 grid((unsigned) ((N + TN - 1) / TN), (unsigned) ((T + TM - 1) / TM)), block(256);
     g_launches++;
-    k_dense_tile<WT><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha);
+    k_dense_tile<WT><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, act);
     return (int) cudaGetLastError();
 }
 
@@ -258,6 +264,15 @@ int launch_dense_planes(int type, const void * A, int64_t a_plane, int64_t lda, 
         if (rc) return rc;
     }
     return 0;
+}
+
+int launch_dense_act(int type, const void * A, int64_t lda, const void * W, int64_t ldw, const DenseAct & act, int T, int N, int K, cudaStream_t st) {
+    if (T <= 0 || N <= 0) return 0;
+    if (K <= 0 || !A || !W || !act.xielu || !act.y || (type != 0 && type != T_BF16)) return (int) cudaErrorInvalidValue;
+    if (type == 0) return dense_typed<float>((const float *) A, lda, (const float *) W, ldw, nullptr, 0, T, N, K, nullptr, nullptr, 0, 1.f, st, 0, 0, act);
+    const __nv_bfloat16 * a = (const __nv_bfloat16 *) A, * w = (const __nv_bfloat16 *) W;
+    if (T > rows_max_t() && dense_tc_ok(T, N, K, lda, ldw, A, W)) return launch_dense_tc(a, lda, w, ldw, nullptr, 0, T, N, K, nullptr, nullptr, 0, 1.f, st, 0, 0, act);
+    return dense_typed<__nv_bfloat16>(a, lda, w, ldw, nullptr, 0, T, N, K, nullptr, nullptr, 0, 1.f, st, 0, 0, act);
 }
 
 int launch_dense(int type, const void * A, int64_t lda, const void * W, int64_t ldw, float * C, int64_t ldc, int T, int N, int K, const float * bias,

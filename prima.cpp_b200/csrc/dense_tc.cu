@@ -2,7 +2,7 @@
 //   C[t][n] = alpha * sum_k A[t][k] W[n][k] (+ bias[n]) (+ resid[t][n]),   A [T][K], W [N][K] row-major bf16, C f32.
 // One CTA computes a tile of 128 weight rows x BN tokens: tcgen05.mma kind::f16 (bf16 operands, M = 128, N = BN, K = 16) with the fp32
 // accumulator in TMEM, both operands staged from their row-major global layout into the swizzle-128B K-major shared-memory image by
-// 16-byte cp.async pieces (4 producer warps, 4 stages of 64 k), one elected thread issuing the MMAs, tcgen05.commit handing stages back,
+// 16-byte cp.async pieces (4 producer warps, 4 to 8 stages of 64 k: narrow token tiles keep more of them in flight), one elected thread issuing the MMAs, tcgen05.commit handing stages back,
 // and all 8 warps reading the accumulator out with tcgen05.ld for the epilogue (lane = weight row, so a warp stores 32 consecutive
 // floats of one token's row).  K is never split: an output element is one fixed-order sum.  Every wait is bounded (common.cuh).
 #include <cuda_bf16.h>
@@ -12,16 +12,17 @@
 
 #include "launch.h"
 #include "layers.h"
-
-extern std::atomic<uint64_t> g_launches;
+#include "mixers.cuh"
 
 namespace pb {
 namespace {
 
-constexpr int TC_BM = 128, TC_BK = 64, TC_STAGES = 4, TC_LAG = 2, TC_PRODUCERS = 128, TC_THREADS = 256;
+constexpr int TC_BM = 128, TC_BK = 64, TC_MAX_STAGES = 8, TC_PRODUCERS = 128, TC_THREADS = 256;
+
+// Stages: up to 192 KB of them while every CTA has an SM to itself; with more tiles than SMs the narrow tile takes four, so that two CTAs share one.
 
 struct TcCtl {
-    uint64_t full[TC_STAGES], empty[TC_STAGES], acc_ready;
+    uint64_t full[TC_MAX_STAGES], empty[TC_MAX_STAGES], acc_ready;
     uint32_t tmem_base;
     int abort;
 };
@@ -40,6 +41,7 @@ struct TcParams {
     const int32_t * grp_start; const int32_t * grp_count; int64_t grp_w_stride; int groups;
     // planes: weight rows [p * plane_rows, + plane_rows) meet the operand a_plane * p elements further on (plane_rows a multiple of the row tile)
     int plane_rows; int64_t a_plane;
+    DenseAct act;
 };
 
 __device__ __forceinline__ uint64_t desc_sw128(uint32_t saddr) {   // K-major, SWIZZLE_128B: rows of 128 B, 8-row groups 1024 B apart
@@ -83,7 +85,20 @@ __device__ __forceinline__ void stage_rows(uint32_t dst, const __nv_bfloat16 * M
     }
 }
 
-template <int BN>
+// waits until at most n of this thread's newest copy groups are still in flight
+__device__ __forceinline__ void cp_wait(int n) {
+    switch (n) {
+    case 0: asm volatile("cp.async.wait_group 0;" ::: "memory"); break;
+    case 1: asm volatile("cp.async.wait_group 1;" ::: "memory"); break;
+    case 2: asm volatile("cp.async.wait_group 2;" ::: "memory"); break;
+    case 3: asm volatile("cp.async.wait_group 3;" ::: "memory"); break;
+    case 4: asm volatile("cp.async.wait_group 4;" ::: "memory"); break;
+    case 5: asm volatile("cp.async.wait_group 5;" ::: "memory"); break;
+    default: asm volatile("cp.async.wait_group 6;" ::: "memory"); break;
+    }
+}
+
+template <int BN, int TC_STAGES>
 __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constant__ TcParams P) {
     const __nv_bfloat16 * Am = P.A, * Wm = P.W;
     float * Cm = P.C;
@@ -103,6 +118,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constan
     }
     extern __shared__ uint8_t smem_raw[];
     uint8_t * smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
+    constexpr int TC_LAG = TC_STAGES - 2;
     constexpr int A_BYTES = TC_BM * 128, B_BYTES = BN * 128, STAGE = A_BYTES + B_BYTES;
     TcCtl * ctl = reinterpret_cast<TcCtl *>(smem + TC_STAGES * STAGE);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -126,7 +142,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constan
     volatile int * cta_abort = &ctl->abort;
 
     if (warp < 4) {
-        // ---- producers: stage u of A (weights) and B (activations) into ring slot u % 4 ----
+        // ---- producers: stage u of A (weights) and B (activations) into its ring slot ----
         const int p = threadIdx.x;
         int signalled = 0;
         auto signal = [&](int u) {
@@ -141,13 +157,12 @@ __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constan
             stage_rows<BN>(base + A_BYTES, Am, P.lda, t0, Tn, u * TC_BK, P.K, p);
             asm volatile("cp.async.commit_group;" ::: "memory");
             if (u - signalled >= TC_LAG) {
-                asm volatile("cp.async.wait_group 2;" ::: "memory");
+                cp_wait(TC_LAG);
                 signal(signalled++);
             }
         }
         while (signalled < nk) {
-            if (nk - 1 - signalled >= 1) asm volatile("cp.async.wait_group 1;" ::: "memory");
-            else asm volatile("cp.async.wait_group 0;" ::: "memory");
+            cp_wait(nk - 1 - signalled);
             signal(signalled++);
         }
     } else if (warp == 4) {
@@ -174,6 +189,9 @@ __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constan
         const int quad = warp & 3, half = warp >> 2;
         const int n = n0 + quad * 32 + lane;
         const float bias = (P.bias && n < P.N) ? P.bias[n] : 0.f;
+        const float * pq = P.act.xielu;
+        const float xp = pq ? softplus_f(pq[0]) : 0.f, xn = pq ? 0.5f + softplus_f(pq[1]) : 0.f;
+        __nv_bfloat16 * ya = (__nv_bfloat16 *) P.act.y;
         for (int c0 = half * (BN / 2); c0 < (half + 1) * (BN / 2); c0 += 16) {
             if (t0 + c0 >= Tn) break;                                   // uniform over the warp
             uint32_t v[16];
@@ -192,7 +210,8 @@ __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constan
                     if (t < Tn) {
                         float y = P.alpha * __uint_as_float(v[i]) + bias;
                         if (P.resid) y += P.resid[(int64_t) t * P.ldr + n];
-                        Cm[(int64_t) t * P.ldc + n] = y;
+                        if (pq) put(ya, (int64_t) t * P.act.ldy + n, xielu_f(y, xp, xn));
+                        else Cm[(int64_t) t * P.ldc + n] = y;
                     }
                 }
             }
@@ -206,17 +225,23 @@ __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constan
     }
 }
 
-template <int BN> constexpr size_t tc_smem() { return 1024 + (size_t) TC_STAGES * (TC_BM * 128 + BN * 128) + sizeof(TcCtl) + 64; }
+template <int BN, int STAGES> constexpr size_t tc_smem() { return 1024 + (size_t) STAGES * (TC_BM * 128 + BN * 128) + sizeof(TcCtl) + 64; }
 
+template <int BN, int STAGES>
+int launch_tc_stages(const TcParams & P, const dim3 & grid, cudaStream_t st) {
+    static FuncAttrCache cache;
+    cudaError_t e = ensure_dyn_smem(cache, (const void *) k_dense_tc<BN, STAGES>, tc_smem<BN, STAGES>(), BN == 256);
+    if (e != cudaSuccess) return (int) e;
+    g_launches++;
+    k_dense_tc<BN, STAGES><<<grid, TC_THREADS, tc_smem<BN, STAGES>(), st>>>(P);
+    return (int) cudaGetLastError();
+}
 template <int BN>
 int launch_tc(const TcParams & P, cudaStream_t st) {
-    static FuncAttrCache cache;
-    cudaError_t e = ensure_dyn_smem(cache, (const void *) k_dense_tc<BN>, tc_smem<BN>(), BN == 256);
-    if (e != cudaSuccess) return (int) e;
     const dim3 grid((unsigned) ((P.N + TC_BM - 1) / TC_BM), (unsigned) ((P.T + BN - 1) / BN + (P.grp_count ? P.groups : 0)));
-    g_launches++;
-    k_dense_tc<BN><<<grid, TC_THREADS, tc_smem<BN>(), st>>>(P);
-    return (int) cudaGetLastError();
+    if (BN == 256) return launch_tc_stages<256, 4>(P, grid, st);
+    if (BN == 128) return launch_tc_stages<128, 6>(P, grid, st);
+    return (int64_t) grid.x * grid.y <= 148 ? launch_tc_stages<64, 8>(P, grid, st) : launch_tc_stages<64, 4>(P, grid, st);
 }
 
 }  // namespace
@@ -227,16 +252,26 @@ bool dense_tc_ok(int T, int N, int K, int64_t lda, int64_t ldw, const void * A, 
 }
 
 int launch_dense_tc(const __nv_bfloat16 * A, int64_t lda, const __nv_bfloat16 * W, int64_t ldw, float * C, int64_t ldc, int T, int N, int K, const float * bias,
-                    const float * resid, int64_t ldr, float alpha, cudaStream_t st, int plane_rows, int64_t a_plane) {
-    TcParams P{A, lda, W, ldw, C, ldc, bias, resid, ldr, alpha, T, N, K, abort_flag(), nullptr, nullptr, 0, 0, plane_rows, a_plane};
-    return T <= 64 ? launch_tc<64>(P, st) : T <= 128 ? launch_tc<128>(P, st) : launch_tc<256>(P, st);
+                    const float * resid, int64_t ldr, float alpha, cudaStream_t st, int plane_rows, int64_t a_plane, DenseAct act) {
+    TcParams P{A, lda, W, ldw, C, ldc, bias, resid, ldr, alpha, T, N, K, abort_flag(), nullptr, nullptr, 0, 0, plane_rows, a_plane, act};
+    if (T <= 64) return launch_tc<64>(P, st);
+    // token tile: the one whose waves of CTAs cost least, a k step of a tile being about its tokens plus the weight rows' share of the loads.  Few
+    // weight rows leave most SMs idle under wide tiles; an element's sum runs over k in the same order under any of them.
+    int best = 0;
+    int64_t best_cost = 0;
+    for (const int bn : {256, 128, 64}) {
+        if (bn > 64 && T <= bn / 2) continue;
+        const int64_t tiles = (int64_t) ((N + TC_BM - 1) / TC_BM) * ((T + bn - 1) / bn), cost = (tiles + 147) / 148 * (bn + 48);
+        if (!best || cost < best_cost) { best = bn; best_cost = cost; }
+    }
+    return best == 64 ? launch_tc<64>(P, st) : best == 128 ? launch_tc<128>(P, st) : launch_tc<256>(P, st);
 }
 
 int launch_dense_tc_grouped(const __nv_bfloat16 * A, int64_t lda, const __nv_bfloat16 * W, int64_t ldw, int64_t w_stride, float * C, int64_t ldc,
                             const int32_t * start, const int32_t * count, int groups, int max_rows, int N, int K, cudaStream_t st) {
     if (groups <= 0 || max_rows <= 0) return 0;
     // T bounds the grid only (all groups together hold max_rows rows); the kernel reads each group's own count
-    TcParams P{A, lda, W, ldw, C, ldc, nullptr, nullptr, 0, 1.f, max_rows, N, K, abort_flag(), start, count, w_stride, groups, 0, 0};
+    TcParams P{A, lda, W, ldw, C, ldc, nullptr, nullptr, 0, 1.f, max_rows, N, K, abort_flag(), start, count, w_stride, groups, 0, 0, DenseAct()};
     const int avg = (max_rows + groups - 1) / groups;   // the token tile follows the expected rows of a group
     return avg <= 64 ? launch_tc<64>(P, st) : avg <= 128 ? launch_tc<128>(P, st) : launch_tc<256>(P, st);
 }

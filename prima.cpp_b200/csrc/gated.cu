@@ -10,11 +10,16 @@
 #include <math.h>
 
 #include <algorithm>
+#include <cstdlib>
 
 #include "layers.h"
 #include "mixers.cuh"
 
 namespace pb {
+
+int wkv_scan_ok(const GatedLinIO & io, const GatedLinParams & p);   // wkv.cu
+int launch_wkv_scan(const GatedLinIO & io, const BatchView & b, const GatedLinParams & p, float * state, int64_t slot_stride, float * y, cudaStream_t st);
+
 namespace {
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -713,6 +718,8 @@ int launch_gated_linattn(const GatedLinIO & io, const BatchView & b, const Gated
         (p.tied_key && (!p.decay_per_channel || p.delta)) || (!p.tied_key && !io.k) || (p.decay_per_channel && !p.tied_key && !p.bonus) ||
         (p.bonus && (!p.decay_per_channel || p.delta || p.tied_key || !io.bonus)))
         return (int) cudaErrorInvalidValue;
+    static const bool plain_wkv = getenv("PB200_WKV_PLAIN") != nullptr;   // A/B and tests: the shared kernels below for the bonus form too
+    if (p.bonus && !plain_wkv && wkv_scan_ok(io, p)) return launch_wkv_scan(io, b, p, state, slot_stride, y, st);
     // the register kernels: delta rule with one decay per head, tied key with a decay per channel, bonus form with a decay per channel
     if (p.dim <= 256 && ((p.delta && !p.decay_per_channel) || (p.tied_key && !p.delta) || p.bonus)) {
         const int ln = p.dim <= 32 ? 8 : p.dim <= 64 ? 16 : 32;

@@ -178,17 +178,25 @@ __global__ void __launch_bounds__(256) k_latent_up_v(const float * __restrict__ 
 // value is the row's latent part) -- a row is read once for all heads of the group.  Partial (sum, max, normaliser) per split go to
 // `part` [entry][split][head][kv_rank + 2]; k_latent_merge_up_v combines them.  The share of a split depends on the sequence's own
 // length only, so a token's result does not depend on the batch around it.
+// VEC: rows whose size is a multiple of 4 travel and are scored in 16-byte pieces (the padded row stride is an odd number of pieces: no bank
+// conflicts between the 16 rows a warp scores).
 constexpr int LT_ROWS = 16, LT_HEADS = 16;
+__host__ __device__ inline bool latent_vec(const LatentParams & p) { return p.kv_rank % 4 == 0 && p.rot_dim % 4 == 0; }
+__host__ __device__ inline int latent_row_stride(const LatentParams & p) {
+    const int RW = p.kv_rank + p.rot_dim;
+    return latent_vec(p) ? (RW / 4 | 1) * 4 : RW | 1;
+}
+template <bool VEC>
 __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __restrict__ qa, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
                                                              const int32_t * __restrict__ pos0, LatentParams p, const float * __restrict__ cache,
                                                              int64_t slot_stride, int splits, float * __restrict__ part) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     const int s = blockIdx.x, e = blockIdx.y, h0 = blockIdx.z * LT_HEADS;
-    const int H = p.heads, R = p.kv_rank, RW = R + p.rot_dim, RWP = RW | 1;
+    const int H = p.heads, R = p.kv_rank, RW = R + p.rot_dim, RWP = latent_row_stride(p);
     const int nh = min(LT_HEADS, H - h0);
     float * tile = sm;                        // [LT_ROWS][RWP]
     float * qs = tile + LT_ROWS * RWP;        // [LT_HEADS][RW]
-    float * P = qs + LT_HEADS * RW;           // [LT_HEADS][LT_ROWS]
+    float * P = qs + LT_HEADS * RW;           // [LT_ROWS][LT_HEADS]
     float * mrun = P + LT_HEADS * LT_ROWS;    // [LT_HEADS] running max, then running sum, then this tile's factor on what was gathered before
     float * lrun = mrun + LT_HEADS;
     float * corr = lrun + LT_HEADS;
@@ -197,7 +205,14 @@ __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __res
     const int per = ((rows_used + splits - 1) / splits + LT_ROWS - 1) / LT_ROWS * LT_ROWS;
     const int r_lo = s * per, r_hi = min(rows_used, r_lo + per);
     const float * qrow = qa + ((int64_t) off[e] * H + h0) * RW;
-    for (int i0 = tid; i0 < nh * RW; i0 += 256 * 8) {   // eight loads in flight per thread
+    if constexpr (VEC) {
+        const float4 * q4 = reinterpret_cast<const float4 *>(qrow);
+#pragma unroll 4
+        for (int i = tid; i < nh * RW / 4; i += 256) {
+            const float4 v = q4[i];
+            reinterpret_cast<float4 *>(qs)[i] = make_float4(v.x * p.scale, v.y * p.scale, v.z * p.scale, v.w * p.scale);
+        }
+    } else for (int i0 = tid; i0 < nh * RW; i0 += 256 * 8) {   // eight loads in flight per thread
         float v[8];
 #pragma unroll
         for (int u = 0; u < 8; u++) { const int i = i0 + 256 * u; v[u] = i < nh * RW ? qrow[i] : 0.f; }
@@ -213,7 +228,20 @@ __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __res
     for (int r0 = r_lo; r0 < r_hi; r0 += LT_ROWS) {
         const int nr = min(LT_ROWS, r_hi - r0);
         __syncthreads();
-        {   // the tile's rows are one contiguous piece of the cache: eight loads per thread in flight before the first store
+        if constexpr (VEC) {
+            const float4 * src = reinterpret_cast<const float4 *>(crow + (int64_t) r0 * RW);
+            const int RQ = RW / 4, n_src = nr * RQ, n_all = LT_ROWS * RQ;
+            for (int i0 = tid; i0 < n_all; i0 += 256 * 4) {
+                float4 v[4];
+#pragma unroll
+                for (int u = 0; u < 4; u++) { const int i = i0 + 256 * u; v[u] = i < n_src ? src[i] : make_float4(0.f, 0.f, 0.f, 0.f); }
+#pragma unroll
+                for (int u = 0; u < 4; u++) {
+                    const int i = i0 + 256 * u;
+                    if (i < n_all) { const int rr = i / RQ; *reinterpret_cast<float4 *>(tile + rr * RWP + 4 * (i - rr * RQ)) = v[u]; }
+                }
+            }
+        } else {   // the tile's rows are one contiguous piece of the cache: eight loads per thread in flight before the first store
             const float * src = crow + (int64_t) r0 * RW;
             const int n_src = nr * RW, n_all = LT_ROWS * RW;
             for (int i0 = tid; i0 < n_all; i0 += 256 * 8) {
@@ -233,7 +261,13 @@ __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __res
             const float * q = qs + hl * RW, * k = tile + r * RWP;
             float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
             int d = 0;
-            for (; d + 3 < RW; d += 4) {
+            if constexpr (VEC) {
+#pragma unroll 4
+                for (; d < RW; d += 4) {
+                    const float4 qv = *reinterpret_cast<const float4 *>(q + d), kv = *reinterpret_cast<const float4 *>(k + d);
+                    a0 = fmaf(qv.x, kv.x, a0); a1 = fmaf(qv.y, kv.y, a1); a2 = fmaf(qv.z, kv.z, a2); a3 = fmaf(qv.w, kv.w, a3);
+                }
+            } else for (; d + 3 < RW; d += 4) {
                 a0 = fmaf(q[d], k[d], a0); a1 = fmaf(q[d + 1], k[d + 1], a1);
                 a2 = fmaf(q[d + 2], k[d + 2], a2); a3 = fmaf(q[d + 3], k[d + 3], a3);
             }
@@ -249,7 +283,7 @@ __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __res
         float ps = pv;
 #pragma unroll
         for (int o = 8; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
-        P[hl * LT_ROWS + r] = pv;
+        P[r * LT_HEADS + hl] = pv;
         __syncwarp();
         if (r == 0) {
             const float c = mn == -INFINITY ? 1.f : (mo == -INFINITY ? 0.f : expf(mo - mn));
@@ -263,10 +297,12 @@ __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __res
         for (int rr = 0; rr < nr; rr++) {
             const float v0 = c0ok ? tile[rr * RWP + tid] : 0.f, v1 = c1ok ? tile[rr * RWP + tid + 256] : 0.f;
 #pragma unroll
-            for (int h = 0; h < LT_HEADS; h++) {
-                const float pw = P[h * LT_ROWS + rr];
-                acc[h][0] = fmaf(pw, v0, acc[h][0]);
-                acc[h][1] = fmaf(pw, v1, acc[h][1]);
+            for (int h = 0; h < LT_HEADS; h += 4) {
+                const float4 pw = *reinterpret_cast<const float4 *>(P + rr * LT_HEADS + h);
+                acc[h][0] = fmaf(pw.x, v0, acc[h][0]); acc[h][1] = fmaf(pw.x, v1, acc[h][1]);
+                acc[h + 1][0] = fmaf(pw.y, v0, acc[h + 1][0]); acc[h + 1][1] = fmaf(pw.y, v1, acc[h + 1][1]);
+                acc[h + 2][0] = fmaf(pw.z, v0, acc[h + 2][0]); acc[h + 2][1] = fmaf(pw.z, v1, acc[h + 2][1]);
+                acc[h + 3][0] = fmaf(pw.w, v0, acc[h + 3][0]); acc[h + 3][1] = fmaf(pw.w, v1, acc[h + 3][1]);
             }
         }
     }
@@ -397,11 +433,15 @@ int launch_latent_decode(const float * qa, const BatchView & b, const LatentPara
     if (b.n_entries <= 0) return 0;
     if (!latent_ok(p) || p.kv_rank > 512 || splits < 1 || splits > 64 || !part || b.n_tokens != b.n_entries) return (int) cudaErrorInvalidValue;
     const int RW = latent_row(p);
-    const size_t smem = ((size_t) LT_ROWS * (RW | 1) + (size_t) LT_HEADS * RW + LT_HEADS * LT_ROWS + 3 * LT_HEADS) * sizeof(float);
-    int rc = raise_smem(k_latent_decode_split, smem);
+    const size_t smem = ((size_t) LT_ROWS * latent_row_stride(p) + (size_t) LT_HEADS * RW + LT_HEADS * LT_ROWS + 3 * LT_HEADS) * sizeof(float);
+    const bool vec = latent_vec(p) && slot_stride % 4 == 0 && ((uintptr_t) cache & 15) == 0 && ((uintptr_t) qa & 15) == 0;
+    int rc = vec ? raise_smem(k_latent_decode_split<true>, smem) : raise_smem(k_latent_decode_split<false>, smem);
     if (rc) return rc;
     const dim3 grid((unsigned) splits, (unsigned) b.n_entries, (unsigned) ((p.heads + LT_HEADS - 1) / LT_HEADS));
-    rc = ck_launch([&] { k_latent_decode_split<<<grid, 256, smem, st>>>(qa, b.slot, b.off, b.pos0, p, cache, slot_stride, splits, part); });
+    rc = ck_launch([&] {
+        if (vec) k_latent_decode_split<true><<<grid, 256, smem, st>>>(qa, b.slot, b.off, b.pos0, p, cache, slot_stride, splits, part);
+        else k_latent_decode_split<false><<<grid, 256, smem, st>>>(qa, b.slot, b.off, b.pos0, p, cache, slot_stride, splits, part);
+    });
     if (rc) return rc;
     const dim3 grid2((unsigned) p.heads, (unsigned) b.n_entries, 2);
     const size_t smem2 = ((size_t) p.kv_rank + 64) * sizeof(float);

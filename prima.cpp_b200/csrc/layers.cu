@@ -2026,11 +2026,19 @@ static int ff_xielu(pb200_model * m, int T, LLayer & L, float * x) {
     LayerList & ll = *m->ll;
     cudaStream_t st = m->stream;
     const int W = ll.width, ct = ll.ctype, ff = L.ff;
+    // the activation is the up product's epilogue (PB200_FF_UNFUSED: a kernel of its own, as the layers were brought up; for A/B runs and tests)
+    static const bool unfused = getenv("PB200_FF_UNFUSED") != nullptr;
     CAT(CAT_DENSE);
-    CK(launch_dense(ct, ll.act, W, L.gateup.data, W, ll.big, ff, T, ff, W, nullptr, nullptr, 0, 1.f, st));
-    CAT(CAT_ELEM);
-    CK(launch_xielu(ll.big, L.ff_act.data, ll.act2, ct, (int64_t) T * ff, st));
-    CAT(CAT_DENSE);
+    if (unfused) {
+        CK(launch_dense(ct, ll.act, W, L.gateup.data, W, ll.big, ff, T, ff, W, nullptr, nullptr, 0, 1.f, st));
+        CAT(CAT_ELEM);
+        CK(launch_xielu(ll.big, L.ff_act.data, ll.act2, ct, (int64_t) T * ff, st));
+        CAT(CAT_DENSE);
+    } else {
+        DenseAct act;
+        act.xielu = L.ff_act.data; act.y = ll.act2; act.ldy = ff;
+        CK(launch_dense_act(ct, ll.act, W, L.gateup.data, W, act, T, ff, W, st));
+    }
     return launch_dense(ct, ll.act2, ff, L.down.data, ff, x, W, T, W, ff, nullptr, x, W, 1.f, st);
 }
 // ---- mixture of experts over ll.act.  accumulate: x[t] += shared(h) + sum_k w_k expert_k(h) (the stream itself); otherwise x receives the

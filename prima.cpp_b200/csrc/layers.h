@@ -44,6 +44,14 @@ int launch_dense(int type, const void * A, int64_t lda, const void * W, int64_t 
 // each) into the same rows of C, g < groups; start / count are device arrays and no group has more than max_rows rows.  Tensor-core
 // kernel only (bf16, aligned shapes): dense_grouped_ok says whether it applies; otherwise the caller multiplies group by group.
 int dense_grouped_ok(int type, int N, int K, int64_t lda, int64_t ldw, int64_t w_stride, const void * A, const void * W);
+// Epilogue of a product that feeds another one through xIELU: instead of C[t][n], y[t * ldy + n] = xielu(C[t][n]) in the operand type, with the
+// activation's two numbers at xielu (device).
+struct DenseAct {
+    const float * xielu = nullptr;
+    void * y = nullptr;
+    int64_t ldy = 0;
+};
+int launch_dense_act(int type, const void * A, int64_t lda, const void * W, int64_t ldw, const DenseAct & act, int T, int N, int K, cudaStream_t stream);
 // Several products of one shape over operands of their own, side by side: C[t][p * N + n] = sum_k A[p * a_plane + t * lda + k] * W[p * N + n][k],
 // p < planes (W: one [planes * N][K] matrix).
 int launch_dense_planes(int type, const void * A, int64_t a_plane, int64_t lda, const void * W, int64_t ldw, float * C, int64_t ldc, int planes, int T, int N,

@@ -134,14 +134,11 @@ __global__ void k_relu2(const float * __restrict__ u, OT * __restrict__ y, int64
     const float v = fmaxf(u[i], 0.f);
     put(y, i, v * v);
 }
-__device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 template <typename OT>
 __global__ void k_xielu(const float * __restrict__ u, const float * __restrict__ pq, OT * __restrict__ y, int64_t n) {
     const int64_t i = (int64_t) blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
-    const float z = u[i];
-    const float v = z > 0.f ? softplus_f(pq[0]) * z * z : (0.5f + softplus_f(pq[1])) * (expm1f(z) - z);
-    put(y, i, v + 0.5f * z);
+    put(y, i, xielu_f(u[i], softplus_f(pq[0]), 0.5f + softplus_f(pq[1])));
 }
 __global__ void k_softcap(float * __restrict__ x, int64_t n, float cap) {
     const int64_t i = (int64_t) blockIdx.x * blockDim.x + threadIdx.x;

@@ -42,6 +42,10 @@ __device__ __forceinline__ float block_sum(float v, float * red) {
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
 
+__device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log1pf(expf(v)); }
+// xIELU with its two numbers already through softplus: pos = softplus(p), neg = 1/2 + softplus(q)
+__device__ __forceinline__ float xielu_f(float z, float pos, float neg) { return (z > 0.f ? pos * z * z : neg * (expm1f(z) - z)) + 0.5f * z; }
+
 __device__ __forceinline__ float ld_f(const float * p, int64_t i) { return p[i]; }
 __device__ __forceinline__ float ld_f(const __nv_bfloat16 * p, int64_t i) { return __bfloat162float(p[i]); }
 
