@@ -445,6 +445,9 @@ ODD = {   # configuration, inner size of the decay's map
     "many_heads": lambda: (config([att(heads=20, kv_heads=4, dim=8, vdim=8, chunk=16, rot=4), lat(heads=35, dim=4, rot_dim=4, vdim=4, kv_rank=16), wkv(heads=17, dim=8)], vocab=31), 130),
     "tensor_core_shapes": lambda: (config([att(heads=4, kv_heads=2, dim=32, vdim=32, chunk=24, rot=32, ff=256), wkv(heads=4, dim=32, ff=128),
                                            lat(heads=4, dim=32, rot_dim=16, vdim=32, kv_rank=64, ff=128), again(wkv(heads=4, dim=32, ff=128), 1)], width=128, vocab=128), 24),
+    "state_of_64": lambda: (config([wkv(heads=3, dim=64), wkv(heads=1, dim=64)], vocab=31), 8),
+    "state_of_128": lambda: (config([wkv(heads=2, dim=128)], vocab=31), 12),
+    "state_of_256": lambda: (config([wkv(heads=1, dim=256)], vocab=31), 8),
     "state_in_shared_memory": lambda: (config([wkv(heads=2, dim=264)], vocab=31), 3),
     "chunk_longer_than_the_context": lambda: (config([att(chunk=100000), lat()]), 8),
     "kv_heads_not_given": lambda: (config([{"type": "attention", "mlp": None, "mixer": {"heads": 3, "dim": 8, "scale": 0.3, "softcap": 9.0, "mask": {"size": 9}, "rot": {"base": 50.0, "dims": 4}}}]), 8),
@@ -462,6 +465,42 @@ def test_other_sizes(pkg, cuda, which, dtype, tol):
     check(run_whole(m, toks), want, tol)
     check(run_decoded(m, toks, 20), want, tol)
     m.close()
+
+
+@pytest.mark.parametrize("dim", [32, 64, 128, 256])
+def test_recurrence_across_its_chunks(pkg, cuda, dim):
+    # the recurrence takes 16 tokens at a time: whole chunks, a rest of every kind, cuts inside a chunk, and several entries at once
+    cfg = config([wkv(heads=2, dim=dim, ff=0)], width=32, vocab=31)
+    bits, W = R.random_weights(cfg, seed=28)
+    m = load(pkg, cfg, bits, n_seq=6)
+    reqs = [tokens_for(cfg, n, n) for n in (48, 31, 17, 1, 65)]
+    wants = [R.forward(cfg, W, r)[0] for r in reqs]
+    slots = [m.seq_alloc() for _ in reqs]
+    lg, _ = m.batch_step([(s, r, list(range(len(r)))) for s, r in zip(slots, reqs)])
+    at = 0
+    for r, w in zip(reqs, wants):
+        check(lg[at:at + len(r)], w, F32_TOL)
+        at += len(r)
+    for s in slots:
+        m.seq_free(s)
+    for first in (16, 33, 40):
+        check(run_decoded(m, reqs[0], first), wants[0], F32_TOL)
+    m.close()
+
+
+def test_a_prompt_of_more_than_a_thousand_tokens(pkg, cuda):
+    # wide token tiles everywhere; two requests, the shorter one ends inside a tile
+    cfg = config([wkv(heads=2, dim=32, ff=64), att(heads=2, kv_heads=1, dim=16, vdim=16, chunk=300, rot=16, ff=0), lat(heads=2, dim=16, rot_dim=8, vdim=16, ff=64)], width=64, vocab=53)
+    bits, W = R.random_weights(cfg, seed=29)
+    a, b = tokens_for(cfg, 1100, 1), tokens_for(cfg, 333, 2)
+    wa, wb = R.forward(cfg, W, a)[0], R.forward(cfg, W, b)[0]
+    for dtype, tol in (("float32", F32_TOL), ("bfloat16", BF16_TOL)):
+        m = load(pkg, cfg, bits, dtype, n_ctx=1200, n_seq=2)
+        s, t = m.seq_alloc(), m.seq_alloc()
+        lg, _ = m.batch_step([(s, a, list(range(1100))), (t, b, list(range(333)))])
+        check(lg[:1100], wa, tol)
+        check(lg[1100:], wb, tol)
+        m.close()
 
 
 def test_tensors_arrive_in_any_order(pkg, cuda):
@@ -541,3 +580,33 @@ def test_directory_loader_and_command_line(pkg, cuda, tmp_path):
                         ",".join(map(str, b)), "--max-new", "5", "--n-ctx", "64"], capture_output=True, text=True, timeout=600)
     assert p.returncode == 0, p.stderr[-2000:]
     assert [[int(t) for t in line.split(",")] for line in p.stdout.split()] == mine
+
+
+def test_fused_and_single_step_kernels_agree(pkg, cuda, tmp_path):
+    # the recurrence's own kernel against the one every gated recurrence shares (PB200_WKV_PLAIN), xIELU in the up product's epilogue against a
+    # kernel of its own (PB200_FF_UNFUSED), through the command-line replay: a prompt of two requests, then decoded tokens
+    cfg = config([wkv(heads=2, dim=32, ff=72), lat(ff=33), wkv(heads=1, dim=64, ff=40)])
+    bits, W = R.random_weights(cfg, seed=22)
+    d = tmp_path / "model"
+    R.write_model_dir(str(d), cfg, bits, R.tensor_shapes(cfg))
+    a, b = tokens_for(cfg, 40, 6), tokens_for(cfg, 9, 7)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:36], "want": list(range(36))}, {"id": "b", "tokens": b[:5], "want": [0, 4]}], "end": []}]
+    for k in range(4):
+        steps.append({"step": k + 1, "entries": [{"id": "a", "tokens": [a[36 + k]], "want": [0]}, {"id": "b", "tokens": [b[5 + k]], "want": [0]}], "end": ["a", "b"] if k == 3 else []})
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    rows = {}
+    for mode in ("fused", "single"):
+        env = {k: v for k, v in os.environ.items() if k not in ("PB200_WKV_PLAIN", "PB200_FF_UNFUSED")}
+        if mode == "single":
+            env["PB200_WKV_PLAIN"] = env["PB200_FF_UNFUSED"] = "1"
+        out = tmp_path / mode
+        p = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", str(d), "--dtype", "float32", "--out", str(out), "--max-tokens", "64"],
+                           input="\n".join(json.dumps(s) for s in steps) + "\n", capture_output=True, text=True, timeout=600, env=env)
+        assert p.returncode == 0, p.stderr[-2000:]
+        rows[mode] = np.concatenate([np.fromfile(out / f"{k}.f32", dtype="<f4").reshape(-1, cfg["vocab"]) for k in range(5)])
+    wa, _ = R.forward(cfg, W, a)
+    wb, _ = R.forward(cfg, W, b)
+    want = np.concatenate([wa[:36], wb[[0, 4]]] + [np.stack([wa[36 + k], wb[5 + k]]) for k in range(4)])
+    check(rows["fused"], want, F32_TOL)
+    check(rows["single"], want, F32_TOL)
+    assert np.abs(rows["fused"] - rows["single"]).max() < 2e-5 * np.abs(want).max()
