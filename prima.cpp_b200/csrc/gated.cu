@@ -197,7 +197,7 @@ __device__ __forceinline__ void hgrn2_prep_rows(float * qr, float * fr, const fl
 // One CTA per token prepares everything the token's branches need before their kernels.  With `staged` the token's q, k, v rows (and the
 // recurrence's q and k rows) are copied into shared memory once, every step runs there, and the rows go back to global memory (and the
 // K / V rows later tokens can still see to the cache) once: two passes over global memory instead of one per step.
-__global__ void __launch_bounds__(256) k_dual_prep_store(RecPrep rc, float * __restrict__ q, int64_t ldq, float * __restrict__ k, int64_t ldk,
+__global__ void __launch_bounds__(1024) k_dual_prep_store(RecPrep rc, float * __restrict__ q, int64_t ldq, float * __restrict__ k, int64_t ldk,
                                                          float * __restrict__ v, int64_t ldv, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
                                                          const int32_t * __restrict__ pos0, const int32_t * __restrict__ entry_of, AttnParams a, AttnPrep pr,
                                                          float * __restrict__ kcache, float * __restrict__ vcache, int64_t slot_stride, int staged) {
@@ -676,7 +676,7 @@ static int dual_prep_launch(const RecPrep & rc, float * q, int64_t ldq, float * 
     int e = raise_smem(k_dual_prep_store, smem);
     if (e) return e;
     return ck_launch([&] {
-        k_dual_prep_store<<<b.n_tokens, 256, smem, st>>>(rc, q, ldq, k, ldk, v, ldv, b.slot, b.off, b.pos0, b.entry_of, a, pr, kcache, vcache, slot_stride, staged);
+        k_dual_prep_store<<<b.n_tokens, row_threads(b.n_tokens, (int) floats / 2), smem, st>>>(rc, q, ldq, k, ldk, v, ldv, b.slot, b.off, b.pos0, b.entry_of, a, pr, kcache, vcache, slot_stride, staged);
     });
 }
 int launch_attn_prep_store(float * q, int64_t ldq, float * k, int64_t ldk, float * v, int64_t ldv, const BatchView & b, const AttnParams & a,

@@ -8,6 +8,8 @@
 #include <cuda_runtime.h>
 #include <math.h>
 
+#include <algorithm>
+
 #include "layers.h"
 #include "mixers.cuh"
 
@@ -110,13 +112,14 @@ __global__ void k_latent_gather(const float * __restrict__ cache, int64_t slot_s
     for (int i = threadIdx.x; i < Dr; i += blockDim.x) kr[(int64_t) t * Dr + i] = crow[R + i];
 }
 
-// CTA (head, token, 128 latent entries): qa[r] = sum_d W_uk[h * dim + d][r] q[d]; thread r walks a column of the head's block (coalesced
-// over r, eight loads in flight)
+// CTA (head, token, 128 latent entries): qa[r] = sum_d W_uk[h * dim + d][r] q[d]; four groups of 128 threads walk a quarter of the head's rows
+// each (coalesced over r, eight loads in flight); the quarters are summed in order
 template <typename WT>
-__global__ void __launch_bounds__(128) k_latent_absorb_q(const float * __restrict__ q, int64_t ldq, const int32_t * __restrict__ off, const int32_t * __restrict__ pos0,
+__global__ void __launch_bounds__(512) k_latent_absorb_q(const float * __restrict__ q, int64_t ldq, const int32_t * __restrict__ off, const int32_t * __restrict__ pos0,
                                                          const int32_t * __restrict__ entry_of, const WT * __restrict__ wuk, LatentParams p,
                                                          const float * __restrict__ freq, float * __restrict__ qa) {
     extern __shared__ float qs[];   // [dim]
+    __shared__ float quarter[4][128];
     const int h = blockIdx.x, t = blockIdx.y;
     const int D = p.dim, Dr = p.rot_dim, R = p.kv_rank;
     const float * qr = q + (int64_t) t * ldq + (int64_t) h * (D + Dr);
@@ -124,20 +127,23 @@ __global__ void __launch_bounds__(128) k_latent_absorb_q(const float * __restric
     __syncthreads();
     float * out = qa + ((int64_t) t * p.heads + h) * (R + Dr);
     const WT * w = wuk + (int64_t) h * D * R;
-    const int r = blockIdx.z * 128 + threadIdx.x;
+    const int grp = threadIdx.x >> 7, r = blockIdx.z * 128 + (threadIdx.x & 127);
+    const int per = (D + 3) / 4, d_end = min(D, (grp + 1) * per);
+    float acc = 0.f;
     if (r < R) {
-        float acc = 0.f;
-        int d = 0;
-        for (; d + 7 < D; d += 8) {
+        int d = grp * per;
+        for (; d + 7 < d_end; d += 8) {
             float wv[8];
 #pragma unroll
             for (int u = 0; u < 8; u++) wv[u] = ld_f(w, (int64_t) (d + u) * R + r);
 #pragma unroll
             for (int u = 0; u < 8; u++) acc = fmaf(wv[u], qs[d + u], acc);
         }
-        for (; d < D; d++) acc = fmaf(ld_f(w, (int64_t) d * R + r), qs[d], acc);
-        out[r] = acc;
+        for (; d < d_end; d++) acc = fmaf(ld_f(w, (int64_t) d * R + r), qs[d], acc);
     }
+    quarter[grp][threadIdx.x & 127] = acc;
+    __syncthreads();
+    if (grp == 0 && r < R) out[r] = (quarter[0][threadIdx.x] + quarter[1][threadIdx.x]) + (quarter[2][threadIdx.x] + quarter[3][threadIdx.x]);
     if (blockIdx.z == 0) {   // the rotated part, turned here by the token's position
         const int e = entry_of[t], pos = pos0[e] + (t - off[e]), half = p.rot_dims / 2;
         for (int i = threadIdx.x; i < Dr; i += blockDim.x) {
@@ -186,6 +192,7 @@ __host__ __device__ inline int latent_row_stride(const LatentParams & p) {
     const int RW = p.kv_rank + p.rot_dim;
     return latent_vec(p) ? (RW / 4 | 1) * 4 : RW | 1;
 }
+__device__ __forceinline__ int latent_rows_per_split(int rows_used, int splits) { return ((rows_used + splits - 1) / splits + LT_ROWS - 1) / LT_ROWS * LT_ROWS; }
 template <bool VEC>
 __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __restrict__ qa, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
                                                              const int32_t * __restrict__ pos0, LatentParams p, const float * __restrict__ cache,
@@ -202,8 +209,9 @@ __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __res
     float * corr = lrun + LT_HEADS;
     const int tid = threadIdx.x, hl = tid >> 4, r = tid & 15;
     const int rows_used = pos0[e] + 1;        // the token's own row is in the cache already
-    const int per = ((rows_used + splits - 1) / splits + LT_ROWS - 1) / LT_ROWS * LT_ROWS;
+    const int per = latent_rows_per_split(rows_used, splits);
     const int r_lo = s * per, r_hi = min(rows_used, r_lo + per);
+    if (r_lo >= rows_used) return;            // no rows left for this split: the merge does not read it
     const float * qrow = qa + ((int64_t) off[e] * H + h0) * RW;
     if constexpr (VEC) {
         const float4 * q4 = reinterpret_cast<const float4 *>(qrow);
@@ -318,18 +326,20 @@ __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __res
     if (tid < nh) { pp[(int64_t) tid * (R + 2) + R] = mrun[tid]; pp[(int64_t) tid * (R + 2) + R + 1] = lrun[tid]; }
 }
 
-// CTA (head, entry, half of the value rows): the splits' partial sums become the weighted sum of latents (both halves compute it), then
+// CTA (head, entry, share of the value rows): the splits' partial sums become the weighted sum of latents (every share computes it), then
 // a warp per output row of the head's block of W_uv (lanes split the latent) and the output gate.  Up to 64 splits: a lane of warp 0
 // weighs splits lane and lane + 32.
 template <typename WT, typename OT>
-__global__ void __launch_bounds__(256) k_latent_merge_up_v(const float * __restrict__ part, int splits, const int32_t * __restrict__ off, const WT * __restrict__ wuv,
+__global__ void __launch_bounds__(256) k_latent_merge_up_v(const float * __restrict__ part, int all_splits, const int32_t * __restrict__ off,
+                                                           const int32_t * __restrict__ pos0, const WT * __restrict__ wuv,
                                                            LatentParams p, const float * __restrict__ sink, const float * __restrict__ gate, int64_t ldg,
                                                            OT * __restrict__ out) {
     extern __shared__ float os[];   // [kv_rank], then [64] weights of the splits
     const int h = blockIdx.x, e = blockIdx.y, t = off[e];
     const int R = p.kv_rank, DV = p.vdim, H = p.heads;
     float * w = os + R;
-    const float * pe = part + ((int64_t) e * splits * H + h) * (R + 2);
+    const float * pe = part + ((int64_t) e * all_splits * H + h) * (R + 2);
+    const int rows_used = pos0[e] + 1, per = latent_rows_per_split(rows_used, all_splits), splits = (rows_used + per - 1) / per;   // the rest hold no rows
     const int64_t stride = (int64_t) H * (R + 2);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (warp == 0) {
@@ -358,7 +368,7 @@ __global__ void __launch_bounds__(256) k_latent_merge_up_v(const float * __restr
         os[r] = a;
     }
     __syncthreads();
-    const int dv_lo = blockIdx.z * ((DV + 1) / 2), dv_hi = min(DV, dv_lo + (DV + 1) / 2);
+    const int share = (DV + gridDim.z - 1) / gridDim.z, dv_lo = blockIdx.z * share, dv_hi = min(DV, dv_lo + share);
     for (int dv = dv_lo + warp; dv < dv_hi; dv += (int) (blockDim.x >> 5)) {
         const float acc = wsum(dot_lane8(wuv + ((int64_t) h * DV + dv) * R, os, R, lane));
         if (lane == 0) put(out, (int64_t) t * H * DV + h * DV + dv, gate ? acc * sigmoid_f(gate[(int64_t) t * ldg + h * DV + dv]) : acc);
@@ -407,8 +417,8 @@ int launch_latent_absorb_q(const float * q, int64_t ldq, const BatchView & b, co
     const dim3 grid((unsigned) p.heads, (unsigned) n_tokens, (unsigned) ((p.kv_rank + 127) / 128));
     const size_t smem = (size_t) p.dim * sizeof(float);
     return ck_launch([&] {
-        if (wtype == T_BF16) k_latent_absorb_q<__nv_bfloat16><<<grid, 128, smem, st>>>(q, ldq, b.off, b.pos0, b.entry_of, (const __nv_bfloat16 *) wuk, p, freq, qa);
-        else k_latent_absorb_q<float><<<grid, 128, smem, st>>>(q, ldq, b.off, b.pos0, b.entry_of, (const float *) wuk, p, freq, qa);
+        if (wtype == T_BF16) k_latent_absorb_q<__nv_bfloat16><<<grid, 512, smem, st>>>(q, ldq, b.off, b.pos0, b.entry_of, (const __nv_bfloat16 *) wuk, p, freq, qa);
+        else k_latent_absorb_q<float><<<grid, 512, smem, st>>>(q, ldq, b.off, b.pos0, b.entry_of, (const float *) wuk, p, freq, qa);
     });
 }
 int launch_latent_up_v(const float * olat, const void * wuv, int wtype, const LatentParams & p, const float * gate, int64_t ldg, void * out, int otype,
@@ -443,15 +453,17 @@ int launch_latent_decode(const float * qa, const BatchView & b, const LatentPara
         else k_latent_decode_split<false><<<grid, 256, smem, st>>>(qa, b.slot, b.off, b.pos0, p, cache, slot_stride, splits, part);
     });
     if (rc) return rc;
-    const dim3 grid2((unsigned) p.heads, (unsigned) b.n_entries, 2);
+    // shares: enough CTAs for the machine when heads and entries are few (an output row is the same sum under any number of them)
+    const int shares = std::max(2, std::min(std::min(8, (p.vdim + 7) / 8), 296 / (p.heads * b.n_entries)));
+    const dim3 grid2((unsigned) p.heads, (unsigned) b.n_entries, (unsigned) shares);
     const size_t smem2 = ((size_t) p.kv_rank + 64) * sizeof(float);
     return ck_launch([&] {
         if (wtype == T_BF16) {
-            if (otype == T_BF16) k_latent_merge_up_v<__nv_bfloat16, __nv_bfloat16><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const __nv_bfloat16 *) wuv, p, sink, gate, ldg, (__nv_bfloat16 *) out);
-            else k_latent_merge_up_v<__nv_bfloat16, float><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const __nv_bfloat16 *) wuv, p, sink, gate, ldg, (float *) out);
+            if (otype == T_BF16) k_latent_merge_up_v<__nv_bfloat16, __nv_bfloat16><<<grid2, 256, smem2, st>>>(part, splits, b.off, b.pos0, (const __nv_bfloat16 *) wuv, p, sink, gate, ldg, (__nv_bfloat16 *) out);
+            else k_latent_merge_up_v<__nv_bfloat16, float><<<grid2, 256, smem2, st>>>(part, splits, b.off, b.pos0, (const __nv_bfloat16 *) wuv, p, sink, gate, ldg, (float *) out);
         } else {
-            if (otype == T_BF16) k_latent_merge_up_v<float, __nv_bfloat16><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const float *) wuv, p, sink, gate, ldg, (__nv_bfloat16 *) out);
-            else k_latent_merge_up_v<float, float><<<grid2, 256, smem2, st>>>(part, splits, b.off, (const float *) wuv, p, sink, gate, ldg, (float *) out);
+            if (otype == T_BF16) k_latent_merge_up_v<float, __nv_bfloat16><<<grid2, 256, smem2, st>>>(part, splits, b.off, b.pos0, (const float *) wuv, p, sink, gate, ldg, (__nv_bfloat16 *) out);
+            else k_latent_merge_up_v<float, float><<<grid2, 256, smem2, st>>>(part, splits, b.off, b.pos0, (const float *) wuv, p, sink, gate, ldg, (float *) out);
         }
     });
 }

@@ -30,7 +30,7 @@ __global__ void k_embed(const WT * __restrict__ table, int width, const int32_t 
 
 // one CTA per token: the table row normed, and (y given) normed again for the first layer; every thread re-reads only what it has written itself
 template <typename WT, typename OT>
-__global__ void __launch_bounds__(256) k_embed_rmsnorm(const WT * __restrict__ table, int width, const int32_t * __restrict__ tokens, const float * __restrict__ w,
+__global__ void __launch_bounds__(1024) k_embed_rmsnorm(const WT * __restrict__ table, int width, const int32_t * __restrict__ tokens, const float * __restrict__ w,
                                                        float eps, float * __restrict__ x, const float * __restrict__ wn, OT * __restrict__ y) {
     __shared__ float red[33];
     const int t = blockIdx.x;
@@ -871,8 +871,8 @@ int launch_embed_rmsnorm(const void * table, int type, int width, const int32_t 
     if (!w || (y && (!wn || otype != type))) return (int) cudaErrorInvalidValue;
     return ck_launch([&] {
         if (type == T_BF16)
-            k_embed_rmsnorm<__nv_bfloat16, __nv_bfloat16><<<n_tokens, 256, 0, st>>>((const __nv_bfloat16 *) table, width, tokens, w, eps, x, wn, (__nv_bfloat16 *) y);
-        else k_embed_rmsnorm<float, float><<<n_tokens, 256, 0, st>>>((const float *) table, width, tokens, w, eps, x, wn, (float *) y);
+            k_embed_rmsnorm<__nv_bfloat16, __nv_bfloat16><<<n_tokens, row_threads(n_tokens, width), 0, st>>>((const __nv_bfloat16 *) table, width, tokens, w, eps, x, wn, (__nv_bfloat16 *) y);
+        else k_embed_rmsnorm<float, float><<<n_tokens, row_threads(n_tokens, width), 0, st>>>((const float *) table, width, tokens, w, eps, x, wn, (float *) y);
     });
 }
 int launch_cast(const float * x, void * y, int otype, int64_t n, cudaStream_t st) {

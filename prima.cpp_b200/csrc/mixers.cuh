@@ -65,6 +65,9 @@ __device__ __forceinline__ float dot_lane8(const T * __restrict__ a, const float
     return acc;
 }
 
+// CTA size of a kernel that gives every token one CTA (launch bounds 1024): few tokens leave most SMs idle, so a token's row gets more threads
+inline int row_threads(int n_tokens, int width) { return n_tokens >= 128 || width <= 512 ? 256 : width <= 1024 ? 512 : 1024; }
+
 template <typename F> int ck_launch(F && f) {
     g_launches++;
     f();

@@ -40,7 +40,7 @@ __device__ __forceinline__ void group_inv_rms(const float * __restrict__ row, in
 }
 
 template <typename OT>
-__global__ void __launch_bounds__(256) k_group_rmsnorm(const float * __restrict__ x, const int32_t * __restrict__ rows, const float * __restrict__ w, int groups,
+__global__ void __launch_bounds__(1024) k_group_rmsnorm(const float * __restrict__ x, const int32_t * __restrict__ rows, const float * __restrict__ w, int groups,
                                                        float eps, OT * __restrict__ y, int width) {
     __shared__ float red[33];
     __shared__ float inv[MAX_NORM_GROUPS];
@@ -228,8 +228,8 @@ int launch_group_rmsnorm(const float * x, const int32_t * rows, const float * w,
     if (n_rows <= 0) return 0;
     if (groups <= 0 || groups > MAX_NORM_GROUPS || width % groups != 0) return (int) cudaErrorInvalidValue;
     return ck_launch([&] {
-        if (otype == T_BF16) k_group_rmsnorm<__nv_bfloat16><<<n_rows, 256, 0, st>>>(x, rows, w, groups, eps, (__nv_bfloat16 *) y, width);
-        else k_group_rmsnorm<float><<<n_rows, 256, 0, st>>>(x, rows, w, groups, eps, (float *) y, width);
+        if (otype == T_BF16) k_group_rmsnorm<__nv_bfloat16><<<n_rows, row_threads(n_rows, width), 0, st>>>(x, rows, w, groups, eps, (__nv_bfloat16 *) y, width);
+        else k_group_rmsnorm<float><<<n_rows, row_threads(n_rows, width), 0, st>>>(x, rows, w, groups, eps, (float *) y, width);
     });
 }
 int launch_group_rmsnorm_shift(const float * x, const BatchView & b, const float * w, int groups, float eps, const float * mu, float * shift_state,
@@ -250,7 +250,7 @@ int launch_rmsnorm_token_mix(const float * x, const BatchView & b, const float *
                              int64_t slot_stride, void * y, int64_t plane, int otype, float * yf, int width, cudaStream_t st) {
     if (b.n_tokens <= 0) return 0;
     if (!mu || !shift_state || n_planes < 0 || (n_planes > 0 && !y)) return (int) cudaErrorInvalidValue;
-    const int threads = b.n_tokens >= 256 || width <= 1024 ? 256 : 1024;   // few tokens: more of a row's loads in flight
+    const int threads = row_threads(b.n_tokens, width);
     int rc = ck_launch([&] {
         if (otype == T_BF16)
             k_rmsnorm_token_mix<__nv_bfloat16><<<b.n_tokens, threads, 0, st>>>(x, b.slot, b.off, b.entry_of, w, eps, mu, n_planes, shift_state, slot_stride,
