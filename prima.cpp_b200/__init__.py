@@ -6,8 +6,9 @@ The same library and model object serve a second family of models, the layer lis
 directory, sequence slots and a ragged batch step (``Model.from_dir`` / ``Model.batch_step``), driven by :class:`BatchScheduler`.
 Designs: Vamidra (windowed attention with kept first tokens, Mamba-2 mixers), Mumizen (decay linear attention, attention over a
 low-rank latent, clamped gated feed-forward and mixtures of experts, token shift, depth average), Sapudra (post-norm layers with a
-position table, windowed attention with normed query / key heads, squared-ReLU feed-forward, router with sigmoid scores and expert groups)
-and Zevedra (dual mixers: windowed or sink attention beside the gated delta rule or HGRN2, bigram embedding, experts weighted on their input).
+position table, windowed attention with normed query / key heads, squared-ReLU feed-forward, router with sigmoid scores and expert groups),
+Zevedra (dual mixers: windowed or sink attention beside the gated delta rule or HGRN2, bigram embedding, experts weighted on their input)
+and Ruvuvik (chunked attention, latent attention with learned sinks, the WKV mixer, xIELU feed-forward, borrowed weights).
 This Python package is only the thin ctypes binding plus the schedulers; it never falls back to a CPU path: importing
 :mod:`host` raises if the CUDA library is missing.
 """

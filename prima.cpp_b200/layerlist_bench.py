@@ -715,10 +715,10 @@ def ruvuvik_layers(s, z):
     mlp = {"kind": "dense", "ff": s["ff"]}
     lat = {"type": "latent_attention", "mlp": mlp,
            "mixer": {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot_dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"],
-                     "scale": (z["dim"] + z["rot_dim"]) ** -0.5, "rot": {"base": 500000.0, "dims": z["rot_dim"]}}}
+                     "scale": (z["dim"] + z["rot_dim"]) ** -0.5, "rot": {"base": 10000.0, "dims": z["rot_dim"]}}}
     att = {"type": "attention", "mlp": mlp,
            "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5, "softcap": 50.0,
-                     "mask": {"size": 2 * s["window"]}, "rot": {"base": 1000000.0, "dims": s["dim"]}}}
+                     "mask": {"size": 2 * s["window"]}, "rot": {"base": 100000.0, "dims": s["dim"]}}}
     wkv = {"type": "wkv", "mlp": mlp, "mixer": {"heads": z["wkv_heads"], "dim": z["wkv_dim"], "decay_rank": z["decay_rank"]}}
     return {"latent": lat, "attention": att, "wkv": wkv}
 
