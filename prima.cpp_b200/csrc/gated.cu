@@ -19,6 +19,8 @@ namespace pb {
 
 int wkv_scan_ok(const GatedLinIO & io, const GatedLinParams & p);   // wkv.cu
 int launch_wkv_scan(const GatedLinIO & io, const BatchView & b, const GatedLinParams & p, float * state, int64_t slot_stride, float * y, cudaStream_t st);
+int delta_scan_ok(const GatedLinIO & io, const GatedLinParams & p);   // delta.cu
+int launch_delta_scan(const GatedLinIO & io, const BatchView & b, const GatedLinParams & p, float * state, int64_t slot_stride, float * y, cudaStream_t st);
 
 namespace {
 
@@ -95,7 +97,7 @@ __device__ __forceinline__ void pair_of(int i, int dims, int layout, int & ia, i
 
 // One CTA per token.  (1) RMS norm over the whole query projection and over the whole key projection with weights; (2) rotation of the
 // leading entries of every query and key head; (3) every head divided by its own root mean square; (4) rotation of the value heads;
-// (3b) every query head times its own factor; (5) the K / V rows later tokens can still see go to the cache.  Steps that the design does not
+// (3b) every query head times its own factor and the position's; (5) the K / V rows later tokens can still see go to the cache.  Steps that the design does not
 // have are skipped.
 // cs: scratch of rot_dims + vdim floats in shared memory: the token's cosines and sines, computed once for all heads
 __device__ __forceinline__ void attn_prep_rows(float * qr, float * kr, float * vr, float fp, const AttnParams & a, const AttnPrep & pr, float * red, float * cs) {
@@ -104,7 +106,11 @@ __device__ __forceinline__ void attn_prep_rows(float * qr, float * kr, float * v
     const int hq = pr.rot_dims / 2, hv2 = pr.v_rot ? a.vdim / 2 : 0;
     float * csv = cs + 2 * hq;
     for (int i = threadIdx.x; i < hq + hv2; i += blockDim.x) {
-        if (i < hq) sincosf(fp * pr.rot_freq[i], &cs[2 * i + 1], &cs[2 * i]);
+        if (i < hq) {
+            sincosf(fp * pr.rot_freq[i], &cs[2 * i + 1], &cs[2 * i]);
+            cs[2 * i] *= pr.rot_mag;
+            cs[2 * i + 1] *= pr.rot_mag;
+        }
         else sincosf(fp * pr.v_freq[i - hq], &csv[2 * (i - hq) + 1], &csv[2 * (i - hq)]);
     }
     // the barrier after the whole-projection norm, or the one below, makes the table visible
@@ -140,9 +146,10 @@ __device__ __forceinline__ void attn_prep_rows(float * qr, float * kr, float * v
             for (int i = lane; i < a.dim; i += 32) hv[i] *= inv;
         }
     }
-    if (pr.q_scale) {
+    if (pr.q_scale || pr.q_temp_every > 0.f) {
         if (pr.norm == QKN_HEAD_UNIT) __syncthreads();
-        for (int i = threadIdx.x; i < QD; i += blockDim.x) qr[i] *= pr.q_scale[i / a.dim];
+        const float ft = pr.q_temp_every > 0.f ? 1.f + pr.q_temp_coef * logf(floorf((fp + 1.f) / pr.q_temp_every) + 1.f) : 1.f;
+        for (int i = threadIdx.x; i < QD; i += blockDim.x) qr[i] *= pr.q_scale ? pr.q_scale[i / a.dim] * ft : ft;
     }
     if (pr.v_rot && a.vdim > 1) {
         const int hp = a.vdim / 2, total = a.kv_heads * hp;
@@ -181,6 +188,7 @@ __device__ __forceinline__ void delta_prep_rows(float * qr, float * kr, float * 
     }
     for (int h = threadIdx.x; h < heads; h += blockDim.x) {
         bp[h] = sigmoid_f(bp[h]);
+        if (!ap) continue;
         const float z = ap[h] + dt_bias[h];
         const float sp = z > 20.f ? z : log1pf(expf(z));
         ap[h] = expf(-expf(A_log[h]) * sp);
@@ -207,7 +215,7 @@ __global__ void __launch_bounds__(1024) k_dual_prep_store(RecPrep rc, float * __
     const int e = entry_of[t];
     const int n = off[e + 1] - off[e];
     const int p = pos0[e] + (t - off[e]), pend = pos0[e] + n;
-    const int QD = a.heads * a.dim, KD = a.kv_heads * a.dim, VD = a.kv_heads * a.vdim, RQ = rc.kind >= 0 ? rc.qk_heads * rc.dim : 0;
+    const int QD = a.heads * a.dim, KD = a.kv_heads * a.dim, VD = attn_v_row(a), RQ = rc.kind >= 0 ? rc.qk_heads * rc.dim : 0;
     float * gq = q + (int64_t) t * ldq, * gk = k + (int64_t) t * ldk, * gv = v + (int64_t) t * ldv;
     float * grq = rc.kind >= 0 ? rc.q + (int64_t) t * rc.ldq : nullptr, * grk = rc.kind >= 0 ? rc.k + (int64_t) t * rc.ldk : nullptr;
     float * qr = gq, * kr = gk, * vr = gv, * rqr = grq, * rkr = grk;
@@ -221,7 +229,7 @@ __global__ void __launch_bounds__(1024) k_dual_prep_store(RecPrep rc, float * __
         for (int i = threadIdx.x; i < RQ; i += blockDim.x) { rqr[i] = grq[i]; rkr[i] = grk[i]; }
         __syncthreads();
     }
-    if (rc.kind == 0) delta_prep_rows(rqr, rkr, rc.beta + (int64_t) t * rc.ldb, rc.a + (int64_t) t * rc.lda, rc.p0, rc.p1, rc.qk_heads, rc.heads, rc.dim);
+    if (rc.kind == 0) delta_prep_rows(rqr, rkr, rc.beta + (int64_t) t * rc.ldb, rc.a ? rc.a + (int64_t) t * rc.lda : nullptr, rc.p0, rc.p1, rc.qk_heads, rc.heads, rc.dim);
     else if (rc.kind == 1) hgrn2_prep_rows(rqr, rkr, rc.p0, rc.p1, RQ);
     attn_prep_rows(qr, kr, vr, (float) p, a, pr, red, cs);
     __syncthreads();
@@ -278,7 +286,7 @@ __global__ void __launch_bounds__(256) k_delta_prep(float * __restrict__ q, int6
                                                     int64_t ldb, float * __restrict__ a, int64_t lda, const float * __restrict__ A_log,
                                                     const float * __restrict__ dt_bias, int qk_heads, int heads, int dim) {
     const int64_t t = blockIdx.x;
-    delta_prep_rows(q + t * ldq, k + t * ldk, beta + t * ldb, a + t * lda, A_log, dt_bias, qk_heads, heads, dim);
+    delta_prep_rows(q + t * ldq, k + t * ldk, beta + t * ldb, a ? a + t * lda : nullptr, A_log, dt_bias, qk_heads, heads, dim);
 }
 __global__ void k_hgrn2_prep(float * __restrict__ q, int64_t ldq, float * __restrict__ f, int64_t ldf, const float * __restrict__ f_bias,
                              const float * __restrict__ lower, int n) {
@@ -346,12 +354,13 @@ __global__ void __launch_bounds__(128) k_dual_post(const float * __restrict__ o,
 // stages the decay rows as well and, once per chunk, one warp per token sums q . (u k), so that a token costs  y = S^T q + (q . u k) v  and
 // S <- diag(w) S + k v^T.
 constexpr int GCHUNK = 16, GCOLS = 16;
-enum : int { GL_DELTA = 0, GL_TIED = 1, GL_BONUS = 2 };
+enum : int { GL_DELTA = 0, GL_TIED = 1, GL_BONUS = 2, GL_DELTA_CH = 3 };
 template <int NREG, int LN, int MODE>
 __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
                                                                   GatedLinParams p, float * __restrict__ state, int64_t slot_stride, float * __restrict__ y) {
     extern __shared__ float sm[];
-    constexpr bool DELTA = MODE == GL_DELTA, TIED = MODE == GL_TIED, BONUS = MODE == GL_BONUS;
+    constexpr bool DELTA = MODE == GL_DELTA, TIED = MODE == GL_TIED, BONUS = MODE == GL_BONUS, DELTA_CH = MODE == GL_DELTA_CH;
+    constexpr bool ROWS3 = BONUS || DELTA_CH;   // the decay per channel is a third staged row
     constexpr int NT = GCOLS * LN;
     constexpr int NV = (GCHUNK * GCOLS + NT - 1) / NT;
     const int N = p.dim, P = p.vdim, inner = p.heads * p.vdim;
@@ -365,7 +374,7 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
     float * Qs = Ks + GCHUNK * N;           // [GCHUNK][N]
     float * Vs = Qs + GCHUNK * N;           // [GCHUNK][GCOLS]
     float * Gs = Vs + GCHUNK * GCOLS;       // [GCHUNK] decay per token (one per head) or the bonus product q . (u k), [GCHUNK] beta
-    float * Ws = Gs + 2 * GCHUNK;           // [GCHUNK][N]  BONUS: the decay per channel
+    float * Ws = Gs + 2 * GCHUNK;           // [GCHUNK][N]  ROWS3: the decay per channel
     float * gst = state + (int64_t) slot[e] * slot_stride + (int64_t) h * N * P;
     float S[NREG];
 #pragma unroll
@@ -392,7 +401,7 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
             }
         }
     };
-    float rk[NREG], rq[NREG], rw[BONUS ? NREG : 1], rv[NV], rg = 0.f;
+    float rk[NREG], rq[NREG], rw[ROWS3 ? NREG : 1], rv[NV], rg = 0.f;
     auto fetch = [&](int c0) {
         const int nc = min(GCHUNK, n - c0);
 #pragma unroll
@@ -401,8 +410,8 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
             if (i < nc * N) {
                 const int tt = i / N, nn = i - tt * N;
                 const int64_t tok = t0 + c0 + tt;
-                rk[k] = TIED ? io.decay[tok * io.ldd + hk * N + nn] : io.k[tok * io.ldk + hk * N + nn];
-                if constexpr (BONUS) rw[k] = io.decay[tok * io.ldd + hk * N + nn];
+                rk[k] = TIED ? io.decay[tok * io.ldd + h * N + nn] : io.k[tok * io.ldk + hk * N + nn];
+                if constexpr (ROWS3) rw[k] = io.decay[tok * io.ldd + h * N + nn];
                 rq[k] = io.q[tok * io.ldq + hk * N + nn];
             }
         }
@@ -416,7 +425,7 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
             rg = 0.f;
             if (tt < nc) {
                 if (tid < GCHUNK) { if (DELTA) rg = io.decay[(int64_t) (t0 + c0 + tt) * io.ldd + h]; }
-                else if (DELTA) rg = io.beta[(int64_t) (t0 + c0 + tt) * io.ldb + h];
+                else if (DELTA || DELTA_CH) rg = io.beta[(int64_t) (t0 + c0 + tt) * io.ldb + h];
             }
         }
     };
@@ -429,7 +438,7 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
             const int i = tid + NT * k;
             if (i < nc * N) {
                 Ks[i] = rk[k]; Qs[i] = rq[k];
-                if constexpr (BONUS) Ws[i] = rw[k];
+                if constexpr (ROWS3) Ws[i] = rw[k];
             }
         }
 #pragma unroll
@@ -473,6 +482,27 @@ __global__ void __launch_bounds__(GCOLS * LN) k_gated_linattn_reg(GatedLinIO io,
 #pragma unroll
                 for (int j = 0; j < NREG; j++) S[j] = fmaf(kk[j], u, g * S[j]);
                 out = fmaf(u, kq, g * sq);
+            } else if constexpr (DELTA_CH) {
+                float ww[NREG];
+                row_regs(Ws + tt * N, ww);
+                float sk = 0.f, sq = 0.f, kq = 0.f;
+#pragma unroll
+                for (int j = 0; j < NREG; j++) {
+                    S[j] *= ww[j];
+                    sk = fmaf(S[j], kk[j], sk);
+                    sq = fmaf(S[j], qq[j], sq);
+                    kq = fmaf(kk[j], qq[j], kq);
+                }
+#pragma unroll
+                for (int o = 1; o < LN; o <<= 1) {
+                    sk += __shfl_xor_sync(0xffffffffu, sk, o);
+                    sq += __shfl_xor_sync(0xffffffffu, sq, o);
+                    kq += __shfl_xor_sync(0xffffffffu, kq, o);
+                }
+                const float u = Gs[GCHUNK + tt] * (xv - sk);
+#pragma unroll
+                for (int j = 0; j < NREG; j++) S[j] = fmaf(kk[j], u, S[j]);
+                out = fmaf(u, kq, sq);
             } else if constexpr (BONUS) {
                 float ww[NREG];
                 row_regs(Ws + tt * N, ww);
@@ -535,7 +565,7 @@ __global__ void __launch_bounds__(256) k_gated_linattn_smem(GatedLinIO io, const
         __syncthreads();
         for (int i = threadIdx.x; i < N; i += blockDim.x) {
             qs[i] = io.q[tok * io.ldq + hk * N + i];
-            const float f = p.decay_per_channel ? io.decay[tok * io.ldd + hk * N + i] : io.decay[tok * io.ldd + h];
+            const float f = p.decay_per_channel ? io.decay[tok * io.ldd + h * N + i] : io.decay[tok * io.ldd + h];
             fs[i] = f;
             ks[i] = p.tied_key ? 1.f - f : io.k[tok * io.ldk + hk * N + i];
         }
@@ -663,13 +693,16 @@ int launch_causal_conv(const float * u, int64_t ldu, const BatchView & b, int ch
     });
 }
 
-static int dual_prep_launch(const RecPrep & rc, float * q, int64_t ldq, float * k, int64_t ldk, float * v, int64_t ldv, const BatchView & b, const AttnParams & a,
+static int dual_prep_launch(const RecPrep & rc, float * q, int64_t ldq, float * k, int64_t ldk, float * v, int64_t ldv, const BatchView & b, const AttnParams & att,
                             const AttnPrep & pr, float * kcache, float * vcache, int64_t slot_stride, cudaStream_t st) {
-    if (a.heads <= 0 || a.kv_heads <= 0 || a.dim <= 0 || a.vdim <= 0 || pr.rot_dims < 0 || pr.rot_dims > a.dim || (pr.rot_dims & 1) ||
+    AttnParams a = att;
+    if (a.kv_heads <= 0 || (a.tied_v && (a.vdim != a.dim || pr.v_rot))) return (int) cudaErrorInvalidValue;
+    if (!a.own_kv) a.kv_heads = 0;   // another layer's keys and values: only the queries are prepared, nothing is stored
+    if (a.heads <= 0 || a.dim <= 0 || a.vdim <= 0 || pr.rot_dims < 0 || pr.rot_dims > a.dim || (pr.rot_dims & 1) ||
         (pr.rot_dims > 0 && !pr.rot_freq) || (pr.v_rot && !pr.v_freq) || (pr.norm == QKN_WHOLE_WEIGHT && (!pr.wq || !pr.wk)))
         return (int) cudaErrorInvalidValue;
     // the token's rows in shared memory when they fit
-    const size_t floats = (size_t) a.heads * a.dim + (size_t) a.kv_heads * (a.dim + a.vdim) + (rc.kind >= 0 ? 2 * (size_t) rc.qk_heads * rc.dim : 0);
+    const size_t floats = (size_t) a.heads * a.dim + (size_t) a.kv_heads * a.dim + (size_t) attn_v_row(a) + (rc.kind >= 0 ? 2 * (size_t) rc.qk_heads * rc.dim : 0);
     const size_t table = (size_t) ((pr.rot_dims + a.vdim + 3) & ~3);   // cosines and sines of the token's position
     const int staged = (floats + table) * sizeof(float) <= 160 * 1024;
     const size_t smem = (table + (staged ? floats : 0)) * sizeof(float);
@@ -703,7 +736,7 @@ int launch_attn_unrotate_gate(const float * o, const BatchView & b, int heads, i
 int launch_delta_prep(float * q, int64_t ldq, float * k, int64_t ldk, float * beta, int64_t ldb, float * a, int64_t lda, const float * A_log,
                       const float * dt_bias, int qk_heads, int heads, int dim, int n_tokens, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
-    if (qk_heads <= 0 || heads <= 0 || dim <= 0 || !A_log || !dt_bias) return (int) cudaErrorInvalidValue;
+    if (qk_heads <= 0 || heads <= 0 || dim <= 0 || (a && (!A_log || !dt_bias))) return (int) cudaErrorInvalidValue;
     return ck_launch([&] { k_delta_prep<<<n_tokens, 256, 0, st>>>(q, ldq, k, ldk, beta, ldb, a, lda, A_log, dt_bias, qk_heads, heads, dim); });
 }
 int launch_hgrn2_prep(float * q, int64_t ldq, float * f, int64_t ldf, const float * f_bias, const float * lower, int n, int n_tokens, cudaStream_t st) {
@@ -715,16 +748,20 @@ int launch_hgrn2_prep(float * q, int64_t ldq, float * f, int64_t ldf, const floa
 int launch_gated_linattn(const GatedLinIO & io, const BatchView & b, const GatedLinParams & p, float * state, int64_t slot_stride, float * y, cudaStream_t st) {
     if (b.n_tokens <= 0) return 0;
     if (p.heads <= 0 || p.qk_heads <= 0 || p.heads % p.qk_heads || p.dim <= 0 || p.vdim <= 0 || !state || !io.q || !io.v || !io.decay || (p.delta && !io.beta) ||
-        (p.tied_key && (!p.decay_per_channel || p.delta)) || (!p.tied_key && !io.k) || (p.decay_per_channel && !p.tied_key && !p.bonus) ||
+        (p.tied_key && (!p.decay_per_channel || p.delta || p.qk_heads != p.heads)) || (!p.tied_key && !io.k) ||
+        (p.decay_per_channel && !p.tied_key && !p.bonus && !p.delta) ||
         (p.bonus && (!p.decay_per_channel || p.delta || p.tied_key || !io.bonus)))
         return (int) cudaErrorInvalidValue;
     static const bool plain_wkv = getenv("PB200_WKV_PLAIN") != nullptr;   // A/B and tests: the shared kernels below for the bonus form too
     if (p.bonus && !plain_wkv && wkv_scan_ok(io, p)) return launch_wkv_scan(io, b, p, state, slot_stride, y, st);
-    // the register kernels: delta rule with one decay per head, tied key with a decay per channel, bonus form with a decay per channel
-    if (p.dim <= 256 && ((p.delta && !p.decay_per_channel) || (p.tied_key && !p.delta) || p.bonus)) {
+    const bool delta_ch = p.delta && p.decay_per_channel;
+    static const bool plain_delta = getenv("PB200_DELTA_PLAIN") != nullptr;   // the same for the delta rule with a decay per channel
+    if (delta_ch && !plain_delta && delta_scan_ok(io, p)) return launch_delta_scan(io, b, p, state, slot_stride, y, st);
+    // the register kernels: delta rule with one decay per head or one per channel, tied key and bonus form with a decay per channel
+    if (p.dim <= 256 && (p.delta || p.tied_key || p.bonus)) {
         const int ln = p.dim <= 32 ? 8 : p.dim <= 64 ? 16 : 32;
         const int nreg = (p.dim + ln - 1) / ln;
-        const size_t smem = ((size_t) (p.bonus ? 3 : 2) * GCHUNK * p.dim + GCHUNK * GCOLS + 2 * GCHUNK) * sizeof(float);
+        const size_t smem = ((size_t) (p.bonus || delta_ch ? 3 : 2) * GCHUNK * p.dim + GCHUNK * GCOLS + 2 * GCHUNK) * sizeof(float);
         const dim3 grid((unsigned) (p.heads * ((p.vdim + GCOLS - 1) / GCOLS)), (unsigned) b.n_entries);
 #define PB_GL(NR, LNV)                                                                                                                               \
     do {                                                                                                                                             \
@@ -732,6 +769,11 @@ int launch_gated_linattn(const GatedLinIO & io, const BatchView & b, const Gated
             const int rc = raise_smem(k_gated_linattn_reg<NR, LNV, GL_BONUS>, smem);                                                                 \
             if (rc) return rc;                                                                                                                       \
             return ck_launch([&] { k_gated_linattn_reg<NR, LNV, GL_BONUS><<<grid, GCOLS * LNV, smem, st>>>(io, b.slot, b.off, p, state, slot_stride, y); });            \
+        }                                                                                                                                            \
+        if (delta_ch) {                                                                                                                              \
+            const int rc = raise_smem(k_gated_linattn_reg<NR, LNV, GL_DELTA_CH>, smem);                                                              \
+            if (rc) return rc;                                                                                                                       \
+            return ck_launch([&] { k_gated_linattn_reg<NR, LNV, GL_DELTA_CH><<<grid, GCOLS * LNV, smem, st>>>(io, b.slot, b.off, p, state, slot_stride, y); });         \
         }                                                                                                                                            \
         if (p.delta) return ck_launch([&] { k_gated_linattn_reg<NR, LNV, GL_DELTA><<<grid, GCOLS * LNV, smem, st>>>(io, b.slot, b.off, p, state, slot_stride, y); }); \
         return ck_launch([&] { k_gated_linattn_reg<NR, LNV, GL_TIED><<<grid, GCOLS * LNV, smem, st>>>(io, b.slot, b.off, p, state, slot_stride, y); });            \
@@ -761,7 +803,8 @@ int launch_dual_prep_store(int rec_kind, float * rq, int64_t ldrq, float * rk, i
                            const float * p1, int qk_heads, int r_heads, int r_dim, float * q, int64_t ldq, float * k, int64_t ldk, float * v, int64_t ldv,
                            const BatchView & b, const AttnParams & a, const AttnPrep & pr, float * kcache, float * vcache, int64_t slot_stride, cudaStream_t st) {
     if (b.n_tokens <= 0) return 0;
-    if (rec_kind < 0 || rec_kind > 1 || !rq || !rk || !p0 || !p1 || qk_heads <= 0 || r_dim <= 0 || (rec_kind == 0 && (!beta || !ra || r_heads <= 0)))
+    if (rec_kind < 0 || rec_kind > 1 || !rq || !rk || qk_heads <= 0 || r_dim <= 0 || (rec_kind == 0 && (!beta || r_heads <= 0)) ||
+        ((rec_kind == 1 || ra) && (!p0 || !p1)))
         return (int) cudaErrorInvalidValue;
     RecPrep rc;
     rc.kind = rec_kind;

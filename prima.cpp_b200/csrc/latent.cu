@@ -29,6 +29,10 @@ __device__ __forceinline__ void turn(float u, float v, int pos, float f, float m
     ov = v * c + u * s;
 }
 
+// factor on output element (head h, entry dv): sigmoid of the head's gate logit, of the element's, or none
+__device__ __forceinline__ float latent_gate(const LatentParams & p, const float * __restrict__ gate, int64_t at, int h, int dv) {
+    return gate ? sigmoid_f(gate[at + (p.gate_mode == 1 ? h : h * p.vdim + dv)]) : 1.f;
+}
 // turns the rotated part of every query head of one token
 __device__ __forceinline__ void rope_q_row(float * __restrict__ row, int pos, const LatentParams & p, const float * __restrict__ freq) {
     const int half = p.rot_dims / 2, DQ = p.dim + p.rot_dim;
@@ -69,10 +73,12 @@ __global__ void __launch_bounds__(256) k_latent_prep(float * __restrict__ proj, 
     float s = 0.f;
     for (int i = threadIdx.x; i < R; i += blockDim.x) s = fmaf(kv[i], kv[i], s);
     const float invk = 1.f / sqrtf(block_sum(s, red) / (float) R + eps);
-    float * crow = cache + (int64_t) slot[e] * slot_stride + (int64_t) pos * (R + Dr);
+    // of the positions that share a row only the last one of this entry is stored
+    const bool keep = pos + p.cache_rows >= pos0[e] + (off[e + 1] - off[e]);
+    float * crow = cache + (int64_t) slot[e] * slot_stride + (int64_t) (pos % p.cache_rows) * (R + Dr);
     for (int i = threadIdx.x; i < R; i += blockDim.x) {
         const float v = kv[i] * invk * wkv[i];
-        crow[i] = v;
+        if (keep) crow[i] = v;
         if (lat) put(lat, (int64_t) t * R + i, v);
     }
     const int half = p.rot_dims / 2;
@@ -82,11 +88,10 @@ __global__ void __launch_bounds__(256) k_latent_prep(float * __restrict__ proj, 
             pair_at(p, i, ia, ib);
             float a, b;
             turn(kv[R + ia], kv[R + ib], pos, freq[i], p.rot_mag, a, b);
-            crow[R + ia] = a;
-            crow[R + ib] = b;
+            if (keep) { crow[R + ia] = a; crow[R + ib] = b; }
             if (kr) { kr[(int64_t) t * Dr + ia] = a; kr[(int64_t) t * Dr + ib] = b; }
         } else if (i >= 2 * half) {
-            crow[R + i] = kv[R + i];
+            if (keep) crow[R + i] = kv[R + i];
             if (kr) kr[(int64_t) t * Dr + i] = kv[R + i];
         }
     }
@@ -107,7 +112,7 @@ __global__ void k_latent_gather(const float * __restrict__ cache, int64_t slot_s
     const int e = entry_of[t];
     const int pos = pos0[e] + (t - off[e]);
     const int R = p.kv_rank, Dr = p.rot_dim;
-    const float * crow = cache + (int64_t) slot[e] * slot_stride + (int64_t) pos * (R + Dr);
+    const float * crow = cache + (int64_t) slot[e] * slot_stride + (int64_t) (pos % p.cache_rows) * (R + Dr);
     for (int i = threadIdx.x; i < R; i += blockDim.x) put(lat, (int64_t) t * R + i, crow[i]);
     for (int i = threadIdx.x; i < Dr; i += blockDim.x) kr[(int64_t) t * Dr + i] = crow[R + i];
 }
@@ -174,7 +179,7 @@ __global__ void __launch_bounds__(256) k_latent_up_v(const float * __restrict__ 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int dv = warp; dv < DV; dv += (int) (blockDim.x >> 5)) {
         const float acc = wsum(dot_lane8(wuv + ((int64_t) h * DV + dv) * R, os, R, lane));
-        if (lane == 0) put(out, (int64_t) t * p.heads * DV + h * DV + dv, gate ? acc * sigmoid_f(gate[(int64_t) t * ldg + h * DV + dv]) : acc);
+        if (lane == 0) put(out, (int64_t) t * p.heads * DV + h * DV + dv, acc * latent_gate(p, gate, (int64_t) t * ldg, h, dv));
     }
 }
 
@@ -208,7 +213,7 @@ __global__ void __launch_bounds__(256) k_latent_decode_split(const float * __res
     float * lrun = mrun + LT_HEADS;
     float * corr = lrun + LT_HEADS;
     const int tid = threadIdx.x, hl = tid >> 4, r = tid & 15;
-    const int rows_used = pos0[e] + 1;        // the token's own row is in the cache already
+    const int rows_used = min(pos0[e] + 1, p.cache_rows);   // the token's own row is in the cache already; a window's ring holds what is visible
     const int per = latent_rows_per_split(rows_used, splits);
     const int r_lo = s * per, r_hi = min(rows_used, r_lo + per);
     if (r_lo >= rows_used) return;            // no rows left for this split: the merge does not read it
@@ -339,7 +344,7 @@ __global__ void __launch_bounds__(256) k_latent_merge_up_v(const float * __restr
     const int R = p.kv_rank, DV = p.vdim, H = p.heads;
     float * w = os + R;
     const float * pe = part + ((int64_t) e * all_splits * H + h) * (R + 2);
-    const int rows_used = pos0[e] + 1, per = latent_rows_per_split(rows_used, all_splits), splits = (rows_used + per - 1) / per;   // the rest hold no rows
+    const int rows_used = min(pos0[e] + 1, p.cache_rows), per = latent_rows_per_split(rows_used, all_splits), splits = (rows_used + per - 1) / per;   // the rest hold no rows
     const int64_t stride = (int64_t) H * (R + 2);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (warp == 0) {
@@ -371,7 +376,7 @@ __global__ void __launch_bounds__(256) k_latent_merge_up_v(const float * __restr
     const int share = (DV + gridDim.z - 1) / gridDim.z, dv_lo = blockIdx.z * share, dv_hi = min(DV, dv_lo + share);
     for (int dv = dv_lo + warp; dv < dv_hi; dv += (int) (blockDim.x >> 5)) {
         const float acc = wsum(dot_lane8(wuv + ((int64_t) h * DV + dv) * R, os, R, lane));
-        if (lane == 0) put(out, (int64_t) t * H * DV + h * DV + dv, gate ? acc * sigmoid_f(gate[(int64_t) t * ldg + h * DV + dv]) : acc);
+        if (lane == 0) put(out, (int64_t) t * H * DV + h * DV + dv, acc * latent_gate(p, gate, (int64_t) t * ldg, h, dv));
     }
 }
 
@@ -379,7 +384,7 @@ __global__ void __launch_bounds__(256) k_latent_merge_up_v(const float * __restr
 
 static bool latent_ok(const LatentParams & p) {
     return p.heads > 0 && p.dim > 0 && p.rot_dim >= 0 && p.vdim > 0 && p.kv_rank > 0 && p.q_rank >= 0 && p.rot_dims >= 0 && p.rot_dims <= p.rot_dim &&
-           p.rot_dims % 2 == 0;
+           p.rot_dims % 2 == 0 && p.cache_rows > 0 && (p.window <= 0 || p.cache_rows <= p.window);
 }
 
 int launch_latent_prep(float * proj, const BatchView & b, const LatentParams & p, const float * wq, const float * wkv, const float * freq, float eps,

@@ -1,12 +1,13 @@
 // prima.cpp_b200/csrc/layers.cu — the engine of the layer-list family (arch.h): a configuration file lists the layers, every layer has
 // a sequence mixer (windowed attention with kept first tokens, a Mamba-2 state-space mixer, linear attention with a fixed decay per
 // head, softmax attention over a low-rank latent, a WKV mixer, or a dual mixer: an attention branch beside a gated linear recurrence) and an
-// optional feed-forward (tanh-GELU gated; squared ReLU; xIELU; clamped gated, dense or a routed mixture of experts), inside one of these layer frames: norms before and after every sublayer (FRAME_SANDWICH), or a grouped RMS norm
+// optional feed-forward (tanh-GELU gated; SiLU gated; squared ReLU; xIELU; clamped gated, dense or a routed mixture of experts), inside one of these layer frames: norms before and after every sublayer (FRAME_SANDWICH), or a grouped RMS norm
 // before it with token shift and a depth average of all layer results (FRAME_PRENORM), or a layer norm with weight and bias on the
 // sublayer's result only, scaled by one factor, with a learned position table on the embedding (FRAME_POSTNORM), or an RMS norm with one
 // learned number before every sublayer, sublayer results times one factor, and a repeated block whose passes add the embedding output and
 // a step vector (FRAME_PRERMS; a norm may also have a weight per entry, and
-// the embedding may be normed).  A layer may borrow another layer's weights; its cache and state stay its own.  Weights are dense f32 / bf16 matrices.  It lives behind the same model object and C ABI as the k-quant transformer engine
+// the embedding may be normed).  A layer may borrow another layer's weights; its cache and state stay its own.  An attention layer may read
+// another layer's keys and values.  Weights are dense f32 / bf16 matrices.  It lives behind the same model object and C ABI as the k-quant transformer engine
 // (engine.cu): pb200_model_set_tensor / _synth / _finalize / _free, sequence slots, device arg-max — and steps through the ragged
 // batch step (pb200_batch_step) that the scheduler drives; the single-sequence entry points of the k-quant family answer PB200_ENOTSUP.
 //
@@ -53,10 +54,10 @@ extern std::atomic<uint64_t> g_launches;
 namespace pb {
 
 enum : int { MIX_ATTENTION = 0, MIX_MAMBA2 = 1, MIX_DECAY = 2, MIX_LATENT = 3, MIX_DUAL = 4, MIX_WKV = 5 };
-enum : int { FF_GELU = 0, FF_CLAMPED = 1, FF_MOE = 2, FF_RELU2 = 3, FF_XIELU = 4 };   // FF_MOE: the expert form is MoeParams::act
+enum : int { FF_GELU = 0, FF_CLAMPED = 1, FF_MOE = 2, FF_RELU2 = 3, FF_XIELU = 4, FF_SILU = 5 };   // FF_MOE: the expert form is MoeParams::act
 enum : int { FRAME_SANDWICH = 0, FRAME_PRENORM = 1, FRAME_POSTNORM = 2, FRAME_PRERMS = 3 };
 enum : int { ROUTE_SOFTMAX_TOP = 0, ROUTE_SIGMOID_GROUPS = 1, ROUTE_SIGMOID_PLAIN = 2 };
-enum : int { REC_DELTA = 0, REC_HGRN2 = 1 };                 // recurrent branch of a dual mixer
+enum : int { REC_DELTA = 0, REC_HGRN2 = 1, REC_DELTA_CH = 2 };   // recurrent branch of a dual mixer (REC_DELTA_CH: gated delta rule with a decay per channel)
 enum : int { JOIN_SCALED_SUM = 0, JOIN_NORMED_MEAN = 1 };    // a * left + b * right through one output product, or the mean of the two normed results
 
 struct DenseW {           // row-major [N][K] in the model's compute type
@@ -81,8 +82,14 @@ struct DualMix {
     int qk_norm = QKN_NONE, rot_dims = 0, rot_layout = ROT_INTERLEAVED, v_rot = 0;
     int gate_mode = 1;                      // 1: a gate logit per head, 2: per output element
     GatedLinParams rp;
-    // columns of the fused projection: left q | k | v, right q | k (HGRN2: forget logits) | v, then gates and per-head numbers; the first
-    // conv_ch columns pass the convolution (the first conv_l of them without activation, the rest with SiLU)
+    float q_temp_coef = 0.f, q_temp_every = 0.f;   // every > 0: query temperature by position
+    bool biased = false;                    // biases on the left q and k
+    int r_gate_act = 1;                     // output gate of the recurrent branch: 0 sigmoid, 1 SiLU, -1 none
+    int a_rank = 0, g_rank = 0;             // REC_DELTA_CH: inner sizes of the low-rank maps of decay and gate (0: a tensor's shape will tell)
+    // columns of the fused projection: left q | k | v, right q | k (HGRN2: forget logits) | v, then gates and per-head numbers (REC_DELTA_CH: then
+    // the inner values of the low-rank maps, joined when their sizes are known); columns [conv_0, conv_0 + conv_ch) pass the convolution (the
+    // first conv_l of them without activation, the rest with SiLU)
+    int conv_0 = 0;
     int c_q = 0, c_k = 0, c_v = 0, c_rq = 0, c_rk = 0, c_rv = 0, c_g = 0, c_rb = 0, c_ra = 0, c_rg = 0, cols = 0, conv_ch = 0, conv_l = 0;
 };
 
@@ -106,7 +113,7 @@ struct LLayer {
     VecF decay, onorm;
     // latent attention (lproj: fused dq | gate | dkv)
     LatentParams lat;
-    int kv_from = -1;                  // >= 0: the layer whose latent cache this one reads
+    int kv_from = -1;                  // >= 0: the layer whose cache (latents, or keys and values) this one reads
     DenseW lproj, uq, ukv;             // ukv: key up-projection [heads * dim], then value up-projection [heads * vdim] of the latent
     VecF dq_norm, dkv_norm, rot_freq, sink;
     bool has_sink = false;             // a learned score per head of one more key without a value
@@ -124,7 +131,8 @@ struct LLayer {
     bool qk_norm = false;
     VecF q_norm, k_norm;
     // attention whose inputs are prepared by launch_attn_prep_store: norm over the whole q / k projection, rotation, a factor per query head
-    bool att_prep = false;
+    bool att_prep = false, att_temp = false;
+    float att_rot_mag = 1.f;
     int att_qkn = QKN_NONE, att_rot_dims = 0, att_rot_layout = ROT_INTERLEAVED;
     VecF temp;
     // mixture of experts: form of the router; the shared expert's per-token gate vector [width] (ROUTE_SIGMOID_GROUPS)
@@ -133,6 +141,8 @@ struct LLayer {
     // dual mixer (qkvg: the fused projection of both branches; out: the output product over [left | right], or the left one; out_r: the right one)
     DualMix dual;
     DenseW out_r;
+    DenseW ra1, rg1;                   // REC_DELTA_CH: down-projections of the low-rank maps until ll_finalize joins them to qkvg
+    VecF ra2, rg2, qk_bias;            // the maps' second matrices (fp32); bias per column of the fused projection (zero where there is none)
     // WKV mixer: token mix with five blends (r, k, v, g, w), qkvg = one matrix of the four projections, decay from a low-rank map (fp32)
     GatedLinParams wkv;
     int decay_rank = 0;                // inner size of the decay's map: the configuration's, or what the first of its tensors to arrive has
@@ -179,6 +189,7 @@ struct LayerList {
     DenseW loop_in;
     VecF loop_step;
     DenseW embed, head;
+    bool tied_head = false;      // logits come from the embedding table itself
     VecF final_norm;
     // FRAME_POSTNORM
     DenseW pos_table;         // learned position vectors [max_pos][width], added to the embedding
@@ -1022,7 +1033,7 @@ static int ruvuvik_configure(const Json & cfg, LayerList & ll, std::string & err
             a.gated = 1;
             if (const Json * mk = mx->get("mask"))
                 if (mk->kind == Json::OBJ) a.chunk = (int) std::min<long long>(std::max<long long>(mk->integer("size", 0), 0), 1 << 30);
-            L.att_prep = true;
+            L.att_prep = L.att_temp = true;
             L.att_qkn = QKN_WHOLE_WEIGHT;
             L.att_rot_layout = ROT_INTERLEAVED;
             if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dim <= 0 || a.vdim <= 0 || a.vdim > 512) { err = "attention sizes"; return PB200_EINVAL; }
@@ -1037,7 +1048,7 @@ static int ruvuvik_configure(const Json & cfg, LayerList & ll, std::string & err
             a.vdim = (int) mx->integer("vdim", a.dim);
             a.kv_rank = (int) mx->integer("kv_rank", 0);
             a.q_rank = 0;
-            a.gated = 0;
+            a.gate_mode = 0;
             a.own_kv = 1;
             a.rot_layout = ROT_INTERLEAVED;
             a.scale = (float) mx->number("scale", a.dim + a.rot_dim > 0 ? 1.0 / std::sqrt((double) (a.dim + a.rot_dim)) : 1.0);
@@ -1145,6 +1156,252 @@ static bool ruvuvik_resolve(LayerList & ll, const std::string & name, TensorPlac
     return false;
 }
 
+// ---------------------------------------------------------------------------------------------------------------
+// Ludusun: configuration keys and tensor names.  The stream starts as embed[token] * scale; every layer is x <- x + mixer(norm x),
+// x <- x + ff(norm x) with an RMS norm whose weight is stored around zero.  Mixers: "attention" (rotate-half partial rotation with the
+// long-context blend, every query / key head divided by its root mean square after it, a learned sink per head; "kv_from" reads another layer's
+// keys and values), "latent_attention" (query latent, no positions, sliding window, a gate per head) and "parallel" (attention whose keys are its
+// values, with biases, a query temperature by position and a gate per element, beside the gated delta rule with a decay per channel and a gate,
+// both from low-rank maps).  SiLU-gated feed-forward; the logits come from the embedding table and are soft-capped.
+static int ludusun_attention(const Json & mx, LayerList & ll, LLayer & L, std::string & err) {
+    L.kind = MIX_ATTENTION;
+    AttnParams & a = L.att;
+    a.heads = (int) mx.integer("heads", 0);
+    a.kv_heads = (int) mx.integer("kv_heads", a.heads);
+    a.dim = (int) mx.integer("dim", 0);
+    a.vdim = (int) mx.integer("vdim", a.dim);
+    a.scale = (float) mx.number("scale", a.dim > 0 ? 1.0 / std::sqrt((double) a.dim) : 1.0);
+    a.gated = 0;
+    a.sink = 1;
+    L.has_sink = true;
+    L.att_prep = true;
+    L.att_qkn = QKN_HEAD_UNIT;
+    L.att_rot_layout = ROT_HALVES;
+    if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dim <= 0 || a.vdim <= 0 || a.vdim > 512) { err = "attention sizes"; return PB200_EINVAL; }
+    const Json * mk = mx.get("mask");
+    if (mk && mk->kind == Json::OBJ) { err = "attention layers are causal without a mask"; return PB200_ENOTSUP; }
+    L.att_rot_dims = 0;
+    const Json * rot = mx.get("rot");
+    if (rot && rot->kind == Json::OBJ) {
+        L.att_rot_dims = (int) rot->integer("dims", a.dim);
+        if (L.att_rot_dims < 0 || L.att_rot_dims > a.dim || L.att_rot_dims % 2 || !(rot->number("base", 10000.0) > 0.0)) { err = "rotated dimensions"; return PB200_EINVAL; }
+        rotary_table(*rot, L.att_rot_dims, L.rot_freq.preset, L.att_rot_mag);
+    } else {
+        L.rot_freq.preset.assign(1, 0.f);
+    }
+    const Json * from = mx.get("kv_from");
+    if (from && from->kind == Json::NUM) {
+        a.own_kv = 0;
+        L.kv_from = (int) from->num;
+        if (L.kv_from < 0 || L.kv_from >= (int) ll.layers.size()) { err = "kv_from must name an earlier layer"; return PB200_EINVAL; }
+        const LLayer & S = ll.layers[(size_t) L.kv_from];
+        if (S.kind != MIX_ATTENTION || !S.att.own_kv || S.att.kv_heads != a.kv_heads || S.att.dim != a.dim || S.att.vdim != a.vdim) {
+            err = "kv_from: the named layer has no keys and values of this shape";
+            return PB200_EINVAL;
+        }
+    }
+    return 0;
+}
+static int ludusun_latent(const Json & mx, LLayer & L, std::string & err) {
+    L.kind = MIX_LATENT;
+    LatentParams & a = L.lat;
+    a.heads = (int) mx.integer("heads", 0);
+    a.dim = (int) mx.integer("dim", 0);
+    a.vdim = (int) mx.integer("vdim", a.dim);
+    a.kv_rank = (int) mx.integer("kv_rank", 0);
+    a.q_rank = (int) mx.integer("q_rank", 0);
+    a.scale = (float) mx.number("scale", a.dim > 0 ? 1.0 / std::sqrt((double) a.dim) : 1.0);
+    a.rot_dim = a.rot_dims = 0;
+    a.gate_mode = 1;
+    L.rot_freq.preset.assign(1, 0.f);
+    if (const Json * mk = mx.get("mask"))
+        if (mk->kind == Json::OBJ) a.window = (int) std::min<long long>(mk->integer("size", 0), 1 << 30);
+    if (a.heads <= 0 || a.dim <= 0 || a.vdim <= 0 || a.vdim > 512 || a.kv_rank <= 0 || a.kv_rank > 512 || a.q_rank <= 0 || a.window < 0) { err = "latent attention sizes"; return PB200_EINVAL; }
+    return 0;
+}
+static int ludusun_parallel(const Json & mx, LLayer & L, std::string & err) {
+    const Json * jl = mx.get("left"), * jr = mx.get("right");
+    if (!jl || jl->kind != Json::OBJ || !jr || jr->kind != Json::OBJ) { err = "a dual mixer needs left and right"; return PB200_EINVAL; }
+    L.kind = MIX_DUAL;
+    DualMix & d = L.dual;
+    AttnParams & a = L.att;
+    a.heads = (int) jl->integer("heads", 0);
+    a.kv_heads = (int) jl->integer("kv_heads", a.heads);
+    a.dim = (int) jl->integer("dim", 0);
+    a.vdim = (int) jl->integer("vdim", a.dim);
+    a.scale = (float) jl->number("scale", a.dim > 0 ? 1.0 / std::sqrt((double) a.dim) : 1.0);
+    a.gated = 0;
+    a.tied_v = 1;
+    if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dim <= 0 || a.dim > 512 || a.vdim != a.dim) { err = "attention sizes (a key is its own value)"; return PB200_EINVAL; }
+    L.rot_freq.preset.assign(1, 0.f);
+    d.biased = true;
+    d.gate_mode = 2;
+    d.join = JOIN_SCALED_SUM;
+    d.left_scale = (float) mx.number("left_scale", 1.0);
+    d.right_scale = (float) mx.number("right_scale", 1.0);
+    const Json * qt = jl->get("q_temp");
+    if (qt && qt->kind == Json::OBJ) {
+        d.q_temp_coef = (float) qt->number("coef", 0.0);
+        d.q_temp_every = (float) qt->number("every", 0.0);
+        if (!(d.q_temp_every > 0.f)) { err = "query temperature"; return PB200_EINVAL; }
+    }
+    d.rec = REC_DELTA_CH;
+    d.r_gate_act = 0;
+    GatedLinParams & rp = d.rp;
+    rp.heads = (int) jr->integer("heads", 0);
+    rp.qk_heads = (int) jr->integer("kv_heads", rp.heads);
+    rp.dim = (int) jr->integer("dim", 0);
+    rp.vdim = (int) jr->integer("vdim", rp.dim);
+    rp.delta = rp.decay_per_channel = 1;
+    d.taps = d.taps_r = (int) jr->integer("conv", 0);
+    d.a_rank = (int) jr->integer("decay_rank", 0);   // 0: the tensors tell
+    d.g_rank = (int) jr->integer("gate_rank", 0);
+    if (rp.heads <= 0 || rp.qk_heads <= 0 || rp.heads % rp.qk_heads || rp.dim <= 0 || rp.vdim <= 0 || rp.dim > 512 || d.taps < 1 || d.taps > 64 || d.a_rank < 0 || d.g_rank < 0) {
+        err = "recurrence sizes";
+        return PB200_EINVAL;
+    }
+    // columns of the fused projection; the inner values of the two maps join at the end
+    const int QD = a.heads * a.dim, KD = a.kv_heads * a.dim, RQ = rp.qk_heads * rp.dim, RV = rp.heads * rp.vdim;
+    int c = 0;
+    d.c_q = c; c += QD;
+    d.c_k = d.c_v = c; c += KD;
+    d.c_g = c; c += QD;
+    d.conv_0 = d.c_rq = c; c += RQ;
+    d.c_rk = c; c += RQ;
+    d.c_rv = c; c += RV;
+    d.conv_ch = c - d.conv_0;
+    d.conv_l = 0;
+    d.c_rb = c; c += rp.heads;
+    d.cols = c;
+    L.dconv_w.n_parts = 3;
+    L.qk_bias.n_parts = 2;
+    return 0;
+}
+static int ludusun_configure(const Json & cfg, LayerList & ll, std::string & err) {
+    ll.frame = FRAME_PRERMS;
+    ll.tied_head = true;
+    ll.width = (int) cfg.integer("width", 0);
+    ll.vocab = (int) cfg.integer("vocab", 0);
+    ll.logit_scale = 1.f;
+    ll.resid_mult = 1.f;
+    ll.logit_softcap = (float) cfg.number("logit_softcap", 0.0);
+    if (const Json * em = cfg.get("embedding"))
+        if (em->kind == Json::OBJ) ll.embed_scale = (float) em->number("scale", 1.0);
+    if (const Json * nrm = cfg.get("norm")) ll.eps = (float) nrm->number("eps", 1e-6);
+    const Json * layers = cfg.get("layers");
+    if (ll.width <= 0 || ll.vocab <= 0 || !layers || layers->kind != Json::ARR || layers->arr.empty()) { err = "width, vocab and layers are required"; return PB200_EINVAL; }
+    for (const Json & jl : layers->arr) {
+        LLayer L;
+        const std::string type = jl.string("type");
+        const Json * mx = jl.get("mixer");
+        if (!mx || mx->kind != Json::OBJ) { err = "layer without mixer"; return PB200_EINVAL; }
+        int rc = PB200_ENOTSUP;
+        if (type == "attention") rc = ludusun_attention(*mx, ll, L, err);
+        else if (type == "latent_attention") rc = ludusun_latent(*mx, L, err);
+        else if (type == "parallel") rc = ludusun_parallel(*mx, L, err);
+        else err = "unknown layer type '" + type + "'";
+        if (rc) return rc;
+        const Json * mlp = jl.get("mlp");
+        if (mlp && mlp->kind == Json::OBJ) {
+            const std::string kind = mlp->string("kind", "dense");
+            if (kind != "dense") { err = "unknown feed-forward kind '" + kind + "'"; return PB200_ENOTSUP; }
+            L.ff_kind = FF_SILU;
+            L.ff = (int) mlp->integer("ff", 0);
+            if (L.ff <= 0) { err = "feed-forward size"; return PB200_EINVAL; }
+        }
+        LRun r;
+        r.layer = (int) ll.layers.size();
+        ll.runs.push_back(r);
+        ll.layers.push_back(std::move(L));
+    }
+    return 0;
+}
+
+static bool ludusun_resolve(LayerList & ll, const std::string & name, TensorPlace & o) {
+    const int64_t W = ll.width;
+    auto mat = [&](DenseW & m, int64_t row0, int64_t rows, int64_t cols, int part) { o.mat = &m; o.row0 = row0; o.rows = rows; o.cols = cols; o.part = part; return true; };
+    auto vec = [&](VecF & v, int64_t n) { o.vec = &v; o.n = n; return true; };
+    auto norm = [&](VecF & v, int64_t n) { o.add = 1.f; return vec(v, n); };   // stored around zero: the factor is 1 + w
+    // n numbers at entry v0 of a vector that several tensors fill
+    auto piece = [&](VecF & v, int64_t v0, int64_t n, int part) { o.part = part; o.v0 = v0; o.vrows = 1; o.vcols = o.vld = n; return vec(v, n); };
+    if (name == "embed") return mat(ll.embed, 0, ll.vocab, W, 0);
+    if (name == "final.norm") return norm(ll.final_norm, W);
+    int il = -1, used = 0;
+    if (sscanf(name.c_str(), "l%d.%n", &il, &used) != 1 || used <= 0 || il < 0 || il >= (int) ll.layers.size()) return false;
+    LLayer & L = ll.layers[(size_t) il];
+    const std::string w = name.substr((size_t) used);
+    if (w == "norm1") return norm(L.norm1, W);
+    if (L.ff > 0) {
+        if (w == "norm2") return norm(L.norm2, W);
+        if (w == "mlp.gate") return mat(L.gateup, 0, L.ff, W, 0);
+        if (w == "mlp.up") return mat(L.gateup, L.ff, L.ff, W, 1);
+        if (w == "mlp.down") return mat(L.down, 0, W, L.ff, 0);
+    }
+    if (L.kind == MIX_ATTENTION) {
+        const AttnParams & a = L.att;
+        const int64_t QD = (int64_t) a.heads * a.dim, KD = (int64_t) a.kv_heads * a.dim, VD = (int64_t) a.kv_heads * a.vdim;
+        if (w == "mix.q") return mat(L.qkvg, 0, QD, W, 0);
+        if (w == "mix.k") return a.own_kv && mat(L.qkvg, QD, KD, W, 1);
+        if (w == "mix.v") return a.own_kv && mat(L.qkvg, QD + KD, VD, W, 2);
+        if (w == "mix.sink") return vec(L.sink, a.heads);
+        if (w == "mix.o") return mat(L.out, 0, W, (int64_t) a.heads * a.vdim, 0);
+        return false;
+    }
+    if (L.kind == MIX_LATENT) {
+        const LatentParams & a = L.lat;
+        const int64_t VD = (int64_t) a.heads * a.vdim;
+        if (w == "mix.dq") return mat(L.lproj, 0, a.q_rank, W, 0);
+        if (w == "mix.g") return mat(L.lproj, latent_q_cols(a), latent_gate_cols(a), W, 1);
+        if (w == "mix.dkv") return mat(L.lproj, latent_kv_col(a), a.kv_rank, W, 2);
+        if (w == "mix.dq.norm") return vec(L.dq_norm, a.q_rank);
+        if (w == "mix.dkv.norm") return vec(L.dkv_norm, a.kv_rank);
+        if (w == "mix.uq") return mat(L.uq, 0, (int64_t) a.heads * a.dim, a.q_rank, 0);
+        if (w == "mix.uk") return mat(L.ukv, 0, (int64_t) a.heads * a.dim, a.kv_rank, 0);
+        if (w == "mix.uv") return mat(L.ukv, (int64_t) a.heads * a.dim, VD, a.kv_rank, 1);
+        if (w == "mix.o") return mat(L.out, 0, W, VD, 0);
+        return false;
+    }
+    DualMix & d = L.dual;
+    const AttnParams & a = L.att;
+    const GatedLinParams & rp = d.rp;
+    const int64_t QD = (int64_t) a.heads * a.dim, KD = (int64_t) a.kv_heads * a.dim, RQ = (int64_t) rp.qk_heads * rp.dim, RD = (int64_t) rp.heads * rp.dim,
+                  RV = (int64_t) rp.heads * rp.vdim;
+    // columns [col0, col0 + cols) of the output product over [left | right]
+    auto out = [&](int64_t col0, int64_t cols, int part) { o.col0 = col0; return mat(L.out, 0, W, cols, part); };
+    // the two tensors of a low-rank map; whichever comes first tells the inner size
+    auto down = [&](DenseW & m, int & rank) { o.size = &rank; o.size_unit = W; return mat(m, 0, rank, W, 0); };
+    auto up = [&](VecF & v, int64_t rows, int & rank) { o.size = &rank; o.size_unit = rows; return vec(v, rows * rank); };
+    if (w.compare(0, 9, "mix.left.") == 0) {
+        const std::string f = w.substr(9);
+        if (f == "q") return mat(L.qkvg, d.c_q, QD, W, 0);
+        if (f == "k") return mat(L.qkvg, d.c_k, KD, W, 1);
+        if (f == "g") return mat(L.qkvg, d.c_g, QD, W, 2);
+        if (f == "q.b") return piece(L.qk_bias, d.c_q, QD, 0);
+        if (f == "k.b") return piece(L.qk_bias, d.c_k, KD, 1);
+        if (f == "o") return out(0, QD, 0);
+        return false;
+    }
+    if (w.compare(0, 10, "mix.right.") == 0) {
+        const std::string f = w.substr(10);
+        if (f == "q") return mat(L.qkvg, d.c_rq, RQ, W, 3);
+        if (f == "k") return mat(L.qkvg, d.c_rk, RQ, W, 4);
+        if (f == "v") return mat(L.qkvg, d.c_rv, RV, W, 5);
+        if (f == "b") return mat(L.qkvg, d.c_rb, rp.heads, W, 6);
+        if (f == "q.conv") return piece(L.dconv_w, 0, RQ * d.taps, 0);
+        if (f == "k.conv") return piece(L.dconv_w, RQ * d.taps, RQ * d.taps, 1);
+        if (f == "v.conv") return piece(L.dconv_w, 2 * RQ * d.taps, RV * d.taps, 2);
+        if (f == "a1") return down(L.ra1, d.a_rank);
+        if (f == "a2") return up(L.ra2, RD, d.a_rank);
+        if (f == "g1") return down(L.rg1, d.g_rank);
+        if (f == "g2") return up(L.rg2, RV, d.g_rank);
+        if (f == "A_log") return vec(L.A_log, rp.heads);
+        if (f == "dt_bias") return vec(L.dt_bias, RD);
+        if (f == "norm") { o.vrows = 1; o.vcols = o.vld = o.vrep = rp.vdim; o.repeat = rp.heads; return vec(L.onorm, rp.vdim); }   // all heads share it
+        if (f == "o") return out(QD, RV, 1);
+    }
+    return false;
+}
+
 static const ArchEntry g_archs[] = {
     {"llama", ARCH_KQUANT, 0, nullptr, nullptr},
     {"qwen2", ARCH_KQUANT, 2, nullptr, nullptr},
@@ -1153,6 +1410,7 @@ static const ArchEntry g_archs[] = {
     {"Sapudra", ARCH_LAYERS, 0, sapudra_configure, sapudra_resolve},
     {"Zevedra", ARCH_LAYERS, 0, zevedra_configure, zevedra_resolve},
     {"Ruvuvik", ARCH_LAYERS, 0, ruvuvik_configure, ruvuvik_resolve},
+    {"Ludusun", ARCH_LAYERS, 0, ludusun_configure, ludusun_resolve},
 };
 int arch_count() { return (int) (sizeof(g_archs) / sizeof(g_archs[0])); }
 const ArchEntry * arch_at(int i) { return (i >= 0 && i < arch_count()) ? &g_archs[i] : nullptr; }
@@ -1171,7 +1429,7 @@ template <typename FM, typename FV>
 static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
     const int64_t W = ll.width;
     fm(ll.embed, (int64_t) ll.vocab, W, 1);
-    fm(ll.head, (int64_t) ll.vocab, W, 1);
+    if (!ll.tied_head) fm(ll.head, (int64_t) ll.vocab, W, 1);
     fv(ll.final_norm, W, 0);
     if (ll.frame == FRAME_POSTNORM) { fm(ll.pos_table, (int64_t) ll.max_pos, W, 1); fv(ll.final_norm_bias, W, 1); }
     if (ll.embed_normed) fv(ll.embed_norm, W, 0);
@@ -1189,13 +1447,14 @@ static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
         else if (ll.frame == FRAME_PRENORM) { fv(L.shift, W, 5); fv(L.dwa, il + 2, 6); }
         il++;
         if (L.kind == MIX_ATTENTION) {
-            fm(L.qkvg, attn_qkvg_cols(L.att), W, L.att.gated ? 4 : 3);
+            fm(L.qkvg, attn_qkvg_cols(L.att), W, (L.att.own_kv ? 3 : 1) + (L.att.gated ? 1 : 0));
             if (L.qk_norm) { fv(L.q_norm, L.att.dim, 0); fv(L.k_norm, L.att.dim, 0); }
             if (L.att_prep) {
                 if (L.att_qkn == QKN_WHOLE_WEIGHT) { fv(L.q_norm, (int64_t) L.att.heads * L.att.dim, 0); fv(L.k_norm, (int64_t) L.att.kv_heads * L.att.dim, 0); }
                 fv(L.rot_freq, (int64_t) L.rot_freq.preset.size(), 0);
-                fv(L.temp, L.att.heads, 0);
+                if (L.att_temp) fv(L.temp, L.att.heads, 0);
             }
+            if (L.has_sink) fv(L.sink, L.att.heads, 1);
             fm(L.out, W, (int64_t) L.att.heads * L.att.vdim, 1);
         } else if (L.kind == MIX_WKV) {
             const int64_t HD = (int64_t) L.wkv.heads * L.wkv.dim;
@@ -1221,12 +1480,18 @@ static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
             const AttnParams & a = L.att;
             const int64_t OD = (int64_t) a.heads * a.vdim, RQ = (int64_t) d.rp.qk_heads * d.rp.dim, RV = (int64_t) d.rp.heads * d.rp.vdim;
             fm(L.qkvg, d.cols, W, d.rec == REC_DELTA ? 10 : 7);
+            if (d.biased) fv(L.qk_bias, d.cols, 1);
+            if (d.rec == REC_DELTA_CH) {
+                fm(L.ra1, d.a_rank, W, 1); fv(L.ra2, (int64_t) d.rp.heads * d.rp.dim * d.a_rank, 7);
+                fm(L.rg1, d.g_rank, W, 1); fv(L.rg2, RV * d.g_rank, 7);
+            }
             fv(L.rot_freq, (int64_t) L.rot_freq.preset.size(), 0);
             if (d.v_rot) fv(L.vrot_freq, (int64_t) L.vrot_freq.preset.size(), 0);
             if (d.taps > 0) fv(L.dconv_w, (int64_t) d.conv_ch * d.taps, 2);
             if (d.qk_norm == QKN_WHOLE_WEIGHT) { fv(L.q_norm, (int64_t) a.heads * a.dim, 0); fv(L.k_norm, (int64_t) a.kv_heads * a.dim, 0); }
             fv(L.onorm, RV, 0);
             if (d.rec == REC_DELTA) { fv(L.A_log, d.rp.heads, 4); fv(L.dt_bias, d.rp.heads, 3); }
+            else if (d.rec == REC_DELTA_CH) { fv(L.A_log, d.rp.heads, 4); fv(L.dt_bias, (int64_t) d.rp.heads * d.rp.dim, 3); }
             else { fv(L.f_bias, RQ, 1); fv(L.f_lower, RQ, 5); }
             if (d.join == JOIN_SCALED_SUM) {
                 fm(L.out, W, OD + RV, 2);
@@ -1236,7 +1501,7 @@ static void for_each_param(LayerList & ll, FM && fm, FV && fv) {
             }
         } else {
             const LatentParams & a = L.lat;
-            fm(L.lproj, latent_proj_cols(a), W, 1 + (a.gated ? 1 : 0) + (a.own_kv ? 1 : 0));
+            fm(L.lproj, latent_proj_cols(a), W, 1 + (a.gate_mode ? 1 : 0) + (a.own_kv ? 1 : 0));
             if (a.q_rank > 0) fv(L.dq_norm, a.q_rank, 0);
             if (a.own_kv) fv(L.dkv_norm, a.kv_rank, 0);
             fv(L.rot_freq, (int64_t) L.rot_freq.preset.size(), 0);
@@ -1279,7 +1544,7 @@ static int ll_alloc_params(pb200_model * m) {
     for_each_param(
         ll,
         [&](DenseW & d, int64_t N, int64_t K, int parts) {
-            if (rc || d.data) return;
+            if (rc || d.data || N <= 0) return;
             d.N = N; d.K = K; d.filled.assign((size_t) parts, 0);
             const size_t b = (size_t) N * K * esize(ll.ctype);
             rc = m->alloc(&d.data, b + 16);
@@ -1403,6 +1668,10 @@ int ll_synth(pb200_model * m, uint64_t seed) {
     int rc = 0;
     for (LLayer & L : ll.layers)
         if (L.kind == MIX_WKV && L.decay_rank == 0) L.decay_rank = std::max(8, ll.width / 64);   // no tensor will tell
+        else if (L.kind == MIX_DUAL && L.dual.rec == REC_DELTA_CH) {
+            if (L.dual.a_rank == 0) L.dual.a_rank = L.dual.rp.dim;
+            if (L.dual.g_rank == 0) L.dual.g_rank = L.dual.rp.vdim;
+        }
     CK(ll_alloc_params(m));
     for_each_param(
         ll,
@@ -1429,19 +1698,53 @@ int ll_synth(pb200_model * m, uint64_t seed) {
     return (int) cudaStreamSynchronize(m->stream);
 }
 
+// the down-projections of a dual mixer's low-rank maps become the last rows of its fused projection (their sizes come with the tensors, so they
+// arrive in matrices of their own)
+static int dual_join_lowrank(pb200_model * m, LLayer & L) {
+    LayerList & ll = *m->ll;
+    DualMix & d = L.dual;
+    const size_t row = (size_t) ll.width * esize(ll.ctype);
+    const int64_t base = d.cols, cols = base + d.a_rank + d.g_rank;
+    void * w = nullptr;
+    CK(m->alloc(&w, (size_t) cols * row + 16));
+    CK(cudaMemcpy(w, L.qkvg.data, (size_t) base * row, cudaMemcpyDeviceToDevice));
+    CK(cudaMemcpy((uint8_t *) w + (size_t) base * row, L.ra1.data, (size_t) d.a_rank * row, cudaMemcpyDeviceToDevice));
+    CK(cudaMemcpy((uint8_t *) w + (size_t) (base + d.a_rank) * row, L.rg1.data, (size_t) d.g_rank * row, cudaMemcpyDeviceToDevice));
+    float * bias = nullptr;
+    if (d.biased) {
+        CK(m->alloc((void **) &bias, (size_t) cols * 4));
+        CK(cudaMemset(bias, 0, (size_t) cols * 4));
+        CK(cudaMemcpy(bias, L.qk_bias.data, (size_t) base * 4, cudaMemcpyDeviceToDevice));
+    }
+    for (void * p : {L.qkvg.data, L.ra1.data, L.rg1.data, (void *) L.qk_bias.data})
+        if (p) {
+            m->allocs.erase(std::remove(m->allocs.begin(), m->allocs.end(), p), m->allocs.end());
+            CK(cudaFree(p));
+        }
+    L.qkvg.data = w; L.qkvg.N = cols;
+    L.ra1 = L.rg1 = DenseW();
+    L.qk_bias.data = bias;
+    d.c_ra = (int) base;
+    d.c_rg = (int) base + d.a_rank;
+    d.cols = (int) cols;
+    return 0;
+}
+
 int ll_finalize(pb200_model * m) {
     LayerList & ll = *m->ll;
     if (m->finalized) return 0;
     cudaSetDevice(m->device);
     bool complete = true;
     for_each_param(
-        ll, [&](DenseW & d, int64_t, int64_t, int) { for (uint8_t f : d.filled) complete = complete && f; },
+        ll, [&](DenseW & d, int64_t, int64_t, int) { complete = complete && d.data; for (uint8_t f : d.filled) complete = complete && f; },
         [&](VecF & v, int64_t, int) {
             if (!v.data) complete = false;   // a size that no tensor has settled
             else if (v.parts.empty()) complete = complete && v.filled;
             else for (uint8_t f : v.parts) complete = complete && f;
         });
     if (!complete) return PB200_ESTATE;
+    for (LLayer & L : ll.layers)
+        if (L.kind == MIX_DUAL && L.dual.rec == REC_DELTA_CH) CK(dual_join_lowrank(m, L));
     // state arena layout of one slot
     int64_t off = 0;
     ll.ctx_limited = false;
@@ -1452,14 +1755,15 @@ int ll_finalize(pb200_model * m) {
         if (L.kind == MIX_DECAY) {
             off += (int64_t) L.dec.heads * L.dec.dim * L.dec.vdim;
         } else if (L.kind == MIX_LATENT) {
-            L.lat.cache_rows = ll.n_ctx;
-            ll.ctx_limited = true;
-            if (L.lat.own_kv) off += (int64_t) ll.n_ctx * latent_row(L.lat);
+            L.lat.cache_rows = attn_cache_rows(L.lat.window, 0, ll.n_ctx);
+            if (L.lat.cache_rows >= ll.n_ctx) ll.ctx_limited = true;
+            if (L.lat.own_kv) off += (int64_t) L.lat.cache_rows * latent_row(L.lat);
             else r.state_off = ll.runs[(size_t) L.kv_from].state_off;   // FRAME_PRENORM: run i is layer i
         } else if (L.kind == MIX_ATTENTION || L.kind == MIX_DUAL) {
             L.att.cache_rows = L.att.chunk > 0 ? std::min(L.att.chunk, ll.n_ctx) : attn_cache_rows(L.att.window, L.att.keep_first, ll.n_ctx);
             if (L.att.cache_rows >= ll.n_ctx) ll.ctx_limited = true;
-            off += (int64_t) L.att.cache_rows * L.att.kv_heads * (L.att.dim + L.att.vdim);
+            if (!L.att.own_kv) r.state_off = ll.runs[(size_t) L.kv_from].state_off;   // the named layer's rows (run i is layer i where layers read others)
+            else off += (int64_t) L.att.cache_rows * (L.att.kv_heads * L.att.dim + attn_v_row(L.att));
             if (L.kind == MIX_DUAL) {   // then the convolution's last inputs and the recurrence's state
                 const DualMix & d = L.dual;
                 off = (off + 3) / 4 * 4;
@@ -1589,6 +1893,7 @@ static int ll_reserve(pb200_model * m, int T, int nW, int nE) {
                 maxact = std::max(maxact, OD + RV);
                 maxact2 = std::max(maxact2, RV);
                 maxbig = std::max<int64_t>(maxbig, d.cols);
+                if (d.rec == REC_DELTA_CH) maxb3 = std::max(maxb3, (int64_t) d.rp.heads * d.rp.dim + RV);   // decays, then gate logits
                 maxch = std::max<int64_t>(maxch, d.conv_ch);
                 maxinner = std::max(maxinner, RV);
                 maxb2 = std::max(maxb2, OD);                       // the attention result before it is turned back
@@ -1596,7 +1901,7 @@ static int ll_reserve(pb200_model * m, int T, int nW, int nE) {
             } else {
                 const LatentParams & a = L.lat;
                 const int64_t H = a.heads;
-                maxact = std::max(maxact, H * a.vdim);
+                maxact = std::max(maxact, std::max<int64_t>(H * a.vdim, a.kv_rank));
                 maxact2 = std::max<int64_t>(maxact2, std::max(a.q_rank, a.kv_rank));
                 maxbig = std::max<int64_t>(maxbig, latent_proj_cols(a));
                 maxb2 = std::max(maxb2, H * (a.dim + a.rot_dim));
@@ -1726,7 +2031,7 @@ static int mix_attention(pb200_model * m, const BatchView & b, bool prefill, con
     const int T = b.n_tokens, W = ll.width, ct = ll.ctype;
     const AttnParams & a = L.att;
     const int C = attn_qkvg_cols(a);
-    float * sbase = ll.state + r.state_off;
+    float * sbase = ll.state + r.state_off;       // this layer's rows, or those of the layer it reads
     CAT(CAT_DENSE);
     CK(launch_dense(ct, ll.act, W, L.qkvg.data, W, ll.big, C, T, C, W, nullptr, nullptr, 0, 1.f, st));
     float * kc = sbase, * vc = sbase + (int64_t) a.cache_rows * a.kv_heads * a.dim;
@@ -1734,14 +2039,21 @@ static int mix_attention(pb200_model * m, const BatchView & b, bool prefill, con
     if (L.att_prep) {   // norm over the whole projections, rotation, temperatures and the cache store in one launch
         AttnPrep pr;
         pr.norm = L.att_qkn; pr.wq = L.q_norm.data; pr.wk = L.k_norm.data; pr.eps = ll.eps;
-        pr.rot_dims = L.att_rot_dims; pr.rot_layout = L.att_rot_layout; pr.rot_freq = L.rot_freq.data;
+        pr.rot_dims = L.att_rot_dims; pr.rot_layout = L.att_rot_layout; pr.rot_freq = L.rot_freq.data; pr.rot_mag = L.att_rot_mag;
         pr.q_scale = L.temp.data;
         float * k = ll.big + a.heads * a.dim, * v = k + a.kv_heads * a.dim;
         CK(launch_attn_prep_store(ll.big, C, k, C, v, C, b, a, pr, kc, vc, ll.slot_floats, st));
     } else if (L.qk_norm) CK(launch_attn_qknorm_kv_store(ll.big, b, a, L.q_norm.data, L.k_norm.data, ll.eps, kc, vc, ll.slot_floats, st));
     else CK(launch_attn_kv_store(ll.big, b, a, kc, vc, ll.slot_floats, st));
-    if (prefill) CK(launch_attn_window_prefill(ll.big, b, a, ll.act, ct, st));
-    else CK(launch_attn_window_decode(ll.big, b, a, kc, vc, ll.slot_floats, ll.act, ct, st, ll.lat_part));
+    AttnIO io = attn_io_fused(ll.big, a);
+    io.sink = L.has_sink ? L.sink.data : nullptr;
+    if (prefill && !a.own_kv) {   // a prompt starts at position 0 and the other layer's cache holds all of it
+        io.k = kc; io.ldk = io.k_row;
+        io.v = vc; io.ldv = io.v_row;
+        io.kv_slot = b.slot; io.kv_slot_stride = ll.slot_floats;
+    }
+    if (prefill) CK(launch_attn_prefill_io(io, b, a, ll.act, ct, st));
+    else CK(launch_attn_decode_io(io, b, a, kc, vc, ll.slot_floats, ll.act, ct, st, ll.lat_part));
     CAT(CAT_DENSE);
     return launch_dense(ct, ll.act, (int64_t) a.heads * a.vdim, L.out.data, (int64_t) a.heads * a.vdim, out, W, T, W, a.heads * a.vdim, nullptr, resid, W, 1.f, st);
 }
@@ -1786,7 +2098,7 @@ static int mix_latent(pb200_model * m, const BatchView & b, bool prefill, const 
     const LatentParams & a = L.lat;
     const int H = a.heads, C = latent_proj_cols(a), DQ = a.dim + a.rot_dim, VD = H * a.vdim, R = a.kv_rank, RW = latent_row(a), KV = H * a.dim + VD;
     float * cache = ll.state + r.state_off;       // this layer's rows, or those of the layer it reads
-    const float * gate = a.gated ? ll.big + latent_q_cols(a) : nullptr;
+    const float * gate = a.gate_mode ? ll.big + latent_q_cols(a) : nullptr;
     const float * sink = L.has_sink ? L.sink.data : nullptr;
     const void * wuk = L.ukv.data, * wuv = (const uint8_t *) L.ukv.data + (size_t) H * a.dim * R * esize(ct);
     const bool direct_q = a.q_rank <= 0;          // the fused projection ends in the queries themselves
@@ -1795,9 +2107,11 @@ static int mix_latent(pb200_model * m, const BatchView & b, bool prefill, const 
     CAT(CAT_DENSE);
     CK(launch_dense(ct, ll.act, W, L.lproj.data, W, ll.big, C, T, C, W, nullptr, nullptr, 0, 1.f, st));
     CAT(CAT_LATENT);
-    // a layer with a cache of its own and queries of its own: the batch's latents and key parts leave in the same launch that stores them
-    const bool fused = prefill && a.own_kv && direct_q;
-    CK(launch_latent_prep(ll.big, b, a, L.dq_norm.data, L.dkv_norm.data, L.rot_freq.data, ll.eps, ll.act2, ct, cache, ll.slot_floats, fused ? ll.act2 : nullptr,
+    // a layer with a cache of its own: the batch's latents and key parts leave in the same launch that stores them (the query latent takes
+    // ll.act2, and the mixer's input in ll.act has been read by then)
+    const bool fused = prefill && a.own_kv;
+    void * lat = direct_q ? ll.act2 : ll.act;
+    CK(launch_latent_prep(ll.big, b, a, L.dq_norm.data, L.dkv_norm.data, L.rot_freq.data, ll.eps, ll.act2, ct, cache, ll.slot_floats, fused ? lat : nullptr,
                           fused ? ll.krb : nullptr, prefill, st));
     if (!direct_q) {
         CAT(CAT_DENSE);
@@ -1809,18 +2123,19 @@ static int mix_latent(pb200_model * m, const BatchView & b, bool prefill, const 
     CAT(CAT_LATENT);
     if (prefill) {   // keys and values of the batch, expanded from the cached latents by one product
         if (!direct_q) CK(launch_latent_rope_q(q, ldq, b, a, L.rot_freq.data, st));
-        if (!fused) CK(launch_latent_gather(cache, ll.slot_floats, b, a, ll.act2, ct, ll.krb, st));
+        if (!fused) CK(launch_latent_gather(cache, ll.slot_floats, b, a, lat, ct, ll.krb, st));
         CAT(CAT_DENSE);
-        CK(launch_dense(ct, ll.act2, R, L.ukv.data, R, ll.big3, KV, T, KV, R, nullptr, nullptr, 0, 1.f, st));
+        CK(launch_dense(ct, lat, R, L.ukv.data, R, ll.big3, KV, T, KV, R, nullptr, nullptr, 0, 1.f, st));
         CAT(CAT_ATTN);
         ap.kv_heads = H; ap.dim = DQ; ap.vdim = a.vdim; ap.shared_dim = a.rot_dim;
+        ap.window = a.window;
         ap.sink = sink ? 1 : 0;
         io.sink = sink;
         io.q = q; io.ldq = ldq;
         io.k = ll.big3; io.ldk = KV;
         io.ks = ll.krb; io.ldks = a.rot_dim;
         io.v = ll.big3 + (int64_t) H * a.dim; io.ldv = KV;
-        io.gate = gate; io.ldg = C; io.gate_mode = gate ? 2 : 0;
+        io.gate = gate; io.ldg = C; io.gate_mode = a.gate_mode;
         CK(launch_attn_prefill_io(io, b, ap, ll.act, ct, st));
     } else if (T == b.n_entries && R <= 512) {   // one token per entry: the key up-projection folded into the query, rows split over CTAs
         CK(launch_latent_absorb_q(q, ldq, b, wuk, ct, a, L.rot_freq.data, ll.big3, st));
@@ -1829,7 +2144,7 @@ static int mix_latent(pb200_model * m, const BatchView & b, bool prefill, const 
     } else {         // the same through the shared decode kernel: one key / value head, the key is the whole row, the value its latent part
         CK(launch_latent_absorb_q(q, ldq, b, wuk, ct, a, L.rot_freq.data, ll.big3, st));
         CAT(CAT_ATTN);
-        ap.kv_heads = 1; ap.dim = RW; ap.vdim = R; ap.cache_rows = a.cache_rows;
+        ap.kv_heads = 1; ap.dim = RW; ap.vdim = R; ap.cache_rows = a.cache_rows; ap.window = a.window;
         ap.sink = sink ? 1 : 0;
         io.sink = sink;
         io.q = ll.big3; io.ldq = (int64_t) H * RW;
@@ -1882,43 +2197,51 @@ static int mix_dual(pb200_model * m, const BatchView & b, bool prefill, const LR
     const GatedLinParams & rp = d.rp;
     const int C = d.cols, OD = a.heads * a.vdim, RV = rp.heads * rp.vdim;
     // the slot's arena for this run: K rows | V rows | convolution inputs | recurrent state
-    float * kc = ll.state + r.state_off, * vc = kc + (int64_t) a.cache_rows * a.kv_heads * a.dim;
-    int64_t o = (int64_t) a.cache_rows * a.kv_heads * (a.dim + a.vdim);
+    float * kc = ll.state + r.state_off, * vc = a.tied_v ? kc : kc + (int64_t) a.cache_rows * a.kv_heads * a.dim;
+    int64_t o = (int64_t) a.cache_rows * (a.kv_heads * a.dim + attn_v_row(a));
     o = (o + 3) / 4 * 4;
     float * conv_state = ll.state + r.state_off + o;
     o += (int64_t) std::max(d.taps - 1, 0) * d.conv_ch;
     o = (o + 3) / 4 * 4;
     float * rec_state = ll.state + r.state_off + o;
     CAT(CAT_DENSE);
-    CK(launch_dense(ct, ll.act, W, L.qkvg.data, W, ll.big, C, T, C, W, nullptr, nullptr, 0, 1.f, st));
-    float * src = ll.big;       // where q, k, v of both branches are read from: the projection, or the convolution's output
-    int64_t ld = C;
+    CK(launch_dense(ct, ll.act, W, L.qkvg.data, W, ll.big, C, T, C, W, d.biased ? L.qk_bias.data : nullptr, nullptr, 0, 1.f, st));
+    // where q, k, v of a branch are read from: the projection, or the convolution's output where its columns pass one
+    float * lq = ll.big + d.c_q, * lk = ll.big + d.c_k, * lv = a.tied_v ? lk : ll.big + d.c_v, * rq = ll.big + d.c_rq, * rk = ll.big + d.c_rk, * rv = ll.big + d.c_rv;
+    int64_t ld = C, ldr = C;
     if (d.taps > 0) {
         CAT(CAT_CONV);
-        CK(launch_causal_conv(ll.big, C, b, d.conv_ch, d.taps, L.dconv_w.data, d.conv_l, conv_state, ll.slot_floats, ll.xbc, d.conv_ch, st));
-        src = ll.xbc;
-        ld = d.conv_ch;
+        CK(launch_causal_conv(ll.big + d.conv_0, C, b, d.conv_ch, d.taps, L.dconv_w.data, d.conv_l, conv_state, ll.slot_floats, ll.xbc, d.conv_ch, st));
+        if (d.taps_l > 0) {
+            lq = ll.xbc + d.c_q - d.conv_0; lk = ll.xbc + d.c_k - d.conv_0; lv = ll.xbc + d.c_v - d.conv_0;
+            ld = d.conv_ch;
+        }
+        rq = ll.xbc + d.c_rq - d.conv_0; rk = ll.xbc + d.c_rk - d.conv_0; rv = ll.xbc + d.c_rv - d.conv_0;
+        ldr = d.conv_ch;
     }
     // ---- attention branch ----
     CAT(CAT_ATTN);
     AttnPrep pr;
     pr.norm = d.qk_norm; pr.wq = L.q_norm.data; pr.wk = L.k_norm.data; pr.eps = ll.eps;
     pr.rot_dims = d.rot_dims; pr.rot_layout = d.rot_layout; pr.rot_freq = L.rot_freq.data;
+    pr.q_temp_coef = d.q_temp_coef; pr.q_temp_every = d.q_temp_every;
     pr.v_rot = d.v_rot; pr.v_layout = d.rot_layout; pr.v_freq = d.v_rot ? L.vrot_freq.data : nullptr;
     // one launch prepares both branches: the recurrence's inputs (unit vectors, gates, decays), then the attention inputs and the cache store
     // (PB200_DUAL_UNFUSED: the same steps as the single ops the layers were brought up on, one launch each; for A/B runs and tests)
     static const bool unfused = getenv("PB200_DUAL_UNFUSED") != nullptr;
+    const bool delta = d.rec == REC_DELTA || d.rec == REC_DELTA_CH;
+    float * ra = d.rec == REC_DELTA ? ll.big + d.c_ra : nullptr;   // decays per head; those per channel come from a map of their own
     if (unfused) {
-        if (d.rec == REC_DELTA)
-            CK(launch_delta_prep(src + d.c_rq, ld, src + d.c_rk, ld, ll.big + d.c_rb, C, ll.big + d.c_ra, C, L.A_log.data, L.dt_bias.data, rp.qk_heads, rp.heads, rp.dim, T, st));
-        else CK(launch_hgrn2_prep(src + d.c_rq, ld, src + d.c_rk, ld, L.f_bias.data, L.f_lower.data, rp.qk_heads * rp.dim, T, st));
-        CK(launch_attn_prep_store(src + d.c_q, ld, src + d.c_k, ld, src + d.c_v, ld, b, a, pr, kc, vc, ll.slot_floats, st));
-    } else if (d.rec == REC_DELTA)
-        CK(launch_dual_prep_store(0, src + d.c_rq, ld, src + d.c_rk, ld, ll.big + d.c_rb, C, ll.big + d.c_ra, C, L.A_log.data, L.dt_bias.data, rp.qk_heads, rp.heads,
-                                  rp.dim, src + d.c_q, ld, src + d.c_k, ld, src + d.c_v, ld, b, a, pr, kc, vc, ll.slot_floats, st));
+        if (delta)
+            CK(launch_delta_prep(rq, ldr, rk, ldr, ll.big + d.c_rb, C, ra, C, L.A_log.data, L.dt_bias.data, rp.qk_heads, rp.heads, rp.dim, T, st));
+        else CK(launch_hgrn2_prep(rq, ldr, rk, ldr, L.f_bias.data, L.f_lower.data, rp.qk_heads * rp.dim, T, st));
+        CK(launch_attn_prep_store(lq, ld, lk, ld, lv, ld, b, a, pr, kc, vc, ll.slot_floats, st));
+    } else if (delta)
+        CK(launch_dual_prep_store(0, rq, ldr, rk, ldr, ll.big + d.c_rb, C, ra, C, L.A_log.data, L.dt_bias.data, rp.qk_heads, rp.heads, rp.dim, lq, ld, lk, ld, lv, ld, b,
+                                  a, pr, kc, vc, ll.slot_floats, st));
     else
-        CK(launch_dual_prep_store(1, src + d.c_rq, ld, src + d.c_rk, ld, nullptr, 0, nullptr, 0, L.f_bias.data, L.f_lower.data, rp.qk_heads, rp.heads, rp.dim,
-                                  src + d.c_q, ld, src + d.c_k, ld, src + d.c_v, ld, b, a, pr, kc, vc, ll.slot_floats, st));
+        CK(launch_dual_prep_store(1, rq, ldr, rk, ldr, nullptr, 0, nullptr, 0, L.f_bias.data, L.f_lower.data, rp.qk_heads, rp.heads, rp.dim, lq, ld, lk, ld, lv, ld, b, a,
+                                  pr, kc, vc, ll.slot_floats, st));
     const bool sum = d.join == JOIN_SCALED_SUM;
     // ---- recurrent branch: on the second stream beside the attention branch, unless every launch is being timed ----
     static const bool one_stream = getenv("PB200_ONE_STREAM") != nullptr;   // A/B: both branches in a row on one stream
@@ -1934,30 +2257,44 @@ static int mix_dual(pb200_model * m, const BatchView & b, bool prefill, const LR
         CK(cudaEventRecord(ll.ev_fork, st));
         CK(cudaStreamWaitEvent(rst, ll.ev_fork, 0));
     }
+    const float * r_gate = d.rec == REC_DELTA ? ll.big + d.c_rg : nullptr;   // gate logits of the recurrence's result
+    int64_t ldrg = C;
+    if (d.rec == REC_DELTA_CH) {   // decays per channel and gate logits from the inner values at the end of the projection
+        CAT(CAT_CONV);
+        LowrankMaps mp;
+        mp.za = ll.big + d.c_ra; mp.zg = ll.big + d.c_rg; mp.ldu = C;
+        mp.wa = L.ra2.data; mp.wg = L.rg2.data; mp.ra = d.a_rank; mp.rg = d.g_rank;
+        mp.A_log = L.A_log.data; mp.dt_bias = L.dt_bias.data;
+        mp.heads = rp.heads; mp.dim = rp.dim; mp.gate_cols = RV;
+        mp.ldd = mp.ldg = ldrg = (int64_t) rp.heads * rp.dim + RV;
+        mp.decay = ll.big3; mp.gate = ll.big3 + (int64_t) rp.heads * rp.dim;
+        r_gate = mp.gate;
+        CK(launch_lowrank_maps(mp, T, rst));
+    }
     CAT(CAT_SCAN);
     GatedLinIO gi;
-    gi.q = src + d.c_rq; gi.ldq = ld;
-    gi.v = src + d.c_rv; gi.ldv = ld;
-    if (d.rec == REC_DELTA) {
-        gi.k = src + d.c_rk; gi.ldk = ld;
-        gi.decay = ll.big + d.c_ra; gi.ldd = C;
+    gi.q = rq; gi.ldq = ldr;
+    gi.v = rv; gi.ldv = ldr;
+    if (delta) {
+        gi.k = rk; gi.ldk = ldr;
+        gi.decay = ra; gi.ldd = C;
+        if (d.rec == REC_DELTA_CH) { gi.decay = ll.big3; gi.ldd = ldrg; }
         gi.beta = ll.big + d.c_rb; gi.ldb = C;
     } else {
-        gi.decay = src + d.c_rk; gi.ldd = ld;
+        gi.decay = rk; gi.ldd = ldr;
     }
     CK(launch_gated_linattn(gi, b, rp, rec_state, ll.slot_floats, ll.yssm, rst));
     if (!sum) {   // every head by its own root mean square with the weight all heads share -> operand of the branch's own output product
         CAT(CAT_NORM);
-        CK(launch_norm_gate(ll.yssm, d.rec == REC_DELTA ? ll.big + d.c_rg : nullptr, C, rp.heads, L.onorm.data, d.rec == REC_DELTA ? 1 : -1, ll.eps, ll.act2, ct, T, RV,
-                            rst, RV, 1.f));
+        CK(launch_norm_gate(ll.yssm, r_gate, ldrg, rp.heads, L.onorm.data, r_gate ? d.r_gate_act : -1, ll.eps, ll.act2, ct, T, RV, rst, RV, 1.f));
     }
     if (forked) CK(cudaEventRecord(ll.ev_join, rst));
     // ---- attention branch ----
     CAT(CAT_ATTN);
     AttnIO io;
-    io.q = src + d.c_q; io.ldq = ld;
-    io.k = src + d.c_k; io.ldk = ld;
-    io.v = src + d.c_v; io.ldv = ld;
+    io.q = lq; io.ldq = ld;
+    io.k = lk; io.ldk = ld;
+    io.v = lv; io.ldv = ld;
     io.k_row = (int64_t) a.kv_heads * a.dim; io.v_row = (int64_t) a.kv_heads * a.vdim;
     const bool post = d.v_rot || sum;   // the head results are turned back, gated and scaled into their place by a kernel of their own
     if (!post) { io.gate = ll.big + d.c_g; io.ldg = C; io.gate_mode = d.gate_mode; }
@@ -1975,7 +2312,7 @@ static int mix_dual(pb200_model * m, const BatchView & b, bool prefill, const LR
     if (sum && unfused) {
         CK(launch_attn_unrotate_gate(ll.big2, b, a.heads, a.vdim, d.rot_layout, d.v_rot ? L.vrot_freq.data : nullptr, ll.big + d.c_g, C, d.gate_mode, d.left_scale,
                                      ll.act, ldo, ct, st));
-        CK(launch_norm_gate(ll.yssm, d.rec == REC_DELTA ? ll.big + d.c_rg : nullptr, C, rp.heads, L.onorm.data, d.rec == REC_DELTA ? 1 : -1, ll.eps,
+        CK(launch_norm_gate(ll.yssm, r_gate, ldrg, rp.heads, L.onorm.data, r_gate ? d.r_gate_act : -1, ll.eps,
                             (uint8_t *) ll.act + (size_t) OD * esize(ct), ct, T, RV, st, ldo, d.right_scale));
         CAT(CAT_DENSE);
         return launch_dense(ct, ll.act, ldo, L.out.data, ldo, x, W, T, W, (int) ldo, nullptr, x, W, mult, st);
@@ -1984,7 +2321,7 @@ static int mix_dual(pb200_model * m, const BatchView & b, bool prefill, const LR
         // attention heads turned back and gated; recurrence heads by their own root mean square, the weight all heads share, the SiLU gate; both
         // with their branch's factor, side by side as the operand of the one output product
         CK(launch_dual_post(ll.big2, b, a.heads, a.vdim, d.rot_layout, d.v_rot ? L.vrot_freq.data : nullptr, ll.big + d.c_g, C, d.gate_mode, d.left_scale, ll.yssm,
-                            rp.heads, rp.vdim, d.rec == REC_DELTA ? ll.big + d.c_rg : nullptr, C, L.onorm.data, d.rec == REC_DELTA ? 1 : -1, ll.eps, d.right_scale,
+                            rp.heads, rp.vdim, r_gate, ldrg, L.onorm.data, r_gate ? d.r_gate_act : -1, ll.eps, d.right_scale,
                             ll.act, ldo, ct, st));
         CAT(CAT_DENSE);
         return launch_dense(ct, ll.act, ldo, L.out.data, ldo, x, W, T, W, (int) ldo, nullptr, x, W, mult, st);
@@ -2039,6 +2376,18 @@ static int ff_xielu(pb200_model * m, int T, LLayer & L, float * x) {
         act.xielu = L.ff_act.data; act.y = ll.act2; act.ldy = ff;
         CK(launch_dense_act(ct, ll.act, W, L.gateup.data, W, act, T, ff, W, st));
     }
+    return launch_dense(ct, ll.act2, ff, L.down.data, ff, x, W, T, W, ff, nullptr, x, W, 1.f, st);
+}
+// ---- SiLU-gated feed-forward: x[t] += down(silu(gate(ll.act[t])) * up(ll.act[t])) ----
+static int ff_silu(pb200_model * m, int T, LLayer & L, float * x) {
+    LayerList & ll = *m->ll;
+    cudaStream_t st = m->stream;
+    const int W = ll.width, ct = ll.ctype, ff = L.ff;
+    CAT(CAT_DENSE);
+    CK(launch_dense(ct, ll.act, W, L.gateup.data, W, ll.big, 2 * ff, T, 2 * ff, W, nullptr, nullptr, 0, 1.f, st));
+    CAT(CAT_ELEM);
+    CK(launch_silu_mul(ll.big, ll.act2, ct, T, ff, nullptr, nullptr, st));
+    CAT(CAT_DENSE);
     return launch_dense(ct, ll.act2, ff, L.down.data, ff, x, W, T, W, ff, nullptr, x, W, 1.f, st);
 }
 // ---- mixture of experts over ll.act.  accumulate: x[t] += shared(h) + sum_k w_k expert_k(h) (the stream itself); otherwise x receives the
@@ -2150,7 +2499,7 @@ static int ll_forward_postnorm(pb200_model * m, const BatchView & b, bool prefil
 
 // FRAME_PRERMS: the stream starts as embed * scale + bigram row; x <- x + mult * mixer(norm1 x), x <- x + mult * ff(norm2 x) with RMS norms of
 // one learned number (kept as a constant vector); every pass of the repeated block first adds the embedding output (not the first pass) and
-// its step vector.  With embed_normed the stream starts as the normed embedding instead; norms may have a weight per entry (kept as factors).
+// its step vector.  With embed_normed the stream starts as the normed embedding instead; with tied_head the logits come from the embedding table; norms may have a weight per entry (kept as factors).
 // ll.act holds the next sublayer's normed input in the operand type.
 static int ll_forward_prerms(pb200_model * m, const BatchView & b, bool prefill, const int32_t * tokens_dev, const int32_t * want_dev, int nW, int lrow0) {
     LayerList & ll = *m->ll;
@@ -2158,10 +2507,10 @@ static int ll_forward_prerms(pb200_model * m, const BatchView & b, bool prefill,
     const int T = b.n_tokens, W = ll.width, ct = ll.ctype;
     CAT(CAT_ELEM);
     bool act_ready = false;   // the kernel that closed the previous sublayer has left this one's normed input in ll.act
-    if (ll.embed_normed) {
+    if (ll.embed_normed || (ll.bigram.buckets <= 0 && ll.loop_times <= 0)) {
         const LLayer & L0 = ll.layers[(size_t) ll.runs[0].layer];
         act_ready = L0.kind != MIX_WKV;
-        CK(launch_embed_rmsnorm(ll.embed.data, ct, W, tokens_dev, T, ll.embed_norm.data, ll.eps, ll.x, L0.norm1.data, act_ready ? ll.act : nullptr, ct, st));
+        CK(launch_embed_rmsnorm(ll.embed.data, ct, W, tokens_dev, T, ll.embed_normed ? ll.embed_norm.data : nullptr, ll.embed_scale, ll.eps, ll.x, L0.norm1.data, act_ready ? ll.act : nullptr, ct, st));
     } else CK(launch_embed_bigram(ll.embed.data, ll.bigram.buckets > 0 ? ll.bigram_table.data : nullptr, ct, W, ll.embed_scale, ll.bigram, tokens_dev, b, ll.x,
                            ll.loop_times > 1 ? ll.x0 : nullptr, st));
     for (size_t ir = 0; ir < ll.runs.size(); ir++) {
@@ -2193,6 +2542,7 @@ static int ll_forward_prerms(pb200_model * m, const BatchView & b, bool prefill,
             }
             if (L.ff_kind == FF_MOE) CK(ff_moe(m, T, prefill, L, ll.x, true, ll.resid_mult));
             else if (L.ff_kind == FF_XIELU && ll.resid_mult == 1.f) CK(ff_xielu(m, T, L, ll.x));
+            else if (L.ff_kind == FF_SILU && ll.resid_mult == 1.f) CK(ff_silu(m, T, L, ll.x));
             else return PB200_ENOTSUP;
         } else {
             act_ready = fused;
@@ -2202,7 +2552,9 @@ static int ll_forward_prerms(pb200_model * m, const BatchView & b, bool prefill,
     if (nW > 0) {
         CAT(CAT_HEAD);
         CK(launch_group_rmsnorm(ll.x, want_dev, ll.final_norm.data, 1, ll.eps, ll.actw, ct, nW, W, st));
-        CK(launch_dense(ct, ll.actw, W, ll.head.data, W, ll.logits + (int64_t) lrow0 * ll.vocab, ll.vocab, nW, ll.vocab, W, nullptr, nullptr, 0, ll.logit_scale, st));
+        float * lg = ll.logits + (int64_t) lrow0 * ll.vocab;
+        CK(launch_dense(ct, ll.actw, W, (ll.tied_head ? ll.embed : ll.head).data, W, lg, ll.vocab, nW, ll.vocab, W, nullptr, nullptr, 0, ll.logit_scale, st));
+        CK(launch_softcap(lg, (int64_t) nW * ll.vocab, ll.logit_softcap, st));
     }
     CAT(-1);
     return 0;

@@ -10,7 +10,9 @@
 // their position), a sink in the softmax denominator, gated linear recurrences with a decay per token (gated delta rule, HGRN2, and the WKV form
 // that reads the state before the token's write with a bonus for the token itself), experts whose routing weight multiplies their input; attention
 // inside fixed chunks of positions, learned sinks and temperatures per head, latent attention with a direct query projection, a token mix with a
-// blend per input, a decay from a low-rank map of the token, the xIELU feed-forward.  Every constant of a mechanism is a parameter, nothing is tied to one model.
+// blend per input, a decay from a low-rank map of the token, the xIELU feed-forward; attention over another layer's cached keys and values, keys
+// that serve as values, a query temperature that grows with the position, a sliding window over latents, the gated delta rule with a decay per
+// channel.  Every constant of a mechanism is a parameter, nothing is tied to one model.
 // All launchers enqueue on `stream` and return a cudaError_t as int (0 = success).
 #pragma once
 #include <cuda_bf16.h>
@@ -63,8 +65,9 @@ int dense_uses_tensor_cores(int type, int T, int N, int K, int64_t lda, int64_t 
 
 // ---- element-wise / norms; `otype` (T_F32 | T_BF16) is the type of an activation that feeds a dense product ----
 // x[t] = rmsnorm(table[tokens[t]]) * w, then (y given) y[t] = rmsnorm(x[t]) * wn in the operand type: a normed embedding and the first layer's norm
-int launch_embed_rmsnorm(const void * table, int type, int width, const int32_t * tokens, int n_tokens, const float * w, float eps, float * x, const float * wn,
-                         void * y, int otype, cudaStream_t stream);
+// w == nullptr: x[t] = table[tokens[t]] * scale instead (an embedding factor), and y its norm
+int launch_embed_rmsnorm(const void * table, int type, int width, const int32_t * tokens, int n_tokens, const float * w, float scale, float eps, float * x,
+                         const float * wn, void * y, int otype, cudaStream_t stream);
 int launch_embed(const void * table, int type, int width, const int32_t * tokens, int n_tokens, float * x, float * x_copy, cudaStream_t stream);
 // x[t] = table[tokens[t]] + pos_table[position of t] (fp32 sum; both tables in `type`); xa (if given) receives x in the operand type
 int launch_embed_pos(const void * table, const void * pos_table, int type, int width, const int32_t * tokens, const BatchView & b, float * x, void * xa,
@@ -115,6 +118,8 @@ struct AttnParams {
     int sink = 0;             // 1: the softmax denominator has one more term, a key without a value: of score 0, or AttnIO::sink[head]
     int chunk = 0;            // > 0: position i sees j <= i only inside its own chunk of positions, floor(i / chunk) = floor(j / chunk); the cache
                               // is a ring of `chunk` rows then (window must be 0)
+    int own_kv = 1;           // 0: keys and values are another layer's cache; the projection holds the queries (and the gate) alone
+    int tied_v = 0;           // 1: a key is its own value (vdim == dim): no value projection, no value rows in the cache
 };
 // lowest position that position i sees (apart from kept first tokens)
 __host__ __device__ inline int attn_first_visible(const AttnParams & a, int i) {
@@ -133,8 +138,17 @@ struct AttnIO {
     int gate_mode = 0;                                  // 0: no gate, 1: one logit per head, 2: one per output element [heads][vdim]
     int64_t k_row = 0, v_row = 0;
     const float * sink = nullptr;                       // AttnParams::sink: the extra key's score per head (nullptr: 0)
+    // set: prompt kernels read keys and values of position p from row p of the entry's slot (k / v: the cache's base, ldk / ldv its row strides;
+    // a cache that holds every position) instead of the batch
+    const int32_t * kv_slot = nullptr;  int64_t kv_slot_stride = 0;
 };
-__host__ __device__ inline int attn_qkvg_cols(const AttnParams & a) { return a.heads * a.dim + a.kv_heads * a.dim + a.kv_heads * a.vdim + (a.gated ? a.heads : 0); }
+// floats of a cached value row (none of its own when a key is its own value)
+__host__ __device__ inline int attn_v_row(const AttnParams & a) { return a.tied_v ? 0 : a.kv_heads * a.vdim; }
+__host__ __device__ inline int attn_qkvg_cols(const AttnParams & a) {
+    return a.heads * a.dim + (a.own_kv ? a.kv_heads * a.dim + attn_v_row(a) : 0) + (a.gated ? a.heads : 0);
+}
+// the fused q | k | v | gate projection of an attention mixer as the kernels' inputs
+AttnIO attn_io_fused(const float * qkvg, const AttnParams & a);
 // rows of a slot's cache so that every position a later token may still see is present, capped at n_ctx
 inline int attn_cache_rows(int window, int keep_first, int n_ctx) {
     if (window <= 0) return n_ctx;
@@ -228,13 +242,15 @@ struct LatentParams {
     int rot_layout = 1;       // ROT_HALVES (i, i + rot_dims / 2) or ROT_INTERLEAVED (2i, 2i + 1)
     float rot_mag = 1.f;      // factor on cos and sin
     float scale = 1.f;
-    int cache_rows = 0;       // rows of kv_rank + rot_dim floats per slot: [normed latent | rotated shared key part] of every position
+    int cache_rows = 0;       // rows of kv_rank + rot_dim floats per slot: [normed latent | rotated shared key part] of position p in row p % cache_rows
     int own_kv = 1;           // 0: the layer reads another layer's cache and has no down-projection of its own
-    int gated = 1;            // a gate logit per output element
+    int gate_mode = 2;        // 0: no gate, 1: a gate logit per head, 2: one per output element
+    int window = 0;           // > 0: position i sees j <= i with i - j < window; the cache is a ring of cache_rows <= window rows then
 };
+__host__ __device__ inline int latent_gate_cols(const LatentParams & p) { return p.gate_mode == 0 ? 0 : p.gate_mode == 1 ? p.heads : p.heads * p.vdim; }
 // columns of the fused projection: the query latent (q_rank 0: the queries themselves, heads * (dim + rot_dim)), then the gate, then dkv
 __host__ __device__ inline int latent_q_cols(const LatentParams & p) { return p.q_rank > 0 ? p.q_rank : p.heads * (p.dim + p.rot_dim); }
-__host__ __device__ inline int latent_kv_col(const LatentParams & p) { return latent_q_cols(p) + (p.gated ? p.heads * p.vdim : 0); }
+__host__ __device__ inline int latent_kv_col(const LatentParams & p) { return latent_q_cols(p) + latent_gate_cols(p); }
 __host__ __device__ inline int latent_proj_cols(const LatentParams & p) { return latent_kv_col(p) + (p.own_kv ? p.kv_rank + p.rot_dim : 0); }
 __host__ __device__ inline int latent_row(const LatentParams & p) { return p.kv_rank + p.rot_dim; }
 // proj: [T][dq or q | gate | dkv] f32 (one fused projection; gate only if gated, dkv only with own_kv).  q_rank > 0: cq[t] = rmsnorm(dq) * wq ->
@@ -252,7 +268,7 @@ int launch_latent_gather(const float * cache, int64_t slot_stride, const BatchVi
 // one dot product.  q comes straight from the projection (not rotated yet).
 int launch_latent_absorb_q(const float * q, int64_t ldq, const BatchView & b, const void * wuk, int wtype, const LatentParams & p, const float * freq, float * qa,
                            cudaStream_t stream);
-// decode: out[t][h][:] = (W_uv[h] olat[t][h]) * sigmoid(gate[t][h][:])   (gate may be null)   olat: [T][heads][kv_rank] (the weighted sum of latents)
+// decode: out[t][h][:] = (W_uv[h] olat[t][h]) * sigmoid(gate[t], form LatentParams::gate_mode)   (gate may be null)   olat: [T][heads][kv_rank] (the weighted sum of latents)
 int launch_latent_up_v(const float * olat, const void * wuv, int wtype, const LatentParams & p, const float * gate, int64_t ldg, void * out, int otype,
                        int n_tokens, cudaStream_t stream);
 
@@ -327,10 +343,12 @@ struct AttnPrep {
     int rot_dims = 0;             // the leading rot_dims entries of every query / key head turn by position * rot_freq[i]
     int rot_layout = ROT_INTERLEAVED;
     const float * rot_freq = nullptr;   // [rot_dims / 2]
+    float rot_mag = 1.f;                // factor on cos and sin of the query / key rotation
     int v_rot = 0;                // 1: every value head turns by its position over all vdim entries (pairs in v_layout, v_freq [vdim / 2]);
     int v_layout = ROT_INTERLEAVED;     // the cache holds the turned values and launch_attn_unrotate_gate turns a head's result back
     const float * v_freq = nullptr;
     const float * q_scale = nullptr;    // [heads]: factor on every prepared query head (a temperature on its scores)
+    float q_temp_coef = 0.f, q_temp_every = 0.f;   // every > 0: queries times 1 + coef ln(floor((position + 1) / every) + 1)
 };
 // q [T][heads][dim], k [T][kv_heads][dim], v [T][kv_heads][vdim] (rows ldq / ldk / ldv floats apart) are prepared in place; then the K / V
 // rows that later tokens can still see go to the cache (layout as launch_attn_kv_store).
@@ -343,7 +361,8 @@ int launch_attn_unrotate_gate(const float * o, const BatchView & b, int heads, i
                               int gate_mode, float out_scale, void * out, int64_t ldo, int otype, cudaStream_t stream);
 
 // the same with the preparation of a recurrent branch's inputs in front, one launch for both branches of a dual mixer: rec_kind 0 =
-// launch_delta_prep(rq, rk, beta, ra, p0 = A_log, p1 = dt_bias), 1 = launch_hgrn2_prep(rq, rk = forget logits, p0 = f_bias, p1 = lower)
+// launch_delta_prep(rq, rk, beta, ra, p0 = A_log, p1 = dt_bias; ra == nullptr: decays come from elsewhere), 1 = launch_hgrn2_prep(rq, rk = forget
+// logits, p0 = f_bias, p1 = lower)
 int launch_dual_prep_store(int rec_kind, float * rq, int64_t ldrq, float * rk, int64_t ldrk, float * beta, int64_t ldb, float * ra, int64_t lda, const float * p0,
                            const float * p1, int qk_heads, int r_heads, int r_dim, float * q, int64_t ldq, float * k, int64_t ldk, float * v, int64_t ldv,
                            const BatchView & b, const AttnParams & a, const AttnPrep & pr, float * kcache, float * vcache, int64_t slot_stride, cudaStream_t stream);
@@ -354,9 +373,9 @@ int launch_dual_post(const float * o, const BatchView & b, int heads, int vdim, 
                      float right_scale, void * out, int64_t ldo, int otype, cudaStream_t stream);
 
 // ---- gated linear recurrences: a state S [dim][vdim] f32 per (sequence slot, head) with a decay that every token brings ----
-//   decay_per_channel 0: S <- g S (g [T][heads]);  1: S <- diag(f) S (f [T][qk_heads][dim])
+//   decay_per_channel 0: S <- g S (g [T][heads]);  1: S <- diag(f) S (f [T][heads][dim])
 //   delta 0: S <- S + k v^T;   1 (delta rule): u = beta (v - S^T k), S <- S + k u^T (beta [T][heads]), after the decay
-//   tied_key 1: k = 1 - f (needs decay_per_channel; io.k unused)
+//   tied_key 1: k = 1 - f (needs decay_per_channel and qk_heads == heads; io.k unused)
 //   y = S^T q, after the token's write; bonus 1 (needs decay_per_channel, no delta, no tied key): y = (S + diag(u) k v^T)^T q with the state
 //   BEFORE the token's decay and write, u = io.bonus.        Head h reads q / k head h / (heads / qk_heads).
 struct GatedLinParams {
@@ -374,7 +393,7 @@ struct GatedLinIO {
 int launch_gated_linattn(const GatedLinIO & io, const BatchView & b, const GatedLinParams & p, float * state, int64_t slot_stride, float * y,
                          cudaStream_t stream);
 // inputs of the gated delta rule, in place: every q / k head (qk_heads of each, dim wide) becomes x / sqrt(sum x^2 + 1e-6), q also times
-// dim^-1/2;  beta <- sigmoid(beta);  a <- exp(-exp(A_log[h]) * softplus(a + dt_bias[h]))    (beta, a: [T][heads])
+// dim^-1/2;  beta <- sigmoid(beta);  a <- exp(-exp(A_log[h]) * softplus(a + dt_bias[h]))    (beta, a: [T][heads]; a may be null)
 int launch_delta_prep(float * q, int64_t ldq, float * k, int64_t ldk, float * beta, int64_t ldb, float * a, int64_t lda, const float * A_log,
                       const float * dt_bias, int qk_heads, int heads, int dim, int n_tokens, cudaStream_t stream);
 // inputs of HGRN2, in place: q <- silu(q);  f <- lower + (1 - lower) * sigmoid(f + f_bias)      (n = heads * dim entries per token)
@@ -390,6 +409,19 @@ int launch_rmsnorm_token_mix(const float * x, const BatchView & b, const float *
 // tmp: [T][rank] floats
 int launch_lowrank_decay(const float * m, const float * w1, const float * w2, const float * w0, int n_tokens, int width, int rank, int channels, float * tmp,
                          float * decay, cudaStream_t stream);
+
+// two low-rank maps of the token whose inner values z = u[t * ldu + ..] a projection has left side by side, fp32 throughout, one launch:
+// decay[t][h * dim + n] = exp(-exp(A_log[h]) * softplus(sum_j wa[h * dim + n][j] z_a[t][j] + dt_bias[h * dim + n]))   (wa [heads * dim][ra])
+// gate[t][c] = sum_j wg[c][j] z_g[t][j], c < gate_cols (wg [gate_cols][rg]); rows of the two results ldd / ldg floats apart
+struct LowrankMaps {
+    const float * za = nullptr, * zg = nullptr;  int64_t ldu = 0;
+    const float * wa = nullptr, * wg = nullptr;  int ra = 0, rg = 0;
+    const float * A_log = nullptr, * dt_bias = nullptr;
+    int heads = 0, dim = 0, gate_cols = 0;
+    float * decay = nullptr;  int64_t ldd = 0;
+    float * gate = nullptr;   int64_t ldg = 0;
+};
+int launch_lowrank_maps(const LowrankMaps & mp, int n_tokens, cudaStream_t stream);
 
 // x[t] += (x0 ? x0[t] : 0) + (vec ? vec : 0), then y[t] = rmsnorm(x[t]) * w in the operand type: what opens a pass of a repeated block whose
 // passes add the embedding output and a step vector, with the first layer's norm

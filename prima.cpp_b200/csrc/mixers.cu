@@ -28,20 +28,24 @@ __global__ void k_embed(const WT * __restrict__ table, int width, const int32_t 
     }
 }
 
-// one CTA per token: the table row normed, and (y given) normed again for the first layer; every thread re-reads only what it has written itself
+// one CTA per token: the table row normed (no weight: times a factor), and (y given) normed again for the first layer; every thread re-reads only
+// what it has written itself
 template <typename WT, typename OT>
 __global__ void __launch_bounds__(1024) k_embed_rmsnorm(const WT * __restrict__ table, int width, const int32_t * __restrict__ tokens, const float * __restrict__ w,
-                                                       float eps, float * __restrict__ x, const float * __restrict__ wn, OT * __restrict__ y) {
+                                                       float scale, float eps, float * __restrict__ x, const float * __restrict__ wn, OT * __restrict__ y) {
     __shared__ float red[33];
     const int t = blockIdx.x;
     const WT * row = table + (int64_t) tokens[t] * width;
     float * xr = x + (int64_t) t * width;
-    float s = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) { const float v = ld_f(row, i); s = fmaf(v, v, s); }
-    const float inv = 1.f / sqrtf(block_sum(s, red) / (float) width + eps);
+    float inv = scale;
+    if (w) {
+        float s = 0.f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) { const float v = ld_f(row, i); s = fmaf(v, v, s); }
+        inv = 1.f / sqrtf(block_sum(s, red) / (float) width + eps);
+    }
     float s2 = 0.f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = ld_f(row, i) * inv * w[i];
+        const float v = w ? ld_f(row, i) * inv * w[i] : ld_f(row, i) * inv;
         xr[i] = v;
         s2 = fmaf(v, v, s2);
     }
@@ -214,9 +218,19 @@ __global__ void __launch_bounds__(1024) k_argmax_rows(const float * __restrict__
 // attention.  Cache row of position p: p itself below keep_first, else keep_first + (p - keep_first) mod ring.
 __device__ __forceinline__ int cache_row(int p, int keep_first, int ring) { return p < keep_first ? p : keep_first + (p - keep_first) % ring; }
 
-// key element d of (token row, kv head): the head's own part, then the part all heads share
-__device__ __forceinline__ float attn_key(const AttnIO & io, int64_t row, int kvh, int d, int DN) {
-    return d < DN ? io.k[row * io.ldk + (int64_t) kvh * DN + d] : io.ks[row * io.ldks + (d - DN)];
+// where a prompt kernel finds keys and values of an entry's positions: the entry's rows of the batch, or its slot's cache
+struct AttnKV {
+    const float * k, * ks, * v;
+    __device__ __forceinline__ AttnKV(const AttnIO & io, int e, int t_begin) {
+        const int64_t at = io.kv_slot ? (int64_t) io.kv_slot[e] * io.kv_slot_stride : 0;
+        k = io.k + (io.kv_slot ? at : (int64_t) t_begin * io.ldk);
+        v = io.v + (io.kv_slot ? at : (int64_t) t_begin * io.ldv);
+        ks = io.ks ? io.ks + (int64_t) t_begin * io.ldks : nullptr;
+    }
+};
+// key element d of (position, kv head): the head's own part, then the part all heads share
+__device__ __forceinline__ float attn_key(const AttnKV & kv, const AttnIO & io, int64_t row, int kvh, int d, int DN) {
+    return d < DN ? kv.k[row * io.ldk + (int64_t) kvh * DN + d] : kv.ks[row * io.ldks + (d - DN)];
 }
 // score of the sink of head h
 __device__ __forceinline__ float attn_sink(const AttnIO & io, int h) { return io.sink ? io.sink[h] : 0.f; }
@@ -320,6 +334,7 @@ __global__ void __launch_bounds__(AQ * 32) k_attn_window_prefill(const AttnIO io
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int D = a.dim, DV = a.vdim, DN = a.dim - a.shared_dim;
     const int kvh = h / (a.heads / a.kv_heads);
+    const AttnKV kv(io, e, t_begin);
     float * qs = sm;                       // [AQ][D]
     float * kt = qs + AQ * D;              // [AKT][D + 1]
     float * vt = kt + AKT * (D + 1);       // [AKT][DV]
@@ -341,11 +356,11 @@ __global__ void __launch_bounds__(AQ * 32) k_attn_window_prefill(const AttnIO io
             const int nk = min(AKT, hi - k0);
             for (int i = threadIdx.x; i < AKT * D; i += blockDim.x) {
                 const int j = i / D, d = i - j * D;
-                kt[j * (D + 1) + d] = j < nk ? attn_key(io, t_begin + k0 + j, kvh, d, DN) : 0.f;
+                kt[j * (D + 1) + d] = j < nk ? attn_key(kv, io, k0 + j, kvh, d, DN) : 0.f;
             }
             for (int i = threadIdx.x; i < AKT * DV; i += blockDim.x) {
                 const int j = i / DV, d = i - j * DV;
-                vt[i] = j < nk ? io.v[(int64_t) (t_begin + k0 + j) * io.ldv + kvh * DV + d] : 0.f;
+                vt[i] = j < nk ? kv.v[(int64_t) (k0 + j) * io.ldv + kvh * DV + d] : 0.f;
             }
             __syncthreads();
             if (!qok) continue;
@@ -390,6 +405,7 @@ __global__ void __launch_bounds__(256) k_attn_window_prefill_tiled(const AttnIO 
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     const int D = a.dim, DV = a.vdim, DN = a.dim - a.shared_dim;
     const int kvh = h / (a.heads / a.kv_heads);
+    const AttnKV src(io, e, t_begin);
     constexpr int PQS = PQ + 4, PKS = PK + 1;   // padded strides: the transposing stores of a tile load spread over the banks
     float * Qt = sm;                    // [D][PQS]  transposed: Qt[d][q]
     float * Kt = Qt + D * PQS;          // [D][PKS]  transposed: Kt[d][k]
@@ -422,7 +438,7 @@ __global__ void __launch_bounds__(256) k_attn_window_prefill_tiled(const AttnIO 
 #pragma unroll
                 for (int u = 0; u < 8; u++) {
                     const int i = i0 + 256 * u, k = i / D, d = i - k * D;
-                    v[u] = (i < PK * D && k < nk) ? attn_key(io, t_begin + k0 + k, kvh, d, DN) : 0.f;
+                    v[u] = (i < PK * D && k < nk) ? attn_key(src, io, k0 + k, kvh, d, DN) : 0.f;
                 }
 #pragma unroll
                 for (int u = 0; u < 8; u++) {
@@ -435,7 +451,7 @@ __global__ void __launch_bounds__(256) k_attn_window_prefill_tiled(const AttnIO 
 #pragma unroll
                 for (int u = 0; u < 8; u++) {
                     const int i = i0 + 256 * u, k = i / DV, d = i - k * DV;
-                    v[u] = (i < PK * DV && k < nk) ? io.v[(int64_t) (t_begin + k0 + k) * io.ldv + kvh * DV + d] : 0.f;
+                    v[u] = (i < PK * DV && k < nk) ? src.v[(int64_t) (k0 + k) * io.ldv + kvh * DV + d] : 0.f;
                 }
 #pragma unroll
                 for (int u = 0; u < 8; u++) {
@@ -865,14 +881,14 @@ int launch_embed(const void * table, int type, int width, const int32_t * tokens
         else k_embed<float><<<n_tokens, 128, 0, st>>>((const float *) table, width, tokens, x, x_copy);
     });
 }
-int launch_embed_rmsnorm(const void * table, int type, int width, const int32_t * tokens, int n_tokens, const float * w, float eps, float * x, const float * wn,
-                         void * y, int otype, cudaStream_t st) {
+int launch_embed_rmsnorm(const void * table, int type, int width, const int32_t * tokens, int n_tokens, const float * w, float scale, float eps, float * x,
+                         const float * wn, void * y, int otype, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
-    if (!w || (y && (!wn || otype != type))) return (int) cudaErrorInvalidValue;
+    if (y && (!wn || otype != type)) return (int) cudaErrorInvalidValue;
     return ck_launch([&] {
         if (type == T_BF16)
-            k_embed_rmsnorm<__nv_bfloat16, __nv_bfloat16><<<n_tokens, row_threads(n_tokens, width), 0, st>>>((const __nv_bfloat16 *) table, width, tokens, w, eps, x, wn, (__nv_bfloat16 *) y);
-        else k_embed_rmsnorm<float, float><<<n_tokens, row_threads(n_tokens, width), 0, st>>>((const float *) table, width, tokens, w, eps, x, wn, (float *) y);
+            k_embed_rmsnorm<__nv_bfloat16, __nv_bfloat16><<<n_tokens, row_threads(n_tokens, width), 0, st>>>((const __nv_bfloat16 *) table, width, tokens, w, scale, eps, x, wn, (__nv_bfloat16 *) y);
+        else k_embed_rmsnorm<float, float><<<n_tokens, row_threads(n_tokens, width), 0, st>>>((const float *) table, width, tokens, w, scale, eps, x, wn, (float *) y);
     });
 }
 int launch_cast(const float * x, void * y, int otype, int64_t n, cudaStream_t st) {
@@ -1059,14 +1075,13 @@ int launch_attn_decode_io(const AttnIO & io, const BatchView & b, const AttnPara
     return 0;
 }
 
-// the fused q | k | v | gate projection of the windowed-attention mixer as the kernels' inputs
-static AttnIO attn_io_fused(const float * qkvg, const AttnParams & a) {
+AttnIO attn_io_fused(const float * qkvg, const AttnParams & a) {
     AttnIO io;
     const int64_t C = attn_qkvg_cols(a);
     io.q = qkvg; io.ldq = C;
     io.k = qkvg + (int64_t) a.heads * a.dim; io.ldk = C;
-    io.v = io.k + (int64_t) a.kv_heads * a.dim; io.ldv = C;
-    io.gate = io.v + (int64_t) a.kv_heads * a.vdim; io.ldg = C; io.gate_mode = a.gated ? 1 : 0;
+    io.v = a.tied_v ? io.k : io.k + (int64_t) a.kv_heads * a.dim; io.ldv = C;
+    io.gate = qkvg + C - (a.gated ? a.heads : 0); io.ldg = C; io.gate_mode = a.gated ? 1 : 0;
     io.k_row = (int64_t) a.kv_heads * a.dim; io.v_row = (int64_t) a.kv_heads * a.vdim;
     return io;
 }

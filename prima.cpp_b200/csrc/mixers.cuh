@@ -65,6 +65,31 @@ __device__ __forceinline__ float dot_lane8(const T * __restrict__ a, const float
     return acc;
 }
 
+// asynchronous copies into shared memory, 16 and 4 bytes; zeros instead of the source unless ok
+__device__ __forceinline__ void cp_async16(void * dst, const void * src, bool ok) {
+    const uint32_t d = (uint32_t) __cvta_generic_to_shared(dst);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(ok ? 16u : 0u) : "memory");
+}
+__device__ __forceinline__ void cp_async4(void * dst, const void * src, bool ok) {
+    const uint32_t d = (uint32_t) __cvta_generic_to_shared(dst);
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(d), "l"(src), "r"(ok ? 4u : 0u) : "memory");
+}
+// values [0, M) summed over the lanes that differ in the bits below 2 O: lane ends up with M / (2 O) of them, value index = its lane bits first
+template <int M, int O>
+__device__ __forceinline__ void joint_sum(float * v, int lane) {
+    if constexpr (O >= 1) {
+        if constexpr (M >= 2) {
+            const bool up = lane & O;
+#pragma unroll
+            for (int i = 0; i < M / 2; i++) {
+                const float send = up ? v[i] : v[i + M / 2], keep = up ? v[i + M / 2] : v[i];
+                v[i] = keep + __shfl_xor_sync(0xffffffffu, send, O);
+            }
+            joint_sum<M / 2, O / 2>(v, lane);
+        }
+    }
+}
+
 // CTA size of a kernel that gives every token one CTA (launch bounds 1024): few tokens leave most SMs idle, so a token's row gets more threads
 inline int row_threads(int n_tokens, int width) { return n_tokens >= 128 || width <= 512 ? 256 : width <= 1024 ? 512 : 1024; }
 

@@ -1,4 +1,5 @@
-// prima.cpp_b200/csrc/wkv.cu — the WKV mixer's own kernels (declarations and semantics: layers.h): the decay, a low-rank map of the token's mix,
+// prima.cpp_b200/csrc/wkv.cu — low-rank maps of the token that end in decays or gates, and the WKV mixer's own kernels (declarations and
+// semantics: layers.h): the WKV decay, a low-rank map of the token's mix,
 // decay = exp(-exp(w0 + W2 tanh(W1 m)))  per channel, and the recurrence for the usual head sizes (any other size runs through the kernels of
 // gated.cu).  Everything that reaches the recurrence's state is fp32 in either compute type: the map's inputs, weights, products, tanh and both
 // exponentials, keys, values and the state.
@@ -141,6 +142,53 @@ __global__ void __launch_bounds__(256) k_lowrank_up(const float * __restrict__ t
     }
 }
 
+// two maps side by side (LowrankMaps): column tiles of the decay first, then those of the gate
+template <int TT>
+__global__ void __launch_bounds__(256) k_lowrank_maps(LowrankMaps mp, int T, int a_tiles) {
+    __shared__ __align__(16) float As[TT][LR_S];
+    __shared__ __align__(16) float Bs[LR_COLS][LR_S];
+    const bool is_a = (int) blockIdx.x < a_tiles;
+    const int t0 = blockIdx.y * TT, n0 = (is_a ? blockIdx.x : blockIdx.x - a_tiles) * LR_COLS;
+    const int N = is_a ? mp.heads * mp.dim : mp.gate_cols, rank = is_a ? mp.ra : mp.rg;
+    const float * z = is_a ? mp.za : mp.zg, * w = is_a ? mp.wa : mp.wg;
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    float acc[TT / 16][4];
+#pragma unroll
+    for (int i = 0; i < TT / 16; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
+    LowrankFetch<TT> fa;
+    LowrankFetch<LR_COLS> fb;
+    for (int k0 = 0; k0 < rank; k0 += LR_K) {
+        fa.load(z, mp.ldu, t0, T, k0, rank);
+        fb.load(w, rank, n0, N, k0, rank);
+        __syncthreads();
+        fa.store(As);
+        fb.store(Bs);
+        __syncthreads();
+        lowrank_tile<TT>(As, Bs, ty, tx, acc);
+    }
+    float rate[4], bias[4];
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+        const int n = n0 + tx + 16 * j;
+        rate[j] = is_a && n < N ? expf(mp.A_log[n / mp.dim]) : 0.f;
+        bias[j] = is_a && n < N ? mp.dt_bias[n] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < TT / 16; i++) {
+        const int t = t0 + ty + 16 * i;
+        if (t >= T) continue;
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const int n = n0 + tx + 16 * j;
+            if (n >= N) continue;
+            if (is_a) mp.decay[(int64_t) t * mp.ldd + n] = expf(-rate[j] * softplus_f(acc[i][j] + bias[j]));
+            else mp.gate[(int64_t) t * mp.ldg + n] = acc[i][j];
+        }
+    }
+}
+
 // ---- the recurrence at head sizes N = 32, 64, 128, 256 ----
 //   y_t = S^T r_t + (r_t . u k_t) v_t,  then  S <- diag(w_t) S + k_t v_t^T
 // CTA = one head x 16 value columns of one entry.  LN = N / 8 lanes share a pair of columns: a lane keeps S[n][2 columns] for 8 n (four
@@ -150,25 +198,6 @@ __global__ void __launch_bounds__(256) k_lowrank_up(const float * __restrict__ t
 constexpr int WS_CHUNK = 16, WS_COLS = 16, WS_STAGES = 2, WS_NREG = 8;
 template <int N> constexpr int ws_stage_floats() { return WS_CHUNK * (3 * N + WS_COLS); }
 
-__device__ __forceinline__ void ws_cp16(void * dst, const void * src, bool ok) {
-    const uint32_t d = (uint32_t) __cvta_generic_to_shared(dst);
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(ok ? 16u : 0u) : "memory");
-}
-// values [0, M) summed over the lanes that differ in the bits below 2 O: lane ends up with M / (2 O) of them, value index = its lane bits first
-template <int M, int O>
-__device__ __forceinline__ void ws_reduce(float * v, int lane) {
-    if constexpr (O >= 1) {
-        if constexpr (M >= 2) {
-            const bool up = lane & O;
-#pragma unroll
-            for (int i = 0; i < M / 2; i++) {
-                const float send = up ? v[i] : v[i + M / 2], keep = up ? v[i + M / 2] : v[i];
-                v[i] = keep + __shfl_xor_sync(0xffffffffu, send, O);
-            }
-            ws_reduce<M / 2, O / 2>(v, lane);
-        }
-    }
-}
 
 template <int N>
 __global__ void __launch_bounds__(WS_COLS / 2 * (N / WS_NREG)) k_wkv_scan(GatedLinIO io, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
@@ -193,12 +222,12 @@ __global__ void __launch_bounds__(WS_COLS / 2 * (N / WS_NREG)) k_wkv_scan(GatedL
             const int which = i / (WS_CHUNK * Q), rem = i % (WS_CHUNK * Q), tt = rem / Q, q = rem % Q;
             const int64_t tok = t0 + c0 + min(tt, nc - 1);
             const float * src = which == 0 ? io.q + tok * io.ldq : which == 1 ? io.k + tok * io.ldk : io.decay + tok * io.ldd;
-            ws_cp16(st + which * WS_CHUNK * N + tt * N + 4 * q, src + hk * N + 4 * q, tt < nc);
+            cp_async16(st + which * WS_CHUNK * N + tt * N + 4 * q, src + (which == 2 ? h : hk) * N + 4 * q, tt < nc);
         }
         for (int i = tid; i < WS_CHUNK * (WS_COLS / 4); i += NT) {
             const int tt = i / (WS_COLS / 4), q = i % (WS_COLS / 4), c = pt * WS_COLS + 4 * q;
             const bool ok = tt < nc && c < P;        // P is a multiple of 4
-            ws_cp16(st + 3 * WS_CHUNK * N + tt * WS_COLS + 4 * q, ok ? io.v + (int64_t) (t0 + c0 + tt) * io.ldv + h * P + c : io.v, ok);
+            cp_async16(st + 3 * WS_CHUNK * N + tt * WS_COLS + 4 * q, ok ? io.v + (int64_t) (t0 + c0 + tt) * io.ldv + h * P + c : io.v, ok);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -250,7 +279,7 @@ __global__ void __launch_bounds__(WS_COLS / 2 * (N / WS_NREG)) k_wkv_scan(GatedL
             float acc[M];                                    // value token * 2 + column
 #pragma unroll
             for (int tt = 0; tt < WS_CHUNK; tt++) token(tt, acc[2 * tt], acc[2 * tt + 1]);
-            ws_reduce<M, LN / 2>(acc, lane);
+            joint_sum<M, LN / 2>(acc, lane);
 #pragma unroll
             for (int i = 0; i < KEEP; i++) {
                 const int idx = ng * KEEP + i, tt = idx >> 1, c = idx & 1;
@@ -301,6 +330,19 @@ int launch_wkv_scan(const GatedLinIO & io, const BatchView & b, const GatedLinPa
     if (p.dim == 128) return wkv_scan_launch<128>(io, b, p, state, slot_stride, y, st);
     if (p.dim == 256) return wkv_scan_launch<256>(io, b, p, state, slot_stride, y, st);
     return (int) cudaErrorInvalidValue;
+}
+
+int launch_lowrank_maps(const LowrankMaps & mp, int n_tokens, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
+    if (!mp.za || !mp.wa || mp.ra <= 0 || !mp.A_log || !mp.dt_bias || !mp.decay || mp.heads <= 0 || mp.dim <= 0 || mp.gate_cols < 0 ||
+        (mp.gate_cols > 0 && (!mp.zg || !mp.wg || mp.rg <= 0 || !mp.gate)))
+        return (int) cudaErrorInvalidValue;
+    const int at = (mp.heads * mp.dim + LR_COLS - 1) / LR_COLS;
+    const unsigned tiles = (unsigned) (at + (mp.gate_cols + LR_COLS - 1) / LR_COLS);
+    return ck_launch([&] {
+        if (n_tokens > 64) k_lowrank_maps<64><<<dim3(tiles, (unsigned) ((n_tokens + 63) / 64)), 256, 0, st>>>(mp, n_tokens, at);
+        else k_lowrank_maps<16><<<dim3(tiles, (unsigned) ((n_tokens + 15) / 16)), 256, 0, st>>>(mp, n_tokens, at);
+    });
 }
 
 int launch_lowrank_decay(const float * m, const float * w1, const float * w2, const float * w0, int n_tokens, int width, int rank, int channels, float * tmp,
