@@ -76,6 +76,14 @@ __global__ void __launch_bounds__(256) k_dense_tile(const WT * __restrict__ A, i
     for (int i = 0; i < 4; i++) {
         const int t = t0 + ty * 4 + i;
         if (t >= T) continue;
+        if (act.silu_glu) {   // a thread holds whole pairs (gate, value)
+#pragma unroll
+            for (int j = 0; j < 4; j += 2) {
+                const int n = n0 + tx * 4 + j;
+                if (n + 1 < N) put((WT *) act.y, (int64_t) t * act.ldy + n / 2, silu_f(alpha * acc[i][j]) * (alpha * acc[i][j + 1]));
+            }
+            continue;
+        }
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int n = n0 + tx * 4 + j;
@@ -109,11 +117,13 @@ template <int N> __device__ __forceinline__ void unpack(const uint4 & raw, float
 
 // KS warps share a weight row (each takes a contiguous part of K, a multiple of the 16-byte load step; the parts are summed in order
 // through shared memory): matrices with few, long rows keep more loads in flight that way.  KS comes from (N, K) alone.
-template <typename WT, int TB, bool VEC>
+// GLU (DenseAct::silu_glu): n counts pairs of rows, a warp streams both rows of its pair.
+template <typename WT, int TB, bool VEC, bool GLU>
 __global__ void __launch_bounds__(256) k_dense_rows(const WT * __restrict__ A, int64_t lda, const WT * __restrict__ W, int64_t ldw, float * C, int64_t ldc,
                                                     int T, int N, int K, const float * __restrict__ bias, const float * resid, int64_t ldr, float alpha,
                                                     int KS, int plane_rows, int64_t a_plane, DenseAct act) {
-    __shared__ float parts[8][TB];
+    constexpr int R = GLU ? 2 : 1;
+    __shared__ float parts[8][R * TB];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int rows_per_cta = (blockDim.x >> 5) / KS;
     const int n = blockIdx.x * rows_per_cta + warp / KS, part = warp % KS;
@@ -122,36 +132,42 @@ __global__ void __launch_bounds__(256) k_dense_rows(const WT * __restrict__ A, i
     constexpr int V = Vec16<WT>::n;
     const int Kc = KS == 1 ? K : ((K + KS - 1) / KS + 32 * V - 1) / (32 * V) * (32 * V);
     const int k_begin = part * Kc, k_end = min(K, k_begin + Kc);
-    const WT * w = W + (int64_t) (live ? n : 0) * ldw;
-    float acc[TB];
+    const WT * w = W + (int64_t) (live ? R * n : 0) * ldw;
+    float acc[R * TB];                       // row r of the pair, token t at r * TB + t
 #pragma unroll
-    for (int t = 0; t < TB; t++) acc[t] = 0.f;
+    for (int t = 0; t < R * TB; t++) acc[t] = 0.f;
     if (live) {
         if (VEC) {
             for (int k = k_begin + lane * V; k < k_end; k += 32 * V) {
-                float wf[V];
-                unpack<V>(__ldcs(reinterpret_cast<const uint4 *>(w + k)), wf, WT());   // streamed once: do not keep in L1
+                float wf[R][V];
+#pragma unroll
+                for (int r = 0; r < R; r++) unpack<V>(__ldcs(reinterpret_cast<const uint4 *>(w + r * ldw + k)), wf[r], WT());   // streamed once: do not keep in L1
 #pragma unroll
                 for (int t = 0; t < TB; t++) {
                     if (t < T) {
                         float af[V];
                         unpack<V>(__ldg(reinterpret_cast<const uint4 *>(A + (int64_t) t * lda + k)), af, WT());
 #pragma unroll
-                        for (int i = 0; i < V; i++) acc[t] = fmaf(af[i], wf[i], acc[t]);
+                        for (int r = 0; r < R; r++)
+#pragma unroll
+                            for (int i = 0; i < V; i++) acc[r * TB + t] = fmaf(af[i], wf[r][i], acc[r * TB + t]);
                     }
                 }
             }
         } else {
             for (int k = k_begin + lane; k < k_end; k += 32) {
-                const float wv = to_f(w[k]);
 #pragma unroll
-                for (int t = 0; t < TB; t++)
-                    if (t < T) acc[t] = fmaf(to_f(A[(int64_t) t * lda + k]), wv, acc[t]);
+                for (int r = 0; r < R; r++) {
+                    const float wv = to_f(w[r * ldw + k]);
+#pragma unroll
+                    for (int t = 0; t < TB; t++)
+                        if (t < T) acc[r * TB + t] = fmaf(to_f(A[(int64_t) t * lda + k]), wv, acc[r * TB + t]);
+                }
             }
         }
     }
 #pragma unroll
-    for (int t = 0; t < TB; t++) {
+    for (int t = 0; t < R * TB; t++) {
         float v = acc[t];
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -160,16 +176,24 @@ __global__ void __launch_bounds__(256) k_dense_rows(const WT * __restrict__ A, i
     if (KS > 1) {
         if (lane == 0) {
 #pragma unroll
-            for (int t = 0; t < TB; t++) parts[warp][t] = acc[t];
+            for (int t = 0; t < R * TB; t++) parts[warp][t] = acc[t];
         }
         __syncthreads();
         if (part != 0) return;
 #pragma unroll
-        for (int t = 0; t < TB; t++) {
+        for (int t = 0; t < R * TB; t++) {
             float v = 0.f;
             for (int j = 0; j < KS; j++) v += parts[warp + j][t];
             acc[t] = v;
         }
+    }
+    if constexpr (GLU) {
+        if (lane == 0 && live) {
+#pragma unroll
+            for (int t = 0; t < TB; t++)
+                if (t < T) put((WT *) act.y, (int64_t) t * act.ldy + n, silu_f(alpha * acc[t]) * (alpha * acc[TB + t]));
+        }
+        return;
     }
     if (lane == 0 && live) {
         const float xp = act.xielu ? softplus_f(act.xielu[0]) : 0.f, xn = act.xielu ? 0.5f + softplus_f(act.xielu[1]) : 0.f;
@@ -204,6 +228,8 @@ int dense_typed(const WT * A, int64_t lda, const WT * W, int64_t ldw, float * C,
                 const float * resid, int64_t ldr, float alpha, cudaStream_t st, int plane_rows = 0, int64_t a_plane = 0,
                 const DenseAct & act = DenseAct()) {
     if (T <= ROWS_MAX_T) {
+        const bool glu = act.silu_glu != 0;
+        if (glu) N /= 2;   // pairs of rows
         constexpr int V = Vec16<WT>::n;
         const bool vec = K % V == 0 && lda % V == 0 && ldw % V == 0 && a_plane % V == 0 && ((uintptr_t) A & 15) == 0 && ((uintptr_t) W & 15) == 0;
         // warps per row: few rows leave most of the machine's load slots empty, so 2, 4 or 8 warps split a long row
@@ -211,16 +237,20 @@ int dense_typed(const WT * A, int64_t lda, const WT * W, int64_t ldw, float * C,
         while (KS < 8 && (int64_t) N * KS < 6144 && K / (2 * KS) >= 1024) KS *= 2;
         const dim3 grid((unsigned) ((N + 8 / KS - 1) / (8 / KS))), block(256);
         g_launches++;
-        if (T <= 1) {
-            if (vec) k_dense_rows<WT, 1, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
-            else k_dense_rows<WT, 1, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
-        } else if (T <= 4) {
-            if (vec) k_dense_rows<WT, 4, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
-            else k_dense_rows<WT, 4, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
-        } else {
-            if (vec) k_dense_rows<WT, ROWS_MAX_T, true><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
-            else k_dense_rows<WT, ROWS_MAX_T, false><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act);
-        }
+#define PB_ROWS(TB, VEC, GLU) k_dense_rows<WT, TB, VEC, GLU><<<grid, block, 0, st>>>(A, lda, W, ldw, C, ldc, T, N, K, bias, resid, ldr, alpha, KS, plane_rows, a_plane, act)
+#define PB_ROWS_TB(TB)                          \
+    do {                                        \
+        if (glu) {                              \
+            if (vec) PB_ROWS(TB, true, true);   \
+            else PB_ROWS(TB, false, true);      \
+        } else if (vec) PB_ROWS(TB, true, false); \
+        else PB_ROWS(TB, false, false);         \
+    } while (0)
+        if (T <= 1) PB_ROWS_TB(1);
+        else if (T <= 4) PB_ROWS_TB(4);
+        else PB_ROWS_TB(ROWS_MAX_T);
+#undef PB_ROWS_TB
+#undef PB_ROWS
         return (int) cudaGetLastError();
     }
     const dim3 grid((unsigned) ((N + TN - 1) / TN), (unsigned) ((T + TM - 1) / TM)), block(256);
@@ -268,7 +298,7 @@ int launch_dense_planes(int type, const void * A, int64_t a_plane, int64_t lda, 
 
 int launch_dense_act(int type, const void * A, int64_t lda, const void * W, int64_t ldw, const DenseAct & act, int T, int N, int K, cudaStream_t st) {
     if (T <= 0 || N <= 0) return 0;
-    if (K <= 0 || !A || !W || !act.xielu || !act.y || (type != 0 && type != T_BF16)) return (int) cudaErrorInvalidValue;
+    if (K <= 0 || !A || !W || (!act.xielu && !act.silu_glu) || (act.silu_glu && (act.xielu || N % 2)) || !act.y || (type != 0 && type != T_BF16)) return (int) cudaErrorInvalidValue;
     if (type == 0) return dense_typed<float>((const float *) A, lda, (const float *) W, ldw, nullptr, 0, T, N, K, nullptr, nullptr, 0, 1.f, st, 0, 0, act);
     const __nv_bfloat16 * a = (const __nv_bfloat16 *) A, * w = (const __nv_bfloat16 *) W;
     if (T > rows_max_t() && dense_tc_ok(T, N, K, lda, ldw, A, W)) return launch_dense_tc(a, lda, w, ldw, nullptr, 0, T, N, K, nullptr, nullptr, 0, 1.f, st, 0, 0, act);

@@ -203,6 +203,17 @@ __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constan
                 : "r"(taddr)
                 : "memory");
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+            if (P.act.silu_glu) {   // neighbouring lanes hold a gate and its value: of two tokens the even lane finishes the first, the odd one the second
+                const bool odd = lane & 1;
+#pragma unroll
+                for (int i = 0; i < 16; i += 2) {
+                    const float mine = P.alpha * __uint_as_float(odd ? v[i + 1] : v[i]);
+                    const float other = __shfl_xor_sync(0xffffffffu, P.alpha * __uint_as_float(odd ? v[i] : v[i + 1]), 1);
+                    const int t = t0 + c0 + i + (odd ? 1 : 0);
+                    if (n < P.N && t < Tn && !*cta_abort) put(ya, (int64_t) t * P.act.ldy + n / 2, odd ? silu_f(other) * mine : silu_f(mine) * other);
+                }
+                continue;
+            }
             if (n < P.N && !*cta_abort) {
 #pragma unroll
                 for (int i = 0; i < 16; i++) {

@@ -163,6 +163,7 @@ struct LRun {
 struct TensorPlace {
     DenseW * mat = nullptr;   // rows [row0, row0 + rows) of a matrix, columns [col0, col0 + cols) (col0 == 0 and cols == K: whole rows) ...
     int64_t row0 = 0, rows = 0, cols = 0, col0 = 0;
+    int64_t row_step = 1;     // (whole rows only) > 1: row r of the tensor is row row0 + r * row_step: matrices whose rows lie in turns
     int part = 0;             // index into mat->filled / vec->parts
     VecF * vec = nullptr;     // ... or a whole fp32 vector of n elements ...
     int64_t n = 0;
@@ -1333,8 +1334,7 @@ static bool ludusun_resolve(LayerList & ll, const std::string & name, TensorPlac
     if (w == "norm1") return norm(L.norm1, W);
     if (L.ff > 0) {
         if (w == "norm2") return norm(L.norm2, W);
-        if (w == "mlp.gate") return mat(L.gateup, 0, L.ff, W, 0);
-        if (w == "mlp.up") return mat(L.gateup, L.ff, L.ff, W, 1);
+        if (w == "mlp.gate" || w == "mlp.up") { o.row_step = 2; return mat(L.gateup, w == "mlp.up", L.ff, W, w == "mlp.up"); }   // FF_SILU: rows in turns
         if (w == "mlp.down") return mat(L.down, 0, W, L.ff, 0);
     }
     if (L.kind == MIX_ATTENTION) {
@@ -1621,8 +1621,8 @@ int ll_set_tensor(pb200_model * m, const char * name, int type, const void * hos
     }
     if (pl.mat) {
         const size_t es = esize(dtype);
-        if (pl.col0 < 0 || pl.col0 + pl.cols > pl.mat->K || pl.row0 + pl.rows > pl.mat->N || (size_t) pl.part >= pl.mat->filled.size()) return PB200_EINVAL;
-        CK(cudaMemcpy2D((uint8_t *) pl.mat->data + ((size_t) pl.row0 * pl.mat->K + (size_t) pl.col0) * es, (size_t) pl.mat->K * es, src, (size_t) pl.cols * es,
+        if (pl.col0 < 0 || pl.col0 + pl.cols > pl.mat->K || pl.row0 + (pl.rows - 1) * pl.row_step >= pl.mat->N || (size_t) pl.part >= pl.mat->filled.size()) return PB200_EINVAL;
+        CK(cudaMemcpy2D((uint8_t *) pl.mat->data + ((size_t) pl.row0 * pl.mat->K + (size_t) pl.col0) * es, (size_t) (pl.mat->K * pl.row_step) * es, src, (size_t) pl.cols * es,
                         (size_t) pl.cols * es, (size_t) pl.rows, cudaMemcpyHostToDevice));
         pl.mat->filled[(size_t) pl.part] = 1;
     } else if (pl.vrows > 0) {
@@ -2260,7 +2260,7 @@ static int mix_dual(pb200_model * m, const BatchView & b, bool prefill, const LR
     const float * r_gate = d.rec == REC_DELTA ? ll.big + d.c_rg : nullptr;   // gate logits of the recurrence's result
     int64_t ldrg = C;
     if (d.rec == REC_DELTA_CH) {   // decays per channel and gate logits from the inner values at the end of the projection
-        CAT(CAT_CONV);
+        CAT(CAT_LATENT);
         LowrankMaps mp;
         mp.za = ll.big + d.c_ra; mp.zg = ll.big + d.c_rg; mp.ldu = C;
         mp.wa = L.ra2.data; mp.wg = L.rg2.data; mp.ra = d.a_rank; mp.rg = d.g_rank;
@@ -2378,16 +2378,24 @@ static int ff_xielu(pb200_model * m, int T, LLayer & L, float * x) {
     }
     return launch_dense(ct, ll.act2, ff, L.down.data, ff, x, W, T, W, ff, nullptr, x, W, 1.f, st);
 }
-// ---- SiLU-gated feed-forward: x[t] += down(silu(gate(ll.act[t])) * up(ll.act[t])) ----
+// ---- SiLU-gated feed-forward: x[t] += down(silu(gate(ll.act[t])) * up(ll.act[t])); gate and up rows in turns, the gating is the product's epilogue
+// (PB200_FF_UNFUSED: a kernel of its own) ----
 static int ff_silu(pb200_model * m, int T, LLayer & L, float * x) {
     LayerList & ll = *m->ll;
     cudaStream_t st = m->stream;
     const int W = ll.width, ct = ll.ctype, ff = L.ff;
+    static const bool unfused = getenv("PB200_FF_UNFUSED") != nullptr;
     CAT(CAT_DENSE);
-    CK(launch_dense(ct, ll.act, W, L.gateup.data, W, ll.big, 2 * ff, T, 2 * ff, W, nullptr, nullptr, 0, 1.f, st));
-    CAT(CAT_ELEM);
-    CK(launch_silu_mul(ll.big, ll.act2, ct, T, ff, nullptr, nullptr, st));
-    CAT(CAT_DENSE);
+    if (unfused) {
+        CK(launch_dense(ct, ll.act, W, L.gateup.data, W, ll.big, 2 * ff, T, 2 * ff, W, nullptr, nullptr, 0, 1.f, st));
+        CAT(CAT_ELEM);
+        CK(launch_silu_mul(ll.big, ll.act2, ct, T, ff, nullptr, nullptr, st, 1));
+        CAT(CAT_DENSE);
+    } else {
+        DenseAct act;
+        act.silu_glu = 1; act.y = ll.act2; act.ldy = ff;
+        CK(launch_dense_act(ct, ll.act, W, L.gateup.data, W, act, T, 2 * ff, W, st));
+    }
     return launch_dense(ct, ll.act2, ff, L.down.data, ff, x, W, T, W, ff, nullptr, x, W, 1.f, st);
 }
 // ---- mixture of experts over ll.act.  accumulate: x[t] += shared(h) + sum_k w_k expert_k(h) (the stream itself); otherwise x receives the
@@ -2846,7 +2854,7 @@ int ll_debug_read(pb200_model * m, const char * name, float * host, int64_t n) {
     cudaSetDevice(m->device);
     CK(cudaStreamSynchronize(m->stream));
     if (strcmp(name, "profile") == 0) {   // ms of the last batch: dense, attention, convolution (or the map of a WKV mixer's decay), scan, norms, element-wise, head, [7] = total,
-        if (n > 10) return PB200_EINVAL;   // [8] = routed experts, [9] = the small steps around latent attention (norm + rotation, gather, folds)
+        if (n > 10) return PB200_EINVAL;   // [8] = routed experts, [9] = the small steps around latent attention (norm + rotation, gather, folds), the low-rank maps of a dual mixer
         memcpy(host, ll.prof_ms, (size_t) n * 4);
         return 0;
     }

@@ -46,10 +46,12 @@ int launch_dense(int type, const void * A, int64_t lda, const void * W, int64_t 
 // each) into the same rows of C, g < groups; start / count are device arrays and no group has more than max_rows rows.  Tensor-core
 // kernel only (bf16, aligned shapes): dense_grouped_ok says whether it applies; otherwise the caller multiplies group by group.
 int dense_grouped_ok(int type, int N, int K, int64_t lda, int64_t ldw, int64_t w_stride, const void * A, const void * W);
-// Epilogue of a product that feeds another one through xIELU: instead of C[t][n], y[t * ldy + n] = xielu(C[t][n]) in the operand type, with the
-// activation's two numbers at xielu (device).
+// Epilogue of a product that feeds another one, instead of C[t][n], in the operand type:
+//   xielu (the activation's two numbers, device):  y[t * ldy + n] = xielu(C[t][n])
+//   silu_glu (rows 2j of W are gates, rows 2j + 1 the values beside them):  y[t * ldy + j] = silu(C[t][2j]) * C[t][2j + 1]
 struct DenseAct {
     const float * xielu = nullptr;
+    int silu_glu = 0;
     void * y = nullptr;
     int64_t ldy = 0;
 };
@@ -310,7 +312,9 @@ int launch_moe_route_sigmoid(const void * h, int htype, const float * wr, const 
 int launch_moe_gateup_rows(const void * h, int type, const void * gateup, const int32_t * idx, const MoeParams & p, int width, void * y, int n_tokens,
                            cudaStream_t stream, const float * in_wt = nullptr);
 // y[r][j] = silu(s gu[r][j]) * (s gu[r][ff + j]),  s = in_wt ? in_wt[perm ? perm[r] : r] : 1      gu: [rows][2 ff] f32
-int launch_silu_mul(const float * gu, void * y, int otype, int n_rows, int ff, const float * in_wt, const int32_t * perm, cudaStream_t stream);
+// interleaved 1: silu(s gu[r][2j]) * (s gu[r][2j + 1]) instead
+int launch_silu_mul(const float * gu, void * y, int otype, int n_rows, int ff, const float * in_wt, const int32_t * perm, cudaStream_t stream,
+                    int interleaved = 0);
 // x[t] = base(x[t]) + sum_k wt[t][k] * down[idx[t][k]] y[t][k]      (k in the order of the choice)
 // base: MOE_ADD x[t] itself, MOE_SET zero, MOE_SCALE x[t] * xscale[t] (a gated shared expert's result waits in x)
 enum : int { MOE_ADD = 0, MOE_SET = 1, MOE_SCALE = 2 };

@@ -284,12 +284,14 @@ __global__ void k_moe_combine(const float * __restrict__ ds, const int32_t * __r
 }
 
 template <typename OT>
-__global__ void k_silu_mul(const float * __restrict__ gu, OT * __restrict__ y, int n_rows, int ff, const float * __restrict__ in_wt, const int32_t * __restrict__ perm) {
+__global__ void k_silu_mul(const float * __restrict__ gu, OT * __restrict__ y, int n_rows, int ff, const float * __restrict__ in_wt, const int32_t * __restrict__ perm,
+                           int interleaved) {
     const int64_t i = (int64_t) blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (int64_t) n_rows * ff) return;
     const int64_t r = i / ff, j = i - r * ff;
     const float s = in_wt ? in_wt[perm ? perm[r] : r] : 1.f;
-    put(y, i, silu_f(s * gu[r * 2 * ff + j]) * (s * gu[r * 2 * ff + ff + j]));
+    const float g = gu[r * 2 * ff + (interleaved ? 2 * j : j)], u = gu[r * 2 * ff + (interleaved ? 2 * j + 1 : ff + j)];
+    put(y, i, silu_f(s * g) * (s * u));
 }
 
 template <typename WT> bool vec_ok(const void * a, const void * b, int K) {
@@ -335,13 +337,14 @@ int launch_moe_route_sigmoid(const void * h, int htype, const float * wr, const 
     if (rc) return rc;
     return ck_launch([&] { k_moe_route_sigmoid<float><<<n_tokens, threads, smem, st>>>((const float *) h, wr, correction, p, width, shared_gate, idx, wt, sg_out); });
 }
-int launch_silu_mul(const float * gu, void * y, int otype, int n_rows, int ff, const float * in_wt, const int32_t * perm, cudaStream_t st) {
+int launch_silu_mul(const float * gu, void * y, int otype, int n_rows, int ff, const float * in_wt, const int32_t * perm, cudaStream_t st,
+                    int interleaved) {
     const int64_t n = (int64_t) n_rows * ff;
     if (n <= 0) return 0;
     const unsigned grid = (unsigned) ((n + 255) / 256);
     return ck_launch([&] {
-        if (otype == T_BF16) k_silu_mul<__nv_bfloat16><<<grid, 256, 0, st>>>(gu, (__nv_bfloat16 *) y, n_rows, ff, in_wt, perm);
-        else k_silu_mul<float><<<grid, 256, 0, st>>>(gu, (float *) y, n_rows, ff, in_wt, perm);
+        if (otype == T_BF16) k_silu_mul<__nv_bfloat16><<<grid, 256, 0, st>>>(gu, (__nv_bfloat16 *) y, n_rows, ff, in_wt, perm, interleaved);
+        else k_silu_mul<float><<<grid, 256, 0, st>>>(gu, (float *) y, n_rows, ff, in_wt, perm, interleaved);
     });
 }
 int launch_moe_gateup_rows(const void * h, int type, const void * gateup, const int32_t * idx, const MoeParams & p, int width, void * y, int n_tokens,

@@ -3,7 +3,8 @@ equal width / feed-forward / head sizes / number of layer runs: Vamidra beside t
 vamidra``), Mumizen beside Vamidra (``bench.py --arch mumizen``, :func:`run_mumizen`), Sapudra beside Vamidra and, for its experts, Mumizen
 (``bench.py --arch sapudra``, :func:`run_sapudra`), Zevedra beside Vamidra (attention, convolution, plain products) and Mumizen (recurrence,
 experts) (``bench.py --arch zevedra``, :func:`run_zevedra`), Ruvuvik beside Mumizen (latent attention, linear attention) and Vamidra
-(windowed attention) (``bench.py --arch ruvuvik``, :func:`run_ruvuvik`).  Prints one JSON line.
+(windowed attention) (``bench.py --arch ruvuvik``, :func:`run_ruvuvik`), Ludusun beside Vamidra, Mumizen (latent attention) and Zevedra (dual
+mixers, gated delta rule) (``bench.py --arch ludusun``, :func:`run_ludusun`).  Prints one JSON line.
 
 Per size: prompt tokens/s (one sequence of 512 and 2048 tokens) and decode tokens/s (batch 1 and 8 at a 1024-token context) of both
 models through their public entry points (host token ids in, host logits / greedy tokens out), the device time of a prompt and of a
@@ -72,6 +73,8 @@ def run(args, pkg, lib):
         return run_zevedra(args, pkg, lib)
     if args.arch == "ruvuvik":
         return run_ruvuvik(args, pkg, lib)
+    if args.arch == "ludusun":
+        return run_ludusun(args, pkg, lib)
     import numpy as np
     import torch
     hbm, tflops, src = peaks()
@@ -831,6 +834,173 @@ def run_ruvuvik(args, pkg, lib):
                 else:
                     r[f"decode_b{B}_scan_gbs"] = 3.0 * B * z["wkv_heads"] * z["wkv_dim"] ** 2 * 8.0 / pm["scan"] / 1e6
                 r[f"decode_b{B}_ms_per_step"] = v[f"decode_b{B}_ms_per_step"]
+            like[name] = r
+        out["like_kernels"] = like
+        res["sizes"][key] = out
+    res["gpu_launches"] = int(lib.c.pb200_kernel_launches())
+    print(json.dumps(res))
+    return res
+
+
+# ---------------------------------------------------------------------------------------------------------------
+LUDUSUN_SIZES = {
+    "w2048": dict(heads=16, dim=128, vdim=128, kv_rank=512, q_rank=1024, r_heads=16, r_kv=4, r_dim=128, r_vdim=128, conv=4, rank=128),
+    "w4096": dict(heads=32, dim=128, vdim=128, kv_rank=512, q_rank=1536, r_heads=32, r_kv=8, r_dim=128, r_vdim=128, conv=4, rank=128),
+}
+
+
+def ludusun_layers(s, z):
+    """One layer of each mixer at the width / feed-forward / head sizes of SIZES."""
+    mlp, D = {"kind": "dense", "ff": s["ff"]}, s["dim"]
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5,
+                     "rot": {"base": 500000.0, "dims": D, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"heads": z["heads"], "dim": z["dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"], "q_rank": z["q_rank"], "scale": z["dim"] ** -0.5,
+                     "mask": {"size": s["window"]}}}
+    par = {"type": "parallel", "mlp": mlp,
+           "mixer": {"left": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5, "q_temp": {"coef": 0.1, "every": 512}},
+                     "right": {"heads": z["r_heads"], "kv_heads": z["r_kv"], "dim": z["r_dim"], "vdim": z["r_vdim"], "conv": z["conv"], "decay_rank": z["rank"],
+                               "gate_rank": z["rank"]}, "left_scale": 0.7, "right_scale": 0.7}}
+    return {"attention": att, "latent": lat, "parallel": par}
+
+
+def ludusun_config(s, layers):
+    return {"architecture": "Ludusun", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "logit_softcap": 30.0, "layers": layers}
+
+
+def reading(layer, of):
+    return dict(layer, mixer=dict(layer["mixer"], kv_from=of))
+
+
+def ludusun_products(s, cfg, prompt):
+    """(N, K) of the dense products of one token through all layer runs (head and the fp32 low-rank maps not included)."""
+    W, out = s["width"], []
+    for l in cfg["layers"]:
+        m = l["mixer"]
+        if l["type"] == "latent_attention":
+            H = m["heads"]
+            out += [(m["q_rank"] + H + m["kv_rank"], W), (H * m["dim"], m["q_rank"]), (W, H * m["vdim"])]
+            if prompt:
+                out += [(H * (m["dim"] + m["vdim"]), m["kv_rank"])]
+        elif l["type"] == "attention":
+            kv = m["kv_heads"] * (m["dim"] + m["vdim"]) if m.get("kv_from") is None else 0
+            out += [(m["heads"] * m["dim"] + kv, W), (W, m["heads"] * m["vdim"])]
+        else:
+            a, r = m["left"], m["right"]
+            RV = r["heads"] * r["vdim"]
+            out += [(2 * a["heads"] * a["dim"] + a["kv_heads"] * a["dim"] + 2 * r["kv_heads"] * r["dim"] + RV + r["heads"] + r["decay_rank"] + r["gate_rank"], W),
+                    (W, a["heads"] * a["dim"] + RV)]
+        if l.get("mlp"):
+            out += [(2 * l["mlp"]["ff"], W), (W, l["mlp"]["ff"])]
+    return out
+
+
+def run_ludusun(args, pkg, lib):
+    """Ludusun beside the models it resembles at equal width / feed-forward / head sizes and six layer runs each: Vamidra (windowed attention, gated
+    feed-forward), Mumizen (latent attention with a query latent) and Zevedra (dual mixers).  Whole-model prompt and decode throughput through the
+    public entry points; for the like kernels, models whose three layers all have ONE mixer: device time per kernel category turned into a distance
+    from the roofline."""
+    import numpy as np
+    import torch
+    hbm, tflops, src = peaks()
+    res = {"metric": "Ludusun prompt / decode throughput beside Vamidra, Mumizen and Zevedra at equal size", "impl": "b200", "arch": "Ludusun", "n_gpus": 1,
+           "dtype": "bf16", "data": "synthetic random weights", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": src}, "sizes": {}}
+    rng = np.random.default_rng(0)
+    CTX = 1024
+
+    def measured(cfg):
+        m = pkg.Model.from_config(cfg, dtype="bfloat16", n_ctx=4096, n_seq=16)
+        m.synth(0, 7)
+        m.finalize()
+        v = measure(m, cfg["vocab"], args, rng, CTX)
+        m.close()
+        torch.cuda.empty_cache()
+        return v
+
+    def dense_fracs(a, prompt_shapes, step_shapes, extra):
+        for T in (512, 2048):
+            a[f"prompt{T}_dense_frac_of_tensor_peak"] = 2.0 * sum(n * k for n, k in prompt_shapes) * T / a[f"prompt{T}_device_ms"]["dense"] / 1e9 / tflops
+        wb = 2.0 * sum(n * k for n, k in step_shapes)
+        a["weight_bytes_per_token"] = wb + 2.0 * extra
+        for B in (1, 8):
+            a[f"decode_b{B}_dense_frac_of_hbm_peak"] = wb / a[f"decode_b{B}_device_ms"]["dense"] / 1e6 / hbm
+            a[f"decode_b{B}_whole_step_frac_of_hbm_peak"] = a["weight_bytes_per_token"] / a[f"decode_b{B}_ms_per_step"] / 1e6 / hbm
+
+    for key in ([args.arch_size] if args.arch_size != "all" else list(SIZES)):
+        s, z, mz, zz = SIZES[key], LUDUSUN_SIZES[key], MUMIZEN_SIZES[key], ZEVEDRA_SIZES[key]
+        W, V, D, H, G = s["width"], s["vocab"], s["dim"], s["heads"], s["kv_heads"]
+        L = ludusun_layers(s, z)
+        out = {"config": dict(z, width=W, ff=s["ff"], kv_heads=G, window=s["window"], vocab=V), "layers": 6}
+        # ---------------- whole models, six layer runs each ----------------
+        cfg = ludusun_config(s, [L["attention"], L["latent"], L["parallel"], reading(L["attention"], 0), L["latent"], L["parallel"]])
+        a = measured(cfg)
+        dense_fracs(a, ludusun_products(s, cfg, True), ludusun_products(s, cfg, False), V * W)
+        out["ludusun"] = a
+        vcfg = vamidra_config(s)
+        b = measured(vcfg)
+        dense_fracs(b, dense_shapes(s, vcfg), dense_shapes(s, vcfg), V * W)
+        out["vamidra"] = b
+        mcfg = mumizen_config(s, mz)
+        ml = {l["type"]: dict(l, mlp=mcfg["layers"][0]["mlp"]) for l in mcfg["layers"][:3]}
+        lin, mlat = ml["retention"], ml["latent_attention"]
+        mcfg = dict(mcfg, layers=[mlat, lin, mlat, lin, lin, lin])       # dense feed-forward in every layer
+        c = measured(mcfg)
+        dense_fracs(c, mumizen_products(mcfg, True)[0], mumizen_products(mcfg, False)[0], V * W)
+        out["mumizen"] = c
+        zcfg = zevedra_config(s, zz)
+        zprods, zexpert, _ = zevedra_products(zcfg)
+        d = measured(zcfg)
+        dense_fracs(d, zprods, zprods, V * W + zexpert)
+        out["zevedra"] = d
+        # ---------------- one mixer at a time, three layers; dual mixers without feed-forward ----------------
+        like = {}
+        bare = lambda l: dict(l, mlp=None)   # noqa: E731
+        plain = dict(zcfg, loop=None)
+        probes = {"ludusun_attention": ludusun_config(s, [L["attention"]] * 3), "ludusun_attention_reading": ludusun_config(s, [L["attention"]] + [reading(L["attention"], 0)] * 2),
+                  "vamidra_attention": dict(vcfg, layers=[vcfg["layers"][0]] * 3, loop=None),
+                  "ludusun_latent": ludusun_config(s, [L["latent"]] * 3), "mumizen_latent": dict(mcfg, layers=[mlat] * 3),
+                  "ludusun_parallel": ludusun_config(s, [bare(L["parallel"])] * 3), "zevedra_parallel": dict(plain, layers=[bare(zcfg["layers"][1])] * 3),
+                  "zevedra_parallel_2": dict(plain, layers=[bare(zcfg["layers"][0])] * 3)}
+        rec = 3.0 * z["r_heads"] * z["r_dim"] * z["r_vdim"]
+        OD, RQ, RV = H * D, z["r_kv"] * z["r_dim"], z["r_heads"] * z["r_vdim"]
+        for name, pc in probes.items():
+            v = measured(pc)
+            r = {}
+            windowed = name in ("vamidra_attention", "ludusun_latent", "zevedra_parallel")
+            keep = s["keep_first"] if name == "vamidra_attention" else 0
+            for T in (512, 2048):
+                pm = v[f"prompt{T}_device_ms"]
+                r[f"prompt{T}_device_ms"] = pm
+                vis = sum(min(i + 1, s["window"]) + max(0, min(keep, i + 1 - s["window"])) for i in range(T)) if windowed else T * (T + 1) // 2
+                dq, dv, hq = (z["dim"], z["vdim"], z["heads"]) if name == "ludusun_latent" else (mz["dim"] + mz["rot_dim"], mz["vdim"], mz["heads"]) if name == "mumizen_latent" else (D, D, H)
+                r[f"prompt{T}_attention_tflops"] = 3 * 2.0 * hq * (dq + dv) * vis / pm["attention"] / 1e9
+                if "parallel" in name:
+                    r[f"prompt{T}_scan_state_updates_per_ns"] = rec * T / pm["scan"] / 1e6
+                if name in ("ludusun_parallel", "zevedra_parallel"):
+                    ch = 2 * RQ + RV + (0 if name.startswith("lud") else OD + 2 * G * D)
+                    r[f"prompt{T}_conv_gbs"] = 3.0 * ch * T * 8.0 / pm["conv"] / 1e6
+                if name == "ludusun_parallel":
+                    r[f"prompt{T}_maps_tflops"] = 3 * 2.0 * z["rank"] * (z["r_heads"] * z["r_dim"] + RV) * T / pm["latent_steps"] / 1e9
+                if name.startswith(("ludusun_attention", "vamidra_attention")):   # two norms a layer; Vamidra: four and two residual sums
+                    r[f"prompt{T}_norm_gbs"] = 3 * T * W * (12.0 if name.startswith("lud") else 36.0) / pm["norm"] / 1e6
+            if name.startswith("ludusun"):
+                dense_fracs(v, ludusun_products(s, pc, True), ludusun_products(s, pc, False), V * W)
+            elif name == "vamidra_attention":
+                one = [(H * D + 2 * G * D + H, W), (W, H * D), (2 * s["ff"], W), (W, s["ff"])]
+                dense_fracs(v, one * 3, one * 3, V * W)
+            elif name == "mumizen_latent":
+                dense_fracs(v, mumizen_products(pc, True)[0], mumizen_products(pc, False)[0], V * W)
+            for B in (1, 8):
+                pm = v[f"decode_b{B}_device_ms"]
+                r[f"decode_b{B}_device_ms"] = pm
+                rows = min(CTX, s["window"] + keep) if windowed else CTX
+                per = z["kv_rank"] if name == "ludusun_latent" else mz["kv_rank"] + mz["rot_dim"] if name == "mumizen_latent" else G * D if name == "ludusun_parallel" else 2 * G * D
+                r[f"decode_b{B}_attention_gbs"] = 3.0 * B * rows * per * 4.0 / pm["attention"] / 1e6
+                if "parallel" in name:
+                    r[f"decode_b{B}_scan_gbs"] = B * rec * 8.0 / pm["scan"] / 1e6
+                r[f"decode_b{B}_ms_per_step"] = v[f"decode_b{B}_ms_per_step"]
+            r.update({k: x for k, x in v.items() if "_dense_frac" in k or k.endswith("tok_s")})
             like[name] = r
         out["like_kernels"] = like
         res["sizes"][key] = out
