@@ -49,7 +49,7 @@ __device__ __forceinline__ void rope_q_row(float * __restrict__ row, int pos, co
 }
 
 template <typename OT>
-__global__ void __launch_bounds__(256) k_latent_prep(float * __restrict__ proj, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
+__global__ void __launch_bounds__(1024) k_latent_prep(float * __restrict__ proj, const int32_t * __restrict__ slot, const int32_t * __restrict__ off,
                                                      const int32_t * __restrict__ pos0, const int32_t * __restrict__ entry_of, LatentParams p,
                                                      const float * __restrict__ wq, const float * __restrict__ wkv, const float * __restrict__ freq, float eps,
                                                      OT * __restrict__ cq, float * __restrict__ cache, int64_t slot_stride, OT * __restrict__ lat,
@@ -391,12 +391,13 @@ int launch_latent_prep(float * proj, const BatchView & b, const LatentParams & p
                        void * cq, int otype, float * cache, int64_t slot_stride, void * lat, float * kr, int turn_q, cudaStream_t st) {
     if (b.n_tokens <= 0) return 0;
     if (!latent_ok(p) || (p.own_kv && (!cache || !wkv)) || (p.q_rank > 0 && (!wq || !cq)) || (p.rot_dims > 0 && !freq)) return (int) cudaErrorInvalidValue;
+    const int threads = row_threads(b.n_tokens, std::max(p.q_rank, p.kv_rank));
     return ck_launch([&] {
         if (otype == T_BF16)
-            k_latent_prep<__nv_bfloat16><<<b.n_tokens, 256, 0, st>>>(proj, b.slot, b.off, b.pos0, b.entry_of, p, wq, wkv, freq, eps, (__nv_bfloat16 *) cq, cache,
+            k_latent_prep<__nv_bfloat16><<<b.n_tokens, threads, 0, st>>>(proj, b.slot, b.off, b.pos0, b.entry_of, p, wq, wkv, freq, eps, (__nv_bfloat16 *) cq, cache,
                                                                      slot_stride, (__nv_bfloat16 *) lat, kr, turn_q);
         else
-            k_latent_prep<float><<<b.n_tokens, 256, 0, st>>>(proj, b.slot, b.off, b.pos0, b.entry_of, p, wq, wkv, freq, eps, (float *) cq, cache, slot_stride,
+            k_latent_prep<float><<<b.n_tokens, threads, 0, st>>>(proj, b.slot, b.off, b.pos0, b.entry_of, p, wq, wkv, freq, eps, (float *) cq, cache, slot_stride,
                                                              (float *) lat, kr, turn_q);
     });
 }

@@ -540,11 +540,15 @@ __global__ void __launch_bounds__(256) k_attn_window_prefill_tiled(const AttnIO 
 // decode: CTA (head, entry, split).  Warp w takes cache rows 4 w .. 4 w + 3 of the split's chunk, then 4 * warps further on, ...: the lanes
 // split the key's dimensions (coalesced row reads, four rows in flight), the score is a warp sum, the running max / sum are uniform over the
 // warp, and every lane accumulates its share of the value dimensions.  The warps' partial softmax states are merged in shared memory.  With
-// one split (32 warps over all rows) the CTA writes the output; with several (8 warps over `chunk` rows each) it writes its partial state
+// one split (16 warps over all rows) the CTA writes the output; with several (8 warps over `chunk` rows each) it writes its partial state
 // [max, sum, weighted values] and k_attn_decode_merge finishes.  The number of splits comes from the cache's row count alone (the layer's
 // window and the context size), so a sequence's result does not depend on the batch around it.
-constexpr int DEC_WARPS = 32, DEC_ROWS = 4, DEC_SPLIT_WARPS = 8;
-template <typename OT, int NV>
+// A split without rows writes nothing, and the merge does not read it.  NV <= 4: the value entries of a step's rows are on their way before the
+// scores are summed.  TIED (a key is its own value, 16-byte rows): the key's registers serve as the value, lane entry 4 c + i of a head being d =
+// 128 c + 4 lane + i.
+constexpr int DEC_WARPS = 16, DEC_ROWS = 4, DEC_SPLIT_WARPS = 8;
+__device__ __forceinline__ int dec_rows_used(const AttnParams & a, int pi) { return min(a.cache_rows, (a.chunk > 0 ? pi % a.chunk : pi) + 1); }   // a chunk's rows start at row 0 of the ring
+template <typename OT, int NV, bool TIED>
 __global__ void __launch_bounds__(DEC_WARPS * 32) k_attn_window_decode(const AttnIO io, const int32_t * __restrict__ slot,
                                                                        const int32_t * __restrict__ off, const int32_t * __restrict__ pos0, AttnParams a,
                                                                        const float * __restrict__ kcache, const float * __restrict__ vcache,
@@ -562,15 +566,19 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) k_attn_window_decode(const Att
     float * qs = sm;                       // [D], scaled
     float * mm = qs + ((D + 3) & ~3);      // [nw] max, [nw] sum
     float * accs = mm + 2 * nw;            // [nw][NV*32]
+    const int rows_used = dec_rows_used(a, pi);
+    const int r_begin = gridDim.z > 1 ? blockIdx.z * chunk : 0, r_end = gridDim.z > 1 ? min(rows_used, r_begin + chunk) : rows_used;
+    if (r_begin >= rows_used) return;      // the whole CTA
+    auto d_of = [&](int c) { return TIED ? 128 * (c >> 2) + 4 * lane + (c & 3) : lane + 32 * c; };   // value dimension of accumulator c
     for (int d = threadIdx.x; d < D; d += blockDim.x) qs[d] = io.q[(int64_t) t * io.ldq + h * D + d] * a.scale;
     __syncthreads();
     const float * kc = kcache + (int64_t) slot[e] * slot_stride, * vc = vcache + (int64_t) slot[e] * slot_stride;
     float m = -INFINITY, l = 0.f, acc[NV];
 #pragma unroll
     for (int c = 0; c < NV; c++) acc[c] = 0.f;
-    const int rows_used = min(a.cache_rows, (a.chunk > 0 ? pi % a.chunk : pi) + 1);   // a chunk's rows start at row 0 of the ring
-    const int r_begin = gridDim.z > 1 ? blockIdx.z * chunk : 0, r_end = gridDim.z > 1 ? min(rows_used, r_begin + chunk) : rows_used;
     const bool vec4 = (D & 3) == 0 && (KD & 3) == 0;
+    constexpr bool AHEAD = !TIED && NV <= 4;
+    float val[TIED || AHEAD ? DEC_ROWS : 1][TIED || AHEAD ? NV : 1];
     for (int r0 = r_begin + warp * DEC_ROWS; r0 < r_end; r0 += nw * DEC_ROWS) {
         // DEC_ROWS rows per step so that their loads are in flight together; which position does row r hold right now?
         float sc[DEC_ROWS];
@@ -590,7 +598,21 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) k_attn_window_decode(const Att
             float s = 0.f;
             if (valid) {
                 const float * kr = kc + (int64_t) r * KD + kvh * D;
-                if (vec4) {
+                if constexpr (AHEAD) {
+                    const float * vr = vc + (int64_t) r * VD + kvh * DV;
+#pragma unroll
+                    for (int c = 0; c < NV; c++) val[j][c] = lane + 32 * c < DV ? vr[lane + 32 * c] : 0.f;
+                }
+                if constexpr (TIED) {
+#pragma unroll
+                    for (int c = 0; c < NV; c += 4) {
+                        const int d = 32 * c + 4 * lane;
+                        const float4 kv = d < D ? *reinterpret_cast<const float4 *>(kr + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                        const float4 qv = d < D ? *reinterpret_cast<const float4 *>(qs + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+                        s = fmaf(qv.x, kv.x, s); s = fmaf(qv.y, kv.y, s); s = fmaf(qv.z, kv.z, s); s = fmaf(qv.w, kv.w, s);
+                        val[j][c] = kv.x; val[j][(c + 1) % NV] = kv.y; val[j][(c + 2) % NV] = kv.z; val[j][(c + 3) % NV] = kv.w;
+                    }
+                } else if (vec4) {
                     for (int d = lane * 4; d < D; d += 128) {
                         const float4 kv = *reinterpret_cast<const float4 *>(kr + d);
                         const float4 qv = *reinterpret_cast<const float4 *>(qs + d);
@@ -621,11 +643,14 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) k_attn_window_decode(const Att
         l = l * corr + psum;
 #pragma unroll
         for (int c = 0; c < NV; c++) {
-            const int d = lane + 32 * c;
+            const int d = d_of(c);
             float v = acc[c] * corr;
 #pragma unroll
             for (int j = 0; j < DEC_ROWS; j++)
-                if (pj[j] != 0.f && d < DV) v = fmaf(pj[j], vc[(int64_t) (r0 + j) * VD + kvh * DV + d], v);
+                if (pj[j] != 0.f && d < DV) {
+                    if constexpr (TIED || AHEAD) v = fmaf(pj[j], val[j][c], v);
+                    else v = fmaf(pj[j], vc[(int64_t) (r0 + j) * VD + kvh * DV + d], v);
+                }
             acc[c] = v;
         }
         m = mn;
@@ -634,62 +659,65 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) k_attn_window_decode(const Att
 #pragma unroll
     for (int c = 0; c < NV; c++) accs[warp * NV * 32 + c * 32 + lane] = acc[c];
     __syncthreads();
-    if (warp == 0) {
-        float M = -INFINITY;
-        for (int w = 0; w < nw; w++) M = fmaxf(M, mm[w]);
-        float L = 0.f, o[NV];
-#pragma unroll
-        for (int c = 0; c < NV; c++) o[c] = 0.f;
-        for (int w = 0; w < nw; w++) {
-            if (mm[w] == -INFINITY) continue;
-            const float f = expf(mm[w] - M);
-            L += mm[nw + w] * f;
-#pragma unroll
-            for (int c = 0; c < NV; c++) o[c] = fmaf(accs[w * NV * 32 + c * 32 + lane], f, o[c]);
-        }
-        if (gridDim.z > 1) {   // partial state of this split
-            float * pp = part + (((int64_t) e * a.heads + h) * gridDim.z + blockIdx.z) * (DV + 2);
-            if (lane == 0) { pp[0] = M; pp[1] = L; }
-#pragma unroll
-            for (int c = 0; c < NV; c++) {
-                const int d = lane + 32 * c;
-                if (d < DV) pp[2 + d] = o[c];
-            }
-            return;
-        }
-        if (a.sink && M != -INFINITY) L += expf(attn_sink(io, h) - M);
-        const float inv = L > 0.f ? 1.f / L : 0.f;
-#pragma unroll
-        for (int c = 0; c < NV; c++) {
-            const int d = lane + 32 * c;
-            if (d < DV) put(out, (int64_t) t * (a.heads * DV) + h * DV + d, o[c] * inv * attn_gate(io, t, h, d, DV));
-        }
+    // the warps' states meet: a thread per accumulator slot
+    float M = -INFINITY;
+    for (int w = 0; w < nw; w++) M = fmaxf(M, mm[w]);
+    float L = 0.f;
+    for (int w = 0; w < nw; w++)
+        if (mm[w] != -INFINITY) L += mm[nw + w] * expf(mm[w] - M);
+    const bool partial = gridDim.z > 1;
+    float * pp = partial ? part + (((int64_t) e * a.heads + h) * gridDim.z + blockIdx.z) * (DV + 2) : nullptr;   // state of this split
+    if (partial && threadIdx.x == 0) { pp[0] = M; pp[1] = L; }
+    if (!partial && a.sink && M != -INFINITY) L += expf(attn_sink(io, h) - M);
+    const float inv = L > 0.f ? 1.f / L : 0.f;
+    for (int i = threadIdx.x; i < NV * 32; i += blockDim.x) {
+        const int c = i >> 5, ln = i & 31, d = TIED ? 128 * (c >> 2) + 4 * ln + (c & 3) : ln + 32 * c;
+        if (d >= DV) continue;
+        float o = 0.f;
+        for (int w = 0; w < nw; w++)
+            if (mm[w] != -INFINITY) o = fmaf(accs[w * NV * 32 + i], expf(mm[w] - M), o);
+        if (partial) pp[2 + d] = o;
+        else put(out, (int64_t) t * (a.heads * DV) + h * DV + d, o * inv * attn_gate(io, t, h, d, DV));
     }
 }
 
-// merges the partial softmax states of a (head, entry): grid (heads, entries), one thread per value dimension
+// merges the partial softmax states of a (head, entry): grid (heads, entries).  A lane of the first warp weighs splits lane and lane + 32 (64 at
+// most), then one thread per value dimension sums the splits that hold rows, eight loads in flight.
 template <typename OT>
-__global__ void __launch_bounds__(128) k_attn_decode_merge(const AttnIO io, const int32_t * __restrict__ off, AttnParams a, const float * __restrict__ part,
-                                                           int splits, OT * __restrict__ out) {
+__global__ void __launch_bounds__(128) k_attn_decode_merge(const AttnIO io, const int32_t * __restrict__ off, const int32_t * __restrict__ pos0, AttnParams a,
+                                                           const float * __restrict__ part, int all_splits, int chunk, OT * __restrict__ out) {
+    __shared__ float w[64];
     const int e = blockIdx.y, h = blockIdx.x, DV = a.vdim;
     const int t = off[e];
-    const float * pp = part + ((int64_t) e * a.heads + h) * splits * (DV + 2);
-    float M = -INFINITY;
-    for (int s = 0; s < splits; s++) M = fmaxf(M, pp[(int64_t) s * (DV + 2)]);
-    float L = 0.f;
-    for (int s = 0; s < splits; s++) {
-        const float ms = pp[(int64_t) s * (DV + 2)];
-        if (ms != -INFINITY) L += pp[(int64_t) s * (DV + 2) + 1] * expf(ms - M);
+    const int splits = (dec_rows_used(a, pos0[e]) + chunk - 1) / chunk;   // the rest hold no rows
+    const int64_t stride = DV + 2;
+    const float * pp = part + ((int64_t) e * a.heads + h) * all_splits * stride;
+    if (threadIdx.x < 32) {
+        const int lane = threadIdx.x;
+        const bool ok0 = lane < splits, ok1 = lane + 32 < splits;
+        const float m0 = ok0 ? pp[lane * stride] : -INFINITY, m1 = ok1 ? pp[(lane + 32) * stride] : -INFINITY;
+        const float l0 = ok0 ? pp[lane * stride + 1] : 0.f, l1 = ok1 ? pp[(lane + 32) * stride + 1] : 0.f;
+        const float M = wmax(fmaxf(m0, m1));
+        const float f0 = m0 == -INFINITY ? 0.f : expf(m0 - M), f1 = m1 == -INFINITY ? 0.f : expf(m1 - M);
+        float L = wsum(l0 * f0 + l1 * f1);
+        if (a.sink && M != -INFINITY) L += expf(attn_sink(io, h) - M);
+        w[lane] = L > 0.f ? f0 / L : 0.f;
+        w[lane + 32] = L > 0.f ? f1 / L : 0.f;
     }
-    if (a.sink && M != -INFINITY) L += expf(attn_sink(io, h) - M);
-    const float inv = L > 0.f ? 1.f / L : 0.f;
+    __syncthreads();
     for (int d = threadIdx.x; d < DV; d += blockDim.x) {
+        const float * pd = pp + 2 + d;
         float o = 0.f;
-        for (int s = 0; s < splits; s++) {
-            const float ms = pp[(int64_t) s * (DV + 2)];
-            if (ms != -INFINITY) o = fmaf(pp[(int64_t) s * (DV + 2) + 2 + d], expf(ms - M), o);
+        int s = 0;
+        for (; s + 7 < splits; s += 8) {
+            float v[8];
+#pragma unroll
+            for (int u = 0; u < 8; u++) v[u] = pd[(s + u) * stride];
+#pragma unroll
+            for (int u = 0; u < 8; u++) o = fmaf(w[s + u], v[u], o);
         }
-        put(out, (int64_t) t * (a.heads * DV) + h * DV + d, o * inv * attn_gate(io, t, h, d, DV));
+        for (; s < splits; s++) o = fmaf(w[s], pd[s * stride], o);
+        put(out, (int64_t) t * (a.heads * DV) + h * DV + d, o * attn_gate(io, t, h, d, DV));
     }
 }
 
@@ -1049,29 +1077,33 @@ int launch_attn_prefill_io(const AttnIO & io, const BatchView & b, const AttnPar
     else PB_NV_DISPATCH(nv, return (attn_prefill_typed<float, NV>(io, b, a, (float *) out, st)));
     return 0;
 }
-template <typename OT, int NV>
+template <typename OT, int NV, bool TIED>
 static int attn_decode_typed(const AttnIO & io, const BatchView & b, const AttnParams & a, const float * kc, const float * vc, int64_t stride, OT * out,
                              float * part, cudaStream_t st) {
     const int splits = part ? attn_decode_splits(a.cache_rows) : 1;
     const int nw = splits > 1 ? DEC_SPLIT_WARPS : DEC_WARPS;
     const size_t smem = ((size_t) ((a.dim + 3) & ~3) + 2 * nw + (size_t) nw * NV * 32) * sizeof(float);
-    int rc = raise_smem(k_attn_window_decode<OT, NV>, ((size_t) ((a.dim + 3) & ~3) + 2 * DEC_WARPS + (size_t) DEC_WARPS * NV * 32) * sizeof(float));
+    int rc = raise_smem(k_attn_window_decode<OT, NV, TIED>, ((size_t) ((a.dim + 3) & ~3) + 2 * DEC_WARPS + (size_t) DEC_WARPS * NV * 32) * sizeof(float));
     if (rc) return rc;
     const dim3 grid((unsigned) a.heads, (unsigned) b.n_entries, (unsigned) splits);
     rc = ck_launch([&] {
-        k_attn_window_decode<OT, NV><<<grid, nw * 32, smem, st>>>(io, b.slot, b.off, b.pos0, a, kc, vc, stride, out, part, attn_decode_chunk(a.cache_rows));
+        k_attn_window_decode<OT, NV, TIED><<<grid, nw * 32, smem, st>>>(io, b.slot, b.off, b.pos0, a, kc, vc, stride, out, part, attn_decode_chunk(a.cache_rows));
     });
     if (rc || splits == 1) return rc;
     const dim3 mgrid((unsigned) a.heads, (unsigned) b.n_entries);
-    return ck_launch([&] { k_attn_decode_merge<OT><<<mgrid, 128, 0, st>>>(io, b.off, a, part, splits, out); });
+    return ck_launch([&] { k_attn_decode_merge<OT><<<mgrid, 128, 0, st>>>(io, b.off, b.pos0, a, part, splits, attn_decode_chunk(a.cache_rows), out); });
 }
 int launch_attn_decode_io(const AttnIO & io, const BatchView & b, const AttnParams & a, const float * kcache, const float * vcache, int64_t slot_stride,
                           void * out, int otype, cudaStream_t st, float * part) {
     if (b.n_tokens <= 0) return 0;
     if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads != 0 || a.dim <= 0 || a.vdim <= 0) return (int) cudaErrorInvalidValue;
     const int nv = (a.vdim + 31) / 32;
-    if (otype == T_BF16) PB_NV_DISPATCH(nv, return (attn_decode_typed<__nv_bfloat16, NV>(io, b, a, kcache, vcache, slot_stride, (__nv_bfloat16 *) out, part, st)));
-    else PB_NV_DISPATCH(nv, return (attn_decode_typed<float, NV>(io, b, a, kcache, vcache, slot_stride, (float *) out, part, st)));
+    if (a.tied_v && kcache == vcache && a.dim <= 128 && a.dim % 4 == 0 && io.k_row % 4 == 0 && slot_stride % 4 == 0 && ((uintptr_t) kcache & 15) == 0) {
+        if (otype == T_BF16) return attn_decode_typed<__nv_bfloat16, 4, true>(io, b, a, kcache, vcache, slot_stride, (__nv_bfloat16 *) out, part, st);
+        return attn_decode_typed<float, 4, true>(io, b, a, kcache, vcache, slot_stride, (float *) out, part, st);
+    }
+    if (otype == T_BF16) PB_NV_DISPATCH(nv, return (attn_decode_typed<__nv_bfloat16, NV, false>(io, b, a, kcache, vcache, slot_stride, (__nv_bfloat16 *) out, part, st)));
+    else PB_NV_DISPATCH(nv, return (attn_decode_typed<float, NV, false>(io, b, a, kcache, vcache, slot_stride, (float *) out, part, st)));
     return 0;
 }
 
