@@ -204,13 +204,15 @@ __global__ void __launch_bounds__(TC_THREADS, 1) k_dense_tc(const __grid_constan
                 : "memory");
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             if (P.act.silu_glu) {   // neighbouring lanes hold a gate and its value: of two tokens the even lane finishes the first, the odd one the second
-                const bool odd = lane & 1;
+                const bool odd = lane & 1, ok = n < P.N && !*cta_abort;
+                __nv_bfloat16 * yp = ya + (int64_t) (t0 + c0 + (odd ? 1 : 0)) * P.act.ldy + n / 2;
 #pragma unroll
                 for (int i = 0; i < 16; i += 2) {
                     const float mine = P.alpha * __uint_as_float(odd ? v[i + 1] : v[i]);
                     const float other = __shfl_xor_sync(0xffffffffu, P.alpha * __uint_as_float(odd ? v[i] : v[i + 1]), 1);
-                    const int t = t0 + c0 + i + (odd ? 1 : 0);
-                    if (n < P.N && t < Tn && !*cta_abort) put(ya, (int64_t) t * P.act.ldy + n / 2, odd ? silu_f(other) * mine : silu_f(mine) * other);
+                    const float g = odd ? other : mine, u = odd ? mine : other;
+                    // the fast exponential and quotient are far more accurate than the operand type the result is rounded to
+                    if (ok && t0 + c0 + i + (odd ? 1 : 0) < Tn) yp[(int64_t) i * P.act.ldy] = __float2bfloat16_rn(__fdividef(g, 1.f + __expf(-g)) * u);
                 }
                 continue;
             }

@@ -17,7 +17,8 @@
 // attention -> the fp32 state [heads][dim][vdim], latent attention -> one row [latent | rotated key part] per position (a layer that
 // reads another layer's latent has none of its own), token shift -> the normed input of the last token, dual mixer -> K and V rows, the
 // last taps-1 convolution inputs of both branches and the recurrence's fp32 state, chunked attention -> K and V rows of one chunk, WKV -> the
-// fp32 state [heads][dim][dim] and the normed input of the last token.  A slot's arena is zeroed when it is handed out, so a
+// fp32 state [heads][dim][dim] and the normed input of the last token.  Keys that are values have K rows alone, a window over latents keeps a
+// ring of its rows, attention that reads another layer's keys and values has none.  A slot's arena is zeroed when it is handed out, so a
 // reused slot starts like a new one; the token before a sequence's next one (bigram embedding) is kept per slot on the host.
 //
 // Precision: the residual stream, norms, attention scores / weights, recurrent state and everything that feeds the recurrence are

@@ -854,7 +854,7 @@ def ludusun_layers(s, z):
     mlp, D = {"kind": "dense", "ff": s["ff"]}, s["dim"]
     att = {"type": "attention", "mlp": mlp,
            "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5,
-                     "rot": {"base": 500000.0, "dims": D, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}}
+                     "rot": {"base": 1000000.0, "dims": D, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}}
     lat = {"type": "latent_attention", "mlp": mlp,
            "mixer": {"heads": z["heads"], "dim": z["dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"], "q_rank": z["q_rank"], "scale": z["dim"] ** -0.5,
                      "mask": {"size": s["window"]}}}
@@ -866,7 +866,7 @@ def ludusun_layers(s, z):
 
 
 def ludusun_config(s, layers):
-    return {"architecture": "Ludusun", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "logit_softcap": 30.0, "layers": layers}
+    return {"architecture": "Ludusun", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "logit_softcap": 25.0, "layers": layers}
 
 
 def reading(layer, of):
